@@ -1,7 +1,7 @@
-from .manager import (CacheManager, OutOfPages, OutOfStateSlots, PageAllocator, PagedLayerCache, RequestCache,
+from .manager import (CacheManager, JointLayerCache, OutOfPages, OutOfStateSlots, PageAllocator, PagedLayerCache, RequestCache,
                       StateLayerCache, group_key)
 
 from .radix import PrefixTree
 
-__all__ = ["PrefixTree", "CacheManager", "OutOfPages", "OutOfStateSlots", "PageAllocator", "PagedLayerCache", "RequestCache",
+__all__ = ["PrefixTree", "CacheManager", "JointLayerCache", "OutOfPages", "OutOfStateSlots", "PageAllocator", "PagedLayerCache", "RequestCache",
            "StateLayerCache", "group_key"]

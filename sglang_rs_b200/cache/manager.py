@@ -23,7 +23,7 @@ from typing import Dict, Hashable, List, Optional, Sequence
 import numpy as np
 import torch
 
-from ..parts.base import CacheNeed, PagedKV, RequestState
+from ..parts.base import CacheNeed, JointNeed, PagedKV, RequestState, simple_needs
 
 GroupKey = Hashable        # ("kv", window) with window None for "all keys"
 
@@ -170,6 +170,16 @@ class StateLayerCache:
         return StateLayerCache(self.state, False)
 
 
+@dataclass
+class JointLayerCache:
+    """What a mixer with a :class:`JointNeed` is handed: the cache of each of its parts, in order (None: a part that
+    keeps nothing)."""
+    parts: tuple
+
+    def read_only(self) -> "JointLayerCache":
+        return JointLayerCache(tuple(part.read_only() if part is not None else None for part in self.parts))
+
+
 class RequestCache:
     """A live request's hold on the cache.  Length, state slot and block tables live in the C++
     books; ``tables`` copies them out (logical page -> page id, -1 = given back)."""
@@ -223,7 +233,7 @@ class CacheManager:
         default_pages = max(1, -(-int(max_tokens) // self.page_size))
         self.windows: Dict[GroupKey, Optional[int]] = {}
         counts: Dict[GroupKey, int] = {}
-        for need in self.needs:
+        for need in simple_needs(self.needs):
             if isinstance(need, PagedKV):
                 key = group_key(need)
                 if key not in counts:
@@ -242,30 +252,36 @@ class CacheManager:
         self._needed = np.zeros(max(len(counts), 1), dtype=np.int32)
         self._short_group, self._shortfall = ctypes.c_int(0), ctypes.c_int(0)
         self.state_pool = _StateSlots(self._core, self.max_requests)
-        self.has_state = any(isinstance(need, RequestState) for need in self.needs)
-        self.layer_caches: List[object] = []
-        for need in self.needs:
-            if isinstance(need, PagedKV):
-                key = group_key(need)
-                pools = (None, None)
-                if device is not None:
-                    # one page more than the allocator owns: rows that pad a captured step write there
-                    shape = (self.allocators[key].num_pages + 1, need.num_kv_heads, self.page_size, need.head_dim)
-                    pools = (torch.zeros(shape, dtype=dtype, device=device),
-                             torch.zeros((*shape[:3], need.value_width), dtype=dtype, device=device) if need.values else None)
-                self.layer_caches.append(PagedLayerCache(key, *pools))
-            elif isinstance(need, RequestState):
-                state = None
-                if device is not None:
-                    # one slot more than requests can hold: rows that pad a captured step use it
-                    state = torch.zeros((self.max_requests + 1, *need.shape), dtype=need.dtype or dtype, device=device)
-                self.layer_caches.append(StateLayerCache(state))
-            elif need is None:
-                self.layer_caches.append(None)
-            else:
-                raise TypeError(f"unknown cache need {need!r}")
+        self.has_state = any(isinstance(need, RequestState) for need in simple_needs(self.needs))
+        #: the state caches of all calls, also those inside joint caches
+        self._states: List[StateLayerCache] = []
+        self.layer_caches: List[object] = [self._make_cache(need) for need in self.needs]
         self.live: Dict[Hashable, RequestCache] = {}
         self.prefix_tree = None
+
+    def _make_cache(self, need: CacheNeed):
+        """The storage of one need (books only without a device)."""
+        if need is None:
+            return None
+        if isinstance(need, JointNeed):
+            return JointLayerCache(tuple(self._make_cache(part) for part in need.parts))
+        if isinstance(need, PagedKV):
+            key = group_key(need)
+            pools = (None, None)
+            if self.device is not None:
+                # one page more than the allocator owns: rows that pad a captured step write there
+                shape = (self.allocators[key].num_pages + 1, need.num_kv_heads, self.page_size, need.head_dim)
+                pools = (torch.zeros(shape, dtype=self.dtype, device=self.device),
+                         torch.zeros((*shape[:3], need.value_width), dtype=self.dtype, device=self.device) if need.values else None)
+            return PagedLayerCache(key, *pools)
+        if isinstance(need, RequestState):
+            state = None
+            if self.device is not None:
+                # one slot more than requests can hold: rows that pad a captured step use it
+                state = torch.zeros((self.max_requests + 1, *need.shape), dtype=need.dtype or self.dtype, device=self.device)
+            self._states.append(StateLayerCache(state))
+            return self._states[-1]
+        raise TypeError(f"unknown cache need {need!r}")
 
     # ------------------------------------------------------------------ prefix reuse
     def prefix_reuse_possible(self) -> bool:
@@ -299,10 +315,9 @@ class CacheManager:
         if index < 0:
             raise OutOfStateSlots(f"{self.max_requests} requests are live already")
         handle = RequestCache(request_id, self, index)
-        if self.has_state and self.device is not None:
-            for cache in self.layer_caches:
-                if isinstance(cache, StateLayerCache):
-                    cache.state[handle.state_slot].zero_()       # a new request starts from zero state
+        if self.device is not None:
+            for cache in self._states:
+                cache.state[handle.state_slot].zero_()           # a new request starts from zero state
         self.live[request_id] = handle
         return handle
 
@@ -315,10 +330,9 @@ class CacheManager:
         # A request that found no free page is opened and closed again inside one scheduling call; by the time its
         # events are read the books have no slot for it (a negative number), and no state may be touched: a negative
         # index would name another request's slot.
-        if self.has_state and self.device is not None and handle.state_slot >= 0:
-            for cache in self.layer_caches:
-                if isinstance(cache, StateLayerCache):
-                    cache.state[handle.state_slot].zero_()       # a new request starts from zero state
+        if self.device is not None and handle.state_slot >= 0:
+            for cache in self._states:
+                cache.state[handle.state_slot].zero_()           # a new request starts from zero state
         self.live[request_id] = handle
         return handle
 

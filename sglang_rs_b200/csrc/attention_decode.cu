@@ -315,9 +315,9 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
         acc *= shrink;
         l = l * shrink + exp2f(sink - m_all);
       }
-      float result = l > 0.f ? acc / l : 0.f;
+      float result = l > 0.f ? acc / l * p.out_scale : 0.f;
       if (p.gates) result *= p.gates[(size_t)row * p.n_q + q_head];
-      out[((size_t)row * p.n_q + q_head) * D + e] = __float2bfloat16_rn(result);
+      out[(size_t)row * p.out_pitch + (size_t)q_head * D + e] = __float2bfloat16_rn(result);
     }
     srb_cluster_sync();                                    // nobody leaves while its memory may still be read
     srb_mark(SRB_MARK_DECODE_ATTENTION, 2);
@@ -361,7 +361,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
     }
     float l = srb_warp_sum(lw);
     if (p.sinks) l += exp2f(sink - m);
-    if (lane == 0) weights[head * (count + 1) + count] = (p.gates ? p.gates[(size_t)row * p.n_q + q_head] : 1.0f) / l;
+    if (lane == 0) weights[head * (count + 1) + count] = (p.gates ? p.gates[(size_t)row * p.n_q + q_head] * p.out_scale : p.out_scale) / l;
   }
   __syncthreads();
   // four (head, element) pairs per thread and eight splits at a time: 32 loads in flight, added in split order
@@ -394,7 +394,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
       const int i = i0 + q * (int)blockDim.x;
       if (i < total) {
         const int head = i / D, e = i % D;
-        out[((size_t)row * p.n_q + (size_t)kv_head * groups + head) * D + e] = __float2bfloat16_rn(acc[q] * w[q][count]);
+        out[(size_t)row * p.out_pitch + ((size_t)kv_head * groups + head) * D + e] = __float2bfloat16_rn(acc[q] * w[q][count]);
       }
     }
   }
@@ -435,13 +435,14 @@ extern "C" int srb_decode_attention_supports(int n_q, int n_kv, int head_dim, in
 // rows * n_kv ints that are zero before the call and zero again after it.
 // `chunk` > 0: a row sees only the keys of its own chunk of positions, counted from position 0.
 // `sinks` (float [n_q], or null): exp(sink_h) joins the softmax's denominator of head h, once per row; `gates` (float
-// [rows, n_q], or null): a factor on the result of every (row, query head).
+// [rows, n_q], or null): a factor on the result of every (row, query head); `out_scale`: a factor on every result;
+// `out_pitch`: elements between rows of the output (0: dense).
 extern "C" int srb_decode_attention_gated(const void* q, const void* k_pool, const void* v_pool, void* out,
                                           float* part_acc, float* part_ml, int* counters, const int* positions,
                                           const int* row_request, const int* block_table, int table_stride, int rows,
                                           int n_q, int n_kv, int head_dim, int page_size, int num_pages, int window,
                                           int chunk, int num_splits, float scale, int* error_word, const float* sinks,
-                                          const float* gates, void* stream) {
+                                          const float* gates, long long out_pitch, float out_scale, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (chunk < 0) SRB_FAIL("decode_attention: the chunk size must be non-negative");
   if (!srb_decode_attention_supports(n_q, n_kv, head_dim, SRB_DTYPE_BF16))
@@ -457,6 +458,8 @@ extern "C" int srb_decode_attention_gated(const void* q, const void* k_pool, con
   p.table_stride = table_stride; p.n_q = n_q; p.n_kv = n_kv; p.head_dim = head_dim;
   p.page_size = page_size; p.num_pages = num_pages; p.window = window; p.chunk = chunk; p.split_size = 0;
   p.max_splits = num_splits; p.scale = scale; p.error_word = error_word; p.sinks = sinks; p.gates = gates;
+  p.value_dim = head_dim; p.out_pitch = out_pitch ? out_pitch : (long long)n_q * head_dim; p.out_scale = out_scale;
+  if (p.out_pitch < (long long)n_q * head_dim) SRB_FAIL("decode_attention: rows of the output overlap");
   dp.scale_log2 = scale * 1.4426950408889634f;
   cudaStream_t s = (cudaStream_t)stream;
   if (head_dim == 64) return launch_decode<64>(q, k_pool, v_pool, out, part_acc, part_ml, counters, dp, rows, s);
@@ -470,7 +473,7 @@ extern "C" int srb_decode_attention_masked(const void* q, const void* k_pool, co
                                            int chunk, int num_splits, float scale, int* error_word, void* stream) {
   return srb_decode_attention_gated(q, k_pool, v_pool, out, part_acc, part_ml, counters, positions, row_request, block_table,
                                     table_stride, rows, n_q, n_kv, head_dim, page_size, num_pages, window, chunk, num_splits,
-                                    scale, error_word, nullptr, nullptr, stream);
+                                    scale, error_word, nullptr, nullptr, 0, 1.0f, stream);
 }
 
 extern "C" int srb_decode_attention(const void* q, const void* k_pool, const void* v_pool, void* out,

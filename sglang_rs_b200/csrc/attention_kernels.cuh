@@ -17,6 +17,8 @@
 //    added exactly one time per row, also when the row's keys are split over several blocks (the merge adds it);
 //  * a gate: `gates` holds one float per (row, query head) that multiplies the head's result (a mixer's output gate,
 //    already passed through its sigmoid), applied where the result is normalised and written;
+//  * a place inside wider rows: `out_pitch` elements lie between rows of the output, and `out_scale` multiplies every
+//    result (a mixer beside another one writes its columns of the row that one output product reads);
 //  * values of another width than the keys: the output and the value rows are `value_dim` wide.  With
 //    `shared_values` the value of a key is the first `value_dim` entries of its key row (a cache that
 //    keeps one latent row per token serves as key and as value), and v_pool is not read.
@@ -53,6 +55,8 @@ struct AttnParams {
   int head_chunks;           // blocks per (row, kv head, split) along the query heads
   int heads_per_block;
   const float* gates = nullptr;   // [rows, n_q] or null: a factor on the result of every (row, query head)
+  float out_scale = 1.0f;         // a factor on every result, taken in 32-bit before it is rounded
+  long long out_pitch = 0;        // elements between rows of the output (a head's results are always dense); 0: n_q * value_dim
 };
 
 // The first key that a row at `pos` may see: the start of its window, or of its chunk of positions, whichever is later.
@@ -186,11 +190,11 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
 #pragma unroll
       for (int j = 0; j < DIM_PER_LANE; ++j) acc[j] *= correction;
     }
-    const float inv = p.gates ? p.gates[(size_t)row * p.n_q + q_head] / l : 1.0f / l;
+    const float inv = (p.gates ? p.gates[(size_t)row * p.n_q + q_head] * p.out_scale : p.out_scale) / l;
 #pragma unroll
     for (int j = 0; j < DIM_PER_LANE; ++j) {
       const int e = lane + 32 * j;
-      if (e < vd) out[((size_t)row * p.n_q + q_head) * vd + e] = srb_from_float<T>(acc[j] * inv);
+      if (e < vd) out[(size_t)row * p.out_pitch + (size_t)q_head * vd + e] = srb_from_float<T>(acc[j] * inv);
     }
   } else {
     const size_t slot = ((size_t)row * p.n_q + q_head) * p.max_splits + split;
@@ -224,12 +228,12 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_acc, con
   for (int s = 0; s < count; ++s) m = fmaxf(m, part_ml[(first + s) * 2]);
   float l = p.sinks ? expf(p.sinks[q_head] - m) : 0.f;   // the sink counts once, whatever the number of splits
   for (int s = 0; s < count; ++s) l += part_ml[(first + s) * 2 + 1] * expf(part_ml[(first + s) * 2] - m);
-  const float inv = p.gates ? p.gates[(size_t)row * p.n_q + q_head] / l : 1.0f / l;
+  const float inv = (p.gates ? p.gates[(size_t)row * p.n_q + q_head] * p.out_scale : p.out_scale) / l;
   for (int e = threadIdx.x; e < p.value_dim; e += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < count; ++s)
       acc += part_acc[(first + s) * p.value_dim + e] * expf(part_ml[(first + s) * 2] - m);
-    out[((size_t)row * p.n_q + q_head) * p.value_dim + e] = srb_from_float<T>(acc * inv);
+    out[(size_t)row * p.out_pitch + (size_t)q_head * p.value_dim + e] = srb_from_float<T>(acc * inv);
   }
 }
 
@@ -266,7 +270,7 @@ static int paged_attention_dispatch_masked(const void* q, const void* k_pool, co
                                            int n_q, int n_kv, int head_dim, int page_size, int num_pages, int window,
                                            int chunk, int split_size, int max_splits, float scale, int* error_word,
                                            int dtype, const float* sinks, int value_dim, void* stream,
-                                           const float* gates = nullptr) {
+                                           const float* gates = nullptr, long long out_pitch = 0, float out_scale = 1.0f) {
   if (rows <= 0) return SRB_OK;
   if (chunk < 0) SRB_FAIL("paged_attention: the chunk size must be non-negative");
   if (n_q <= 0 || n_kv <= 0 || n_q % n_kv != 0)
@@ -291,6 +295,8 @@ static int paged_attention_dispatch_masked(const void* q, const void* k_pool, co
   p.page_size = page_size; p.num_pages = num_pages; p.window = window; p.chunk = chunk; p.split_size = split_size;
   p.max_splits = split_size == 0 ? 1 : max_splits; p.scale = scale; p.error_word = error_word;
   p.sinks = sinks; p.value_dim = value_dim; p.shared_values = v_pool == nullptr; p.gates = gates;
+  p.out_pitch = out_pitch ? out_pitch : (long long)n_q * value_dim; p.out_scale = out_scale;
+  if (p.out_pitch < (long long)n_q * value_dim) SRB_FAIL("paged_attention: rows of the output overlap");
   const int groups = n_q / n_kv;
   p.head_chunks = (groups + 31) / 32;
   p.heads_per_block = (groups + p.head_chunks - 1) / p.head_chunks;

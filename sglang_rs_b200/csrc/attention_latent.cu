@@ -350,6 +350,7 @@ extern "C" int srb_latent_attention_masked(const void* q, const void* pool, void
   else status = launch_latent_attention<16, 4>(p, grid, smem, s);
   if (status != SRB_OK || tiles) return status;
   AttnParams m = {};
+  m.out_pitch = (long long)n_q * vd;
   m.positions = positions; m.n_q = n_q; m.n_kv = 1; m.head_dim = d; m.window = window; m.split_size = split_size;
   m.max_splits = max_splits; m.error_word = error_word; m.sinks = sinks; m.value_dim = vd;
   attention_combine_kernel<__nv_bfloat16><<<dim3(rows, n_q), 64, 0, s>>>(part_acc, part_ml, (__nv_bfloat16*)out, m);

@@ -45,6 +45,8 @@ struct TcArgs {
   int* error_word;
   const float* sinks;      // [n_q] or null: exp(sink_h) joins the softmax's denominator of head h, once per row
   const float* gates;      // [rows, n_q] or null: a factor on the result of every (row, query head)
+  long long out_pitch;     // elements between rows of the output
+  float out_scale;         // a factor on every result
 };
 
 // M = 128, N = n, A and B bfloat16, D float; b_mn_major: B is [K rows][N contiguous] (V), else K-major
@@ -392,9 +394,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         shrink = ex2(m_run - m_all);
         l_all = l_run * shrink + ex2(sink - m_all);
       }
-      float inv = row_live && l_all > 0.f ? shrink / l_all : 0.f;
+      float inv = row_live && l_all > 0.f ? shrink / l_all * args.out_scale : 0.f;
       if (args.gates && row_live) inv *= args.gates[(size_t)(row_begin + r) * args.n_q + head];
-      __nv_bfloat16* dst = args.out + ((size_t)(row_begin + r) * args.n_q + head) * D;
+      __nv_bfloat16* dst = args.out + (size_t)(row_begin + r) * args.out_pitch + (size_t)head * D;
 #pragma unroll 2
       for (int c = 0; c < D; c += 32) {
         float ov[32];
@@ -489,12 +491,14 @@ static int launch_tc(const CUtensorMap& map_q, const CUtensorMap& map_k, const C
 // tiles: [num_tiles, 4] ints with at most 128 rows each.
 // `chunk` > 0: a row sees only the keys of its own chunk of positions, counted from position 0.
 // `sinks` (float [n_q], or null): exp(sink_h) joins the softmax's denominator of head h; `gates` (float [rows, n_q], or
-// null): a factor on the result of every (row, query head).
+// null): a factor on the result of every (row, query head); `out_scale`: a factor on every result; `out_pitch`: elements
+// between rows of the output (a multiple of 8; 0: dense).
 extern "C" int srb_prefill_attention_tc_gated(const void* q, const void* k_pool, const void* v_pool, void* out,
                                               const int* tiles, int num_tiles, int rows, const int* block_table,
                                               int table_stride, int n_q, int n_kv, int head_dim, int page_size,
                                               int num_pages, int window, int chunk, float scale, int* error_word,
-                                              const float* sinks, const float* gates, void* stream) {
+                                              const float* sinks, const float* gates, long long out_pitch,
+                                              float out_scale, void* stream) {
   if (num_tiles <= 0) return SRB_OK;
   if (chunk < 0) SRB_FAIL("prefill_attention_tc: the chunk size must be non-negative");
   if (!srb_prefill_tc_supports(n_q, n_kv, head_dim, page_size, SRB_DTYPE_BF16))
@@ -504,12 +508,15 @@ extern "C" int srb_prefill_attention_tc_gated(const void* q, const void* k_pool,
     SRB_FAIL("prefill_attention_tc: page count, table stride and rows must be positive");
   if ((((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15) != 0)
     SRB_FAIL("prefill_attention_tc: operands must be 16-byte aligned");
+  if (out_pitch == 0) out_pitch = (long long)n_q * head_dim;
+  if (out_pitch < (long long)n_q * head_dim || out_pitch % 8)
+    SRB_FAIL("prefill_attention_tc: rows of the output overlap or start off 16-byte borders");
   EncodeTiledFn encode = encode_tiled();
   if (!encode) SRB_FAIL("prefill_attention_tc: the driver does not offer cuTensorMapEncodeTiled");
   CUtensorMap map_q, map_k, map_v, map_out;
   for (int pass = 0; pass < 2; ++pass) {                     // q, and the output of the same shape
     const cuuint64_t dims[3] = {(cuuint64_t)head_dim, (cuuint64_t)n_q, (cuuint64_t)rows};
-    const cuuint64_t strides[2] = {(cuuint64_t)head_dim * 2, (cuuint64_t)n_q * head_dim * 2};
+    const cuuint64_t strides[2] = {(cuuint64_t)head_dim * 2, pass == 0 ? (cuuint64_t)n_q * head_dim * 2 : (cuuint64_t)out_pitch * 2};
     const cuuint32_t box[3] = {64, 1, TC_ROWS};
     const cuuint32_t elem[3] = {1, 1, 1};
     const CUresult status = encode(pass == 0 ? &map_q : &map_out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3,
@@ -535,7 +542,7 @@ extern "C" int srb_prefill_attention_tc_gated(const void* q, const void* k_pool,
   args.tiles = tiles; args.block_table = block_table; args.out = (__nv_bfloat16*)out; args.table_stride = table_stride;
   args.n_q = n_q; args.n_kv = n_kv; args.page_size = page_size; args.pool_rows = (int)pool_rows; args.window = window; args.chunk = chunk;
   args.scale_log2 = scale * 1.4426950408889634f; args.error_word = error_word;
-  args.sinks = sinks; args.gates = gates;
+  args.sinks = sinks; args.gates = gates; args.out_pitch = out_pitch; args.out_scale = out_scale;
   cudaStream_t s = (cudaStream_t)stream;
   // two query heads per block when the heads of a kv head pair up
   const bool pairs = (n_q / n_kv) % 2 == 0;
@@ -553,7 +560,7 @@ extern "C" int srb_prefill_attention_tc_masked(const void* q, const void* k_pool
                                                void* stream) {
   return srb_prefill_attention_tc_gated(q, k_pool, v_pool, out, tiles, num_tiles, rows, block_table, table_stride, n_q, n_kv,
                                         head_dim, page_size, num_pages, window, chunk, scale, error_word, nullptr, nullptr,
-                                        stream);
+                                        0, 1.0f, stream);
 }
 
 extern "C" int srb_prefill_attention_tc(const void* q, const void* k_pool, const void* v_pool, void* out,

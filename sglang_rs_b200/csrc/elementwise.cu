@@ -160,20 +160,21 @@ add_rmsnorm_vec_kernel(float* __restrict__ residual, const T* __restrict__ delta
 
 // out[row, j] = act(gate_up[row, j]) * gate_up[row, inner + j], act being SRB_ACT_* `activation`
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int rows, int inner, int activation) {
+__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int rows, int inner, int activation,
+                                float act_param) {
   const size_t total = (size_t)rows * inner;
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
        idx += (size_t)gridDim.x * blockDim.x) {
     const size_t row = idx / inner, col = idx % inner;
     const float g = srb_to_float(gate_up[row * 2 * inner + col]);
     const float u = srb_to_float(gate_up[row * 2 * inner + inner + col]);
-    out[idx] = srb_from_float<T>(srb_gated<true>(activation, g, u));
+    out[idx] = srb_from_float<T>(srb_gated<true>(activation, g, u, act_param));
   }
 }
 
 // The same with eight bfloat16 values (16 bytes) per thread and access; `inner` a multiple of 8.
 __global__ void silu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gate_up, __nv_bfloat16* __restrict__ out,
-                                       int rows, int inner, int activation) {
+                                       int rows, int inner, int activation, float act_param) {
   const int per_row = inner / 8;
   const size_t total = (size_t)rows * per_row;
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
@@ -189,7 +190,7 @@ __global__ void silu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gate_up
     for (int j = 0; j < 4; ++j) {
       const float2 g = __bfloat1622float2(g2[j]), u = __bfloat1622float2(u2[j]);
       // the result is rounded to bfloat16 (8 bits): the hardware's exponential and division are exact enough
-      o2[j] = __floats2bfloat162_rn(srb_gated<false>(activation, g.x, u.x), srb_gated<false>(activation, g.y, u.y));
+      o2[j] = __floats2bfloat162_rn(srb_gated<false>(activation, g.x, u.x, act_param), srb_gated<false>(activation, g.y, u.y, act_param));
     }
     *reinterpret_cast<uint4*>(out + row * inner + col) = o4;
   }
@@ -562,26 +563,33 @@ extern "C" int srb_scale_values(float* values, long long total, float factor, vo
   return SRB_OK;
 }
 
-extern "C" int srb_gated_mul(const void* gate_up, void* out, int rows, int inner, int activation, int dtype,
-                             void* stream) {
+// `act_param`: the parameter of an activation that has one
+extern "C" int srb_gated_mul_param(const void* gate_up, void* out, int rows, int inner, int activation, float act_param,
+                                   int dtype, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (inner <= 0) SRB_FAIL("gated_mul: inner width %d must be positive", inner);
   if (activation < 0 || activation >= SRB_ACT_COUNT) SRB_FAIL("gated_mul: unknown activation %d", activation);
   cudaStream_t s = (cudaStream_t)stream;
   const int grid = elementwise_grid((size_t)rows * inner, 256);
   if (dtype == SRB_DTYPE_F32)
-    silu_mul_kernel<float><<<grid, 256, 0, s>>>((const float*)gate_up, (float*)out, rows, inner, activation);
+    silu_mul_kernel<float><<<grid, 256, 0, s>>>((const float*)gate_up, (float*)out, rows, inner, activation, act_param);
   else if (dtype == SRB_DTYPE_BF16 && inner % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0) {
     size_t blocks = ((size_t)rows * (inner / 8) + 255) / 256;
     if (blocks > srb_sm_count() * 64) blocks = srb_sm_count() * 64;
-    silu_mul_bf16x8_kernel<<<(int)blocks, 256, 0, s>>>((const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, rows, inner, activation);
+    silu_mul_bf16x8_kernel<<<(int)blocks, 256, 0, s>>>((const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, rows, inner, activation, act_param);
   } else if (dtype == SRB_DTYPE_BF16)
     silu_mul_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>((const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, rows,
-                                                        inner, activation);
+                                                        inner, activation, act_param);
   else
     SRB_FAIL("gated_mul: unknown dtype %d", dtype);
   SRB_LAUNCH_CHECK("gated_mul");
   return SRB_OK;
+}
+
+extern "C" int srb_gated_mul(const void* gate_up, void* out, int rows, int inner, int activation, int dtype,
+                             void* stream) {
+  if (activation == SRB_ACT_SWIGLU_CLAMP) SRB_FAIL("gated_mul: an activation with a parameter comes with its parameter");
+  return srb_gated_mul_param(gate_up, out, rows, inner, activation, 0.f, dtype, stream);
 }
 
 extern "C" int srb_add_bias(void* values, const float* bias, int rows, int width, int dtype, void* stream) {

@@ -378,9 +378,10 @@ extern "C" int srb_gemm_bf16_block_tokens(int tokens, int mode) {
 // mode 5: out bf16 [tokens, ldo] = activation(x w^T).
 // mode 4: out float [tokens, ldo] += x w^T, K cut into `splits` (at most 8) blocks that form a cluster and add
 //         their sums in block order.
-extern "C" int srb_gemm_bf16(const void* x, const void* w, void* out, int tokens, int features, int k, int ldx,
-                             int ldw, int ldo, int rows_of_w, int up_row_offset, int mode, int splits,
-                             int activation, int* error_word, void* stream) {
+// `act_param`: the parameter of an activation that has one (modes 2 and 5).
+extern "C" int srb_gemm_bf16_param(const void* x, const void* w, void* out, int tokens, int features, int k, int ldx,
+                                   int ldw, int ldo, int rows_of_w, int up_row_offset, int mode, int splits,
+                                   int activation, float act_param, int* error_word, void* stream) {
   if (tokens <= 0 || features <= 0) return SRB_OK;
   if (k <= 0 || k % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0)
     SRB_FAIL("gemm_bf16: inner size %d and the row pitches %d, %d must be positive multiples of 8 (16-byte rows "
@@ -389,8 +390,6 @@ extern "C" int srb_gemm_bf16(const void* x, const void* w, void* out, int tokens
   if (mode < 0 || mode > 5) SRB_FAIL("gemm_bf16: unknown mode %d", mode);
   if ((mode == EPI_SILU || mode == EPI_ACT) && (activation < 0 || activation >= SRB_ACT_COUNT))
     SRB_FAIL("gemm_bf16: unknown activation %d", activation);
-  if ((mode == EPI_SILU || mode == EPI_ACT) && activation == SRB_ACT_SWIGLU_CLAMP)
-    SRB_FAIL("gemm_bf16: an activation with a parameter is taken by the grouped mode only");
   if (ldo < features) SRB_FAIL("gemm_bf16: output pitch %d is smaller than %d features", ldo, features);
   if (mode == EPI_SILU && up_row_offset + features > rows_of_w)
     SRB_FAIL("gemm_bf16: the up rows %d..%d lie outside the %d rows of w", up_row_offset, up_row_offset + features,
@@ -411,7 +410,7 @@ extern "C" int srb_gemm_bf16(const void* x, const void* w, void* out, int tokens
   GemmArgs args;
   args.out = out; args.tokens = tokens; args.features = features; args.k = k; args.ldo = ldo;
   args.up_row_offset = up_row_offset; args.activation = activation; args.error_word = error_word;
-  args.act_param = 0.f;
+  args.act_param = act_param;
   args.plan = nullptr; args.experts = 0; args.expert_rows = 0;
   args.k_blocks_per_split = (total_k_blocks + splits - 1) / splits;
   const int used_splits = (total_k_blocks + args.k_blocks_per_split - 1) / args.k_blocks_per_split;
@@ -425,6 +424,15 @@ extern "C" int srb_gemm_bf16(const void* x, const void* w, void* out, int tokens
     case EPI_ACT: return dispatch_tokens<EPI_ACT>(block_t, map_w, map_x, args, 1, s);
     default: return dispatch_tokens<EPI_PARTIAL>(block_t, map_w, map_x, args, splits, s);
   }
+}
+
+extern "C" int srb_gemm_bf16(const void* x, const void* w, void* out, int tokens, int features, int k, int ldx,
+                             int ldw, int ldo, int rows_of_w, int up_row_offset, int mode, int splits,
+                             int activation, int* error_word, void* stream) {
+  if ((mode == EPI_SILU || mode == EPI_ACT) && activation == SRB_ACT_SWIGLU_CLAMP)
+    SRB_FAIL("gemm_bf16: an activation with a parameter comes with its parameter");
+  return srb_gemm_bf16_param(x, w, out, tokens, features, k, ldx, ldw, ldo, rows_of_w, up_row_offset, mode, splits, activation,
+                             0.f, error_word, stream);
 }
 
 

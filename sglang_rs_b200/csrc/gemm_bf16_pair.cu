@@ -41,6 +41,7 @@ SRB_DEFINE_LAST_ERROR()
 struct PairArgs {
   __nv_bfloat16* out;
   int tokens, features, k, ldo, up_row_offset;
+  float act_param;           // the activation's parameter, for those that have one
   int activation;            // which SRB_ACT_* the gated mode applies to the gate half, or the plain mode to its result (-1: none)
   int tiles_t, tiles_f, num_tiles;
   int* error_word;
@@ -228,7 +229,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
 #pragma unroll
               for (int j = 0; j < 32; ++j) {
                 const float g = acc[j], u = buffer[j * 64 + (quarter & 1) * 32 + lane];
-                staged[(c + j) * FEATURES_PER_CTA + row_in_cta] = __float2bfloat16_rn(srb_gated<false>(args.activation, g, u));
+                staged[(c + j) * FEATURES_PER_CTA + row_in_cta] = __float2bfloat16_rn(srb_gated<false>(args.activation, g, u, args.act_param));
               }
             }
           }
@@ -240,7 +241,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               staged[(c + j) * FEATURES_PER_CTA + row_in_cta] =
-                  __float2bfloat16_rn(args.activation >= 0 ? srb_gated<false>(args.activation, acc[j], 1.0f) : acc[j]);
+                  __float2bfloat16_rn(args.activation >= 0 ? srb_gated<false>(args.activation, acc[j], 1.0f, args.act_param) : acc[j]);
           }
         }
         if (half == PAIR_T / PAIR_OUT_T - 1) {
@@ -314,9 +315,10 @@ static int make_map(CUtensorMap* map, const void* base, long long rows, long lon
 // x [tokens, k] (row pitch ldx), w [rows_of_w, k] (row pitch ldw), out [tokens, ldo], all bfloat16; k and the
 // pitches multiples of 8.  mode 0: out = x w^T over `features` rows of w.  mode 5: out = activation(x w^T).  mode 2: w stacks gate rows
 // [0, features) and up rows [up_row_offset, up_row_offset + features); out = act(x gate^T) * (x up^T), act being SRB_ACT_* `activation` (activations.cuh).
-extern "C" int srb_gemm_bf16_pair(const void* x, const void* w, void* out, int tokens, int features, int k, int ldx,
-                                  int ldw, int ldo, int rows_of_w, int up_row_offset, int mode, int activation,
-                                  int* error_word, void* stream) {
+// `act_param`: the parameter of an activation that has one.
+extern "C" int srb_gemm_bf16_pair_param(const void* x, const void* w, void* out, int tokens, int features, int k, int ldx,
+                                        int ldw, int ldo, int rows_of_w, int up_row_offset, int mode, int activation,
+                                        float act_param, int* error_word, void* stream) {
   if (tokens <= 0 || features <= 0) return SRB_OK;
   if (k <= 0 || k % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0 || ldo % 8 != 0)
     SRB_FAIL("gemm_bf16_pair: inner size %d and the row pitches %d, %d, %d must be positive multiples of 8", k, ldx, ldw,
@@ -335,7 +337,7 @@ extern "C" int srb_gemm_bf16_pair(const void* x, const void* w, void* out, int t
   const int features_per_pair = mode == PAIR_EPI_SILU ? PAIR_F : 2 * PAIR_F;
   PairArgs args;
   args.out = (__nv_bfloat16*)out; args.tokens = tokens; args.features = features; args.k = k; args.ldo = ldo;
-  args.up_row_offset = up_row_offset; args.activation = activation; args.error_word = error_word;
+  args.up_row_offset = up_row_offset; args.activation = activation; args.act_param = act_param; args.error_word = error_word;
   args.tiles_t = (tokens + PAIR_T - 1) / PAIR_T;
   args.tiles_f = (features + features_per_pair - 1) / features_per_pair;
   args.num_tiles = args.tiles_t * args.tiles_f;
@@ -356,4 +358,13 @@ extern "C" int srb_gemm_bf16_pair(const void* x, const void* w, void* out, int t
                                        dim3(2, 1, 1), map_w, map_x, args));
   }
   return SRB_OK;
+}
+
+extern "C" int srb_gemm_bf16_pair(const void* x, const void* w, void* out, int tokens, int features, int k, int ldx,
+                                  int ldw, int ldo, int rows_of_w, int up_row_offset, int mode, int activation,
+                                  int* error_word, void* stream) {
+  if (mode != PAIR_EPI_BF16 && activation == SRB_ACT_SWIGLU_CLAMP)
+    SRB_FAIL("gemm_bf16_pair: an activation with a parameter comes with its parameter");
+  return srb_gemm_bf16_pair_param(x, w, out, tokens, features, k, ldx, ldw, ldo, rows_of_w, up_row_offset, mode, activation, 0.f,
+                                  error_word, stream);
 }

@@ -10,10 +10,7 @@
 // A request's slot of state holds, in 32-bit floats, the last taps - 1 inputs of the convolution
 // [taps - 1][channels] (oldest first) followed by S as [heads][P][N] (a column's N entries together).  Kernels:
 //
-//   srb_mamba_conv        the convolution + SiLU of every row of the step (32-bit result, or rounded to bfloat16 for the
-//                         chunk kernels), reading earlier rows of the
-//                         same request from the step and, before the step's first row, from the slot; then the slot's
-//                         inputs are replaced by the last taps - 1 of the sequence (a second launch: rows read the old ones)
+//   (short_conv.cu)       the convolution + SiLU of every row of the step, and the slot's inputs
 //   srb_mamba_scan        the recurrence, token by token: a block owns a head's N x PB slice of the state in registers
 //                         (PB columns, N cut over the lanes beside each column), stages 16 tokens' B, C, x, dt at a time in
 //                         shared memory and walks them; decoded tokens and prompt portions take the same arithmetic, so a
@@ -32,7 +29,6 @@ SRB_DEFINE_PDL_SWITCH()
 
 #define MAMBA_MAX_TAPS 16
 #define MAMBA_TOKENS 16        // tokens staged in shared memory at a time
-#define MAMBA_CONV_ROWS 8      // rows of the step that one thread of the convolution takes
 #define MAMBA_THREADS 256
 
 struct MambaShape {
@@ -45,144 +41,6 @@ struct MambaShape {
 
 __device__ __forceinline__ float mamba_silu(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float mamba_softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
-
-// SiLU of the convolution's sum as the result's type: a bfloat16 result keeps 8 bits of mantissa, so the quick exponential
-// and quotient (about 22 bits) round to the same number but for ties
-template <typename O> __device__ __forceinline__ O mamba_conv_result(float acc);
-template <> __device__ __forceinline__ float mamba_conv_result<float>(float acc) { return mamba_silu(acc); }
-template <> __device__ __forceinline__ __nv_bfloat16 mamba_conv_result<__nv_bfloat16>(float acc) {
-  return __float2bfloat16_rn(__fdividef(acc, 1.0f + __expf(-acc)));
-}
-
-// grid (channel blocks, ceil(rows / ROWS)), so that blocks that run together read neighbouring pieces of the same rows:
-// a thread takes one channel of ROWS consecutive rows (MAMBA_CONV_ROWS in steps
-// of many rows, so that the filter is read once and the rows' loads are in flight together; 1 in steps of few rows).
-// TAPS: the filter's length, or 0 for any.
-template <typename T, typename O, int TAPS, int ROWS>
-__global__ void mamba_conv_kernel(const T* __restrict__ proj, const float* __restrict__ weight, const float* __restrict__ bias,
-                                  const int* __restrict__ positions, const int* __restrict__ row_request,
-                                  const int* __restrict__ cu_rows, const int* __restrict__ state_slots,
-                                  const float* __restrict__ state, O* __restrict__ out, int rows, MambaShape s) {
-  srb_launch_dependents();
-  srb_grid_dependency_wait();
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= s.channels) return;
-  const int taps = TAPS > 0 ? TAPS : s.taps;
-  constexpr int HELD = TAPS > 0 ? TAPS : 1;
-  float w[HELD];
-  if (TAPS > 0) {
-#pragma unroll
-    for (int j = 0; j < HELD; ++j) w[j] = weight[(size_t)c * TAPS + j];
-  }
-  const float b = bias[c];
-  const int row0 = blockIdx.y * ROWS;
-  // what the rows need to know, all loads in flight together: position, rows of the request before it, the slot
-  int pos[ROWS], ahead[ROWS], slot[ROWS];
-#pragma unroll
-  for (int r = 0; r < ROWS; ++r) {
-    const bool live = row0 + r < rows;
-    pos[r] = live ? positions[row0 + r] : -1;
-    ahead[r] = live ? row_request[row0 + r] : 0;
-  }
-#pragma unroll
-  for (int r = 0; r < ROWS; ++r) {
-    const int request = ahead[r];
-    ahead[r] = row0 + r - cu_rows[request];
-    slot[r] = state_slots[request];
-  }
-  if constexpr (TAPS > 0) {
-    // the inputs of rows row0 - (TAPS - 1) .. row0 + ROWS - 1 of the step, whichever request they belong to
-    float u[ROWS + HELD - 1];
-#pragma unroll
-    for (int k = 0; k < ROWS + HELD - 1; ++k) {
-      const int row = row0 + k - (HELD - 1);
-      u[k] = (row >= 0 && row < rows) ? srb_to_float(proj[(size_t)row * s.proj_pitch + s.inner + c]) : 0.f;
-    }
-    // rows in the middle of a request's rows of the step: every input is one of the step's
-    bool inside = row0 + ROWS <= rows;
-#pragma unroll
-    for (int r = 0; r < ROWS; ++r) inside = inside && pos[r] >= HELD - 1 && ahead[r] >= HELD - 1;
-    if (inside) {
-#pragma unroll
-      for (int r = 0; r < ROWS; ++r) {
-        float acc = b;
-#pragma unroll
-        for (int j = 0; j < HELD; ++j) acc = fmaf(w[j], u[r + j], acc);
-        out[(size_t)(row0 + r) * s.channels + c] = mamba_conv_result<O>(acc);
-      }
-      return;
-    }
-#pragma unroll
-    for (int r = 0; r < ROWS; ++r) {
-      if (row0 + r >= rows) break;
-      O* dst = out + (size_t)(row0 + r) * s.channels + c;
-      if (pos[r] < 0) { *dst = srb_from_float<O>(0.f); continue; }
-      const float* kept = state + (size_t)slot[r] * s.slot_floats;
-      float acc = b;
-#pragma unroll
-      for (int j = 0; j < HELD; ++j) {
-        const int back = HELD - 1 - j;
-        if (pos[r] - back < 0) continue;                   // zeros before the start of the sequence
-        const float v = back <= ahead[r] ? u[r + j] : kept[(size_t)(HELD - 1 - (back - ahead[r])) * s.channels + c];
-        acc = fmaf(w[j], v, acc);
-      }
-      *dst = mamba_conv_result<O>(acc);
-    }
-  } else {
-#pragma unroll
-  for (int r = 0; r < ROWS; ++r) {
-    const int row = row0 + r;
-    if (row >= rows) break;
-    O* dst = out + (size_t)row * s.channels + c;
-    if (pos[r] < 0) { *dst = srb_from_float<O>(0.f); continue; }
-    const float* kept = state + (size_t)slot[r] * s.slot_floats;
-    float acc = b;
-    for (int j = 0; j < taps; ++j) {
-      const int back = taps - 1 - j;
-      if (pos[r] - back < 0) continue;                     // zeros before the start of the sequence
-      float v;
-      if (back <= ahead[r])
-        v = srb_to_float(proj[(size_t)(row - back) * s.proj_pitch + s.inner + c]);
-      else
-        v = kept[(size_t)(taps - 1 - (back - ahead[r])) * s.channels + c];
-      acc = fmaf(weight[(size_t)c * taps + j], v, acc);
-    }
-    *dst = mamba_conv_result<O>(acc);
-  }
-  }
-}
-
-// One thread per (request, channel): the slot's inputs become the last taps - 1 of the sequence after this step.
-template <typename T>
-__global__ void mamba_conv_keep_kernel(const T* __restrict__ proj, const int* __restrict__ positions,
-                                       const int* __restrict__ cu_rows, const int* __restrict__ state_slots,
-                                       float* __restrict__ state, MambaShape s) {
-  srb_launch_dependents();
-  srb_grid_dependency_wait();
-  const int request = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= s.channels) return;
-  const int first = cu_rows[request], count = cu_rows[request + 1] - first;
-  if (count <= 0) return;
-  const int start = positions[first];
-  if (start < 0) return;
-  float* kept = state + (size_t)state_slots[request] * s.slot_floats;
-  const int keep = s.taps - 1;
-  float fresh[MAMBA_MAX_TAPS];
-#pragma unroll
-  for (int k = 0; k < MAMBA_MAX_TAPS; ++k) {
-    if (k >= keep) break;
-    const int at = start + count - keep + k;           // position in the sequence of the k-th kept input
-    float v = 0.f;
-    if (at >= start) v = srb_to_float(proj[(size_t)(first + at - start) * s.proj_pitch + s.inner + c]);
-    else if (at >= 0) v = kept[(size_t)(at - start + keep) * s.channels + c];
-    fresh[k] = v;
-  }
-#pragma unroll
-  for (int k = 0; k < MAMBA_MAX_TAPS; ++k) {
-    if (k >= keep) break;
-    kept[(size_t)k * s.channels + c] = fresh[k];
-  }
-}
 
 // grid (heads * column blocks, requests); NS lanes share a column of the state, each with NR of its N entries
 template <typename T, int NS, int NR>
@@ -345,56 +203,6 @@ extern "C" long long srb_mamba_slot_floats(int heads, int vdim, int nstate, int 
   return (long long)(taps - 1) * (heads * vdim + 2 * groups * nstate) + (long long)heads * nstate * vdim;
 }
 
-template <typename T, typename O>
-static int launch_mamba_conv(const void* proj, const float* weight, const float* bias, const int* positions,
-                             const int* row_request, const int* cu_rows, const int* state_slots, float* state, void* out,
-                             int rows, int requests, int write_state, const MambaShape& s, cudaStream_t st) {
-  const int block = 128;
-  const bool many = rows >= 64 * MAMBA_CONV_ROWS;
-  const int per = many ? MAMBA_CONV_ROWS : 1;
-  const dim3 grid((s.channels + block - 1) / block, (rows + per - 1) / per);
-  if (grid.y > 65535) SRB_FAIL("mamba_conv: %d rows exceed one launch", rows);
-  const dim3 keep_grid((s.channels + block - 1) / block, requests);
-#define MAMBA_CONV_LAUNCH(TAPS, ROWS)                                                                                        \
-  SRB_CUDA_CALL(srb_launch(mamba_conv_kernel<T, O, TAPS, ROWS>, grid, dim3(block), 0, st, (const T*)proj, weight, bias,     \
-                           positions, row_request, cu_rows, state_slots, (const float*)state, (O*)out, rows, s))
-  if (s.taps == 4 && many) MAMBA_CONV_LAUNCH(4, MAMBA_CONV_ROWS);
-  else if (s.taps == 4) MAMBA_CONV_LAUNCH(4, 1);
-  else if (s.taps == 3 && many) MAMBA_CONV_LAUNCH(3, MAMBA_CONV_ROWS);
-  else if (s.taps == 2 && many) MAMBA_CONV_LAUNCH(2, MAMBA_CONV_ROWS);
-  else if (many) MAMBA_CONV_LAUNCH(0, MAMBA_CONV_ROWS);
-  else MAMBA_CONV_LAUNCH(0, 1);
-#undef MAMBA_CONV_LAUNCH
-  if (write_state && s.taps > 1)
-    SRB_CUDA_CALL(srb_launch(mamba_conv_keep_kernel<T>, keep_grid, dim3(block), 0, st, (const T*)proj, positions, cu_rows,
-                             state_slots, state, s));
-  SRB_LAUNCH_CHECK("mamba_conv");
-  return SRB_OK;
-}
-
-// proj: [rows, pitch]; weight [channels, taps], bias [channels] (float); out: [rows, channels] of `out_dtype` (float,
-// or bfloat16 beside a bfloat16 projection: what the chunk kernels read)
-extern "C" int srb_mamba_conv(const void* proj, long long proj_pitch, const float* weight, const float* bias,
-                              const int* positions, const int* row_request, const int* cu_rows, const int* state_slots,
-                              float* state, long long slot_floats, void* out, int rows, int requests, int heads, int vdim,
-                              int nstate, int groups, int taps, int write_state, int dtype, int out_dtype, void* stream) {
-  if (rows <= 0 || requests <= 0) return SRB_OK;
-  MambaShape s;
-  if (mamba_shape(s, heads, vdim, nstate, groups, taps, proj_pitch, slot_floats) != SRB_OK) return SRB_ERR_INVALID;
-  if (requests > 65535) SRB_FAIL("mamba_conv: %d requests exceed one launch", requests);
-  cudaStream_t st = (cudaStream_t)stream;
-  if (dtype == SRB_DTYPE_F32 && out_dtype == SRB_DTYPE_F32)
-    return launch_mamba_conv<float, float>(proj, weight, bias, positions, row_request, cu_rows, state_slots, state, out, rows,
-                                           requests, write_state, s, st);
-  if (dtype == SRB_DTYPE_BF16 && out_dtype == SRB_DTYPE_F32)
-    return launch_mamba_conv<__nv_bfloat16, float>(proj, weight, bias, positions, row_request, cu_rows, state_slots, state, out,
-                                                   rows, requests, write_state, s, st);
-  if (dtype == SRB_DTYPE_BF16 && out_dtype == SRB_DTYPE_BF16)
-    return launch_mamba_conv<__nv_bfloat16, __nv_bfloat16>(proj, weight, bias, positions, row_request, cu_rows, state_slots, state,
-                                                           out, rows, requests, write_state, s, st);
-  SRB_FAIL("mamba_conv: a projection of dtype %d with a result of dtype %d is not taken", dtype, out_dtype);
-}
-
 template <typename T>
 static int launch_mamba_scan(const void* proj, const float* xbc, const float* a_log, const float* d_skip, const float* dt_bias,
                              const int* positions, const int* cu_rows, const int* state_slots, float* state, float* y,
@@ -413,7 +221,7 @@ static int launch_mamba_scan(const void* proj, const float* xbc, const float* a_
   return SRB_OK;
 }
 
-// xbc: float [rows, channels] (what srb_mamba_conv wrote); y: float [rows, inner]
+// xbc: float [rows, channels] (what srb_short_conv wrote); y: float [rows, inner]
 extern "C" int srb_mamba_scan(const void* proj, long long proj_pitch, const float* xbc, const float* a_log, const float* d_skip,
                               const float* dt_bias, const int* positions, const int* cu_rows, const int* state_slots,
                               float* state, long long slot_floats, float* y, int rows, int requests, int heads, int vdim,
@@ -829,7 +637,7 @@ extern "C" int srb_mamba_chunks_supports(int vdim, int nstate, int dtype) {
   return dtype == SRB_DTYPE_BF16 && (nstate == 64 || nstate == 128) && (vdim == 64 || vdim == 128);
 }
 
-// What srb_mamba_scan computes, for prompt portions in bfloat16.  `xbc`: bfloat16 [rows, channels] (srb_mamba_conv with a
+// What srb_mamba_scan computes, for prompt portions in bfloat16.  `xbc`: bfloat16 [rows, channels] (srb_short_conv with a
 // bfloat16 result); `chunks`: at least the number of chunks of the step, sum over the requests of ceil(rows /
 // srb_mamba_chunk_tokens()); `scratch`: chunks * heads * (N * P + 1) floats.
 extern "C" int srb_mamba_chunks(const void* proj, long long proj_pitch, const void* xbc, const float* a_log, const float* d_skip,

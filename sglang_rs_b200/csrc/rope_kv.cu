@@ -651,6 +651,8 @@ extern "C" int srb_qk_norm_rope_kv_ex(const void* qkv, const float* qkv_parts, i
 // Behind the values the projection may hold `gate_cols` logits of an output gate: their sigmoids are written, in
 // 32-bit, to `gate_out` [rows, gate_cols] for the attention kernel that multiplies its result by them.
 // Row of the projection: [n_q * head_dim | n_kv * head_dim | n_kv * value_dim | gate_cols].
+// With `per_head` every q and k head is instead divided by its own root mean square and multiplied by a weight
+// [head_dim] that all heads of its kind share.
 // One block per row; sums of squares, norms, angles and the rotation are 32-bit; a norm whose weight is null is left out.
 // Sum of two values over a block of up to 1024 threads at once; every thread receives both.  Warp partials are added in
 // warp order, so the results do not depend on timing.
@@ -675,7 +677,7 @@ proj_norm_rope_kv_kernel(const T* __restrict__ qkv, const float* __restrict__ qk
                          const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
                          const float* __restrict__ inv_freq, int rotary_dim, int interleaved, float magnitude, int n_q,
                          int n_kv, int head_dim, int value_dim, int gate_cols, int page_size, int num_pages,
-                         int* error_word) {
+                         int* error_word, int per_head) {
   extern __shared__ __align__(16) float staged[];       // the row (q, k, v, gate logits), rotary_dim cosines and sines, 66 of scratch
   const int q_width = n_q * head_dim, k_width = n_kv * head_dim, v_width = n_kv * value_dim;
   const int row_width = q_width + k_width + v_width + gate_cols;
@@ -773,17 +775,23 @@ proj_norm_rope_kv_kernel(const T* __restrict__ qkv, const float* __restrict__ qk
     }
   }
   const float2 sums = block_sum_pair(sum_q, sum_k, scratch);     // (its barrier also publishes the tables and the staged row)
-  const float inv_q = q_weight ? 1.0f / sqrtf(sums.x / (float)q_width + eps) : 1.f;
-  const float inv_k = k_weight ? 1.0f / sqrtf(sums.y / (float)k_width + eps) : 1.f;
+  const float inv_q = q_weight && !per_head ? 1.0f / sqrtf(sums.x / (float)q_width + eps) : 1.f;
+  const float inv_k = k_weight && !per_head ? 1.0f / sqrtf(sums.y / (float)k_width + eps) : 1.f;
   // norm and rotation of a pair by the thread that owns it; entries behind the rotated ones are normed one by one
   // (a warp per head and a lane per pair: no division in the loop)
   const int rest = head_dim - rotary_dim;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   for (int head = warp; head < n_q + n_kv; head += warps) {
     float* v = staged + (size_t)head * head_dim;
-    const float* w = head < n_q ? (q_weight ? q_weight + (size_t)head * head_dim : nullptr)
-                                : (k_weight ? k_weight + (size_t)(head - n_q) * head_dim : nullptr);
-    const float inv = head < n_q ? inv_q : inv_k;
+    const float* w = head < n_q ? q_weight : k_weight;
+    float inv = head < n_q ? inv_q : inv_k;
+    if (w && per_head) {
+      float squares = 0.f;
+      for (int e = lane; e < head_dim; e += 32) squares = __fmaf_rn(v[e], v[e], squares);
+      inv = 1.0f / sqrtf(srb_warp_sum(squares) / (float)head_dim + eps);
+    } else if (w) {
+      w += (size_t)(head < n_q ? head : head - n_q) * head_dim;
+    }
     for (int i = lane; i < half; i += 32) {
       const int ia = interleaved ? 2 * i : i, ib = interleaved ? 2 * i + 1 : i + half;
       const float a = w ? normed(v[ia], inv, w[ia]) : v[ia], b = w ? normed(v[ib], inv, w[ib]) : v[ib];
@@ -839,7 +847,7 @@ extern "C" int srb_proj_norm_rope_kv(const void* qkv, const float* qkv_parts, in
                                      const int* positions, const int* slots, const float* q_weight, const float* k_weight,
                                      float eps, const float* inv_freq, int rotary_dim, int interleaved, float magnitude,
                                      int rows, int n_q, int n_kv, int head_dim, int value_dim, int gate_cols, int page_size,
-                                     int num_pages, int* error_word, int dtype, void* stream) {
+                                     int num_pages, int* error_word, int dtype, int per_head, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (n_q <= 0 || n_kv <= 0 || head_dim <= 0 || value_dim <= 0 || page_size <= 0 || gate_cols < 0)
     SRB_FAIL("proj_norm_rope_kv: head counts, widths and page size must be positive");
@@ -868,7 +876,7 @@ extern "C" int srb_proj_norm_rope_kv(const void* qkv, const float* qkv_parts, in
     SRB_CUDA_CALL(srb_launch(proj_norm_rope_kv_kernel<T, EIGHT>, dim3(rows), dim3(threads), smem, s, (const T*)qkv, qkv_parts, \
                              num_parts, (size_t)part_stride, qkv_stride, (T*)q_out, (T*)k_pool, (T*)v_pool, gate_out,          \
                              positions, slots, q_weight, k_weight, eps, inv_freq, rotary_dim, interleaved, magnitude, n_q,     \
-                             n_kv, head_dim, value_dim, gate_cols, page_size, num_pages, error_word));                         \
+                             n_kv, head_dim, value_dim, gate_cols, page_size, num_pages, error_word, per_head));               \
   } while (0)
   if (dtype == SRB_DTYPE_F32) {
     if (eight) SRB_PROJ_LAUNCH(float, true); else SRB_PROJ_LAUNCH(float, false);

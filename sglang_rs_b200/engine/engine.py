@@ -24,8 +24,8 @@ from .scheduler import Request, Scheduler, SchedulerConfig, StepOutput
 
 
 def kv_bytes_per_token(model, dtype: torch.dtype) -> int:
-    from ..parts.base import PagedKV
-    width = sum(need.num_kv_heads * (need.head_dim + need.value_width) for need in model.cache_needs()
+    from ..parts.base import PagedKV, simple_needs
+    width = sum(need.num_kv_heads * (need.head_dim + need.value_width) for need in simple_needs(model.cache_needs())
                 if isinstance(need, PagedKV))
     return width * (4 if dtype == torch.float32 else 2)
 

@@ -75,6 +75,30 @@ def _need(tensor: torch.Tensor, name: str, dtype: Optional[torch.dtype] = None) 
         raise KernelError(f"{name} must be {dtype}, found {tensor.dtype}")
 
 
+def _need_rows(tensor: torch.Tensor, name: str, dtype: Optional[torch.dtype] = None) -> None:
+    """A matrix on the device whose rows are dense; they may lie further apart than they are long."""
+    if not tensor.is_cuda:
+        raise KernelError(f"{name} must be a CUDA tensor; this engine has no host path")
+    if tensor.dim() != 2 or tensor.stride(1) != 1 or tensor.stride(0) < tensor.shape[1]:
+        raise KernelError(f"{name} must be a matrix with dense rows")
+    if dtype is not None and tensor.dtype != dtype:
+        raise KernelError(f"{name} must be {dtype}, found {tensor.dtype}")
+
+
+def _rows_on_16_bytes(x: torch.Tensor) -> bool:
+    """True if every row of the matrix starts on a 16-byte border."""
+    return x.stride(0) * x.element_size() % 16 == 0 and x.data_ptr() % 16 == 0
+
+
+def _head_rows(out: torch.Tensor, name: str, dtype: torch.dtype) -> int:
+    """Elements between rows of ``out`` [rows, heads, width], whose heads lie densely side by side inside a row."""
+    if not out.is_cuda or out.dtype != dtype:
+        raise KernelError(f"{name} must be a CUDA tensor of {dtype}")
+    if out.dim() != 3 or out.stride(2) != 1 or out.stride(1) != out.shape[2] or out.stride(0) < out.shape[1] * out.shape[2]:
+        raise KernelError(f"{name} must be [rows, heads, width] with dense heads")
+    return out.stride(0)
+
+
 #: kernels of this package launched so far (the bench reports the count of a timed region)
 launch_count = 0
 
@@ -289,7 +313,7 @@ def norm_add_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], inner, 
 #: activations of a gated feed-forward, act(gate) * up, by the numbers of csrc/activations.cuh
 ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu2": 2, "swiglu_clamp": 3}
 #: activations with a parameter (``swiglu_clamp``: min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1),
-#: the parameter being the limit); only the experts' products carry one (``routed_experts(activation_param=)``)
+#: the parameter being the limit); products that take one have an ``activation_param``
 PARAMETRIC_ACTIVATIONS = frozenset({"swiglu_clamp"})
 
 
@@ -304,15 +328,17 @@ def activation_code(name: str, parametric: bool = False) -> int:
 
 
 @traced("activation")
-def gated_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
-    """out[r, j] = act(gate_up[r, j]) * gate_up[r, inner + j]"""
+def gated_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu",
+              activation_param: Optional[float] = None) -> None:
+    """out[r, j] = act(gate_up[r, j]) * gate_up[r, inner + j] (``activation_param``: of an activation that has one)"""
     _need(gate_up, "gate_up"); _need(out, "out", gate_up.dtype)
     rows, inner = out.shape
     if gate_up.shape != (rows, 2 * inner):
         raise KernelError("gated_mul: gate_up must be [rows, 2 * inner]")
     lib = load_library("elementwise")
-    _check(lib, lib.srb_gated_mul(_ptr(gate_up), _ptr(out), rows, inner, activation_code(activation),
-                                  dtype_code(out.dtype), _stream()))
+    _check(lib, lib.srb_gated_mul_param(_ptr(gate_up), _ptr(out), rows, inner,
+                                        activation_code(activation, activation_param is not None),
+                                        ctypes.c_float(activation_param or 0.0), dtype_code(out.dtype), _stream()))
 
 
 @traced("bias")
@@ -394,22 +420,23 @@ def proj_norm_rope_kv(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[t
                       positions: torch.Tensor, slots: Optional[torch.Tensor], q_weight: Optional[torch.Tensor],
                       k_weight: Optional[torch.Tensor], eps: float, inv_freq: Optional[torch.Tensor], rotary_dim: int,
                       interleaved: bool, n_q: int, n_kv: int, head_dim: int, value_dim: int, error_word: torch.Tensor, *,
-                      magnitude: float = 1.0, gate_out: Optional[torch.Tensor] = None) -> None:
+                      magnitude: float = 1.0, gate_out: Optional[torch.Tensor] = None, per_head: bool = False) -> None:
     """The step between the q/k/v product and attention for a mixer that norms q and k over the WHOLE projection (all
     heads of a row together, a weight per entry: ``q_weight`` [n_q * head_dim], ``k_weight`` [n_kv * head_dim]; None: no
     norm), then rotates the leading ``rotary_dim`` entries of every head, writes q to ``q_out`` [rows, n_q, head_dim], k
     into ``k_pool`` [pages, n_kv, page_size, head_dim] and the values, as projected, into ``v_pool`` [pages, n_kv,
     page_size, value_dim].  Rows of ``qkv`` are [q | k | v | gate logits]; ``gate_out`` (float32 [rows, gates]) receives
     the sigmoids of the logits behind the values.  ``qkv`` is of ``q_out``'s dtype or float32 [parts, rows, width]
-    partial sums.  ``slots`` None: nothing is stored."""
-    _need(qkv, "qkv"); _need(q_out, "q_out"); _need(positions, "positions", torch.int32)
+    partial sums; its rows may be columns of wider ones.  ``slots`` None: nothing is stored.  ``per_head``: every q and k
+    head is normed by itself with a weight that its kind's heads share (``q_weight``, ``k_weight`` [head_dim])."""
+    _need(q_out, "q_out"); _need(positions, "positions", torch.int32)
     whole = parts = None
     num_parts = part_stride = 0
     if qkv.dim() == 3:
         _need(qkv, "qkv", torch.float32)
         parts, num_parts, part_stride = qkv, qkv.shape[0], qkv.stride(0)
     else:
-        _need(qkv, "qkv", q_out.dtype)
+        _need_rows(qkv, "qkv", q_out.dtype)
         whole = qkv
     rows = qkv.shape[-2]
     gate_cols = 0
@@ -428,7 +455,8 @@ def proj_norm_rope_kv(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[t
         num_pages, pool_heads, page_size, pool_dim = k_pool.shape
         if (pool_heads, pool_dim) != (n_kv, head_dim) or v_pool.shape != (num_pages, n_kv, page_size, value_dim):
             raise KernelError("proj_norm_rope_kv: pools must be [pages, n_kv, page_size, head_dim] and [..., value_dim]")
-    for name, w, count in (("q_weight", q_weight, n_q * head_dim), ("k_weight", k_weight, n_kv * head_dim)):
+    for name, w, count in (("q_weight", q_weight, head_dim if per_head else n_q * head_dim),
+                           ("k_weight", k_weight, head_dim if per_head else n_kv * head_dim)):
         if w is not None:
             _need(w, name, torch.float32)
             if w.numel() != count:
@@ -443,7 +471,7 @@ def proj_norm_rope_kv(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[t
         _ptr(k_pool) if slots is not None else None, _ptr(v_pool) if slots is not None else None, _ptr(gate_out),
         _ptr(positions), _ptr(slots), _ptr(q_weight), _ptr(k_weight), ctypes.c_float(eps), _ptr(inv_freq), rotary_dim,
         int(interleaved), ctypes.c_float(magnitude), rows, n_q, n_kv, head_dim, value_dim, gate_cols, page_size, num_pages,
-        _ptr(error_word), dtype_code(q_out.dtype), _stream()))
+        _ptr(error_word), dtype_code(q_out.dtype), int(per_head), _stream()))
 
 
 @traced("rope_kv")
@@ -471,7 +499,7 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                     scale: float, window: int, split_size: int, max_splits: int,
                     scratch_acc: Optional[torch.Tensor], scratch_ml: Optional[torch.Tensor],
                     error_word: torch.Tensor, sinks: Optional[torch.Tensor] = None, chunk: int = 0,
-                    gates: Optional[torch.Tensor] = None) -> None:
+                    gates: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
     """out[r, h, :] = softmax over the keys row r may see of (q . k) * scale, times v.
 
     A row at position p sees the keys max(0, p - window + 1) .. p (``window`` 0: from 0) and, with ``chunk`` > 0,
@@ -480,13 +508,15 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     ``sinks`` (float32, one per query head): the softmax's denominator also holds exp(sink_h), a term without
     key or value.  ``v_pool`` may hold rows of another width than the keys (``out`` is as wide as they are), and may be
     None: the value of a key is then the first ``out.shape[2]`` entries of its key row.  ``gates`` (float32
-    [rows, n_q]): a factor on the result of every (row, query head).
+    [rows, n_q]): a factor on the result of every (row, query head).  ``out_scale``: a factor on every result.  The rows of
+    ``out`` may lie further apart than they are long (columns of a wider matrix).
 
     q, out: [rows, n_q, head_dim]; pools [pages, n_kv, page_size, head_dim]; block_table
     [requests, stride].  ``split_size`` 0 walks all keys in one block per (row, kv head);
     otherwise partials go through the scratch tensors and are merged in split order.
     This is the generic kernel (any head_dim that is a multiple of 16, float32 or bfloat16)."""
-    _need(q, "q"); _need(out, "out", q.dtype); _need(k_pool, "k_pool", q.dtype)
+    _need(q, "q"); _need(k_pool, "k_pool", q.dtype)
+    pitch = _head_rows(out, "out", q.dtype)
     _need(positions, "positions", torch.int32); _need(row_request, "row_request", torch.int32)
     _need(block_table, "block_table", torch.int32)
     rows, n_q, head_dim = q.shape
@@ -516,7 +546,8 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(scratch_acc), _ptr(scratch_ml), _ptr(positions),
         _ptr(row_request), _ptr(block_table), block_table.stride(0), rows, n_q, n_kv, head_dim, page_size,
         num_pages, int(window), int(chunk), int(split_size), int(max_splits), ctypes.c_float(scale), _ptr(error_word),
-        dtype_code(q.dtype), _ptr(sinks), value_dim, _ptr(gates), _stream()), launches=2 if split_size else 1)
+        dtype_code(q.dtype), _ptr(sinks), value_dim, _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale),
+        _stream()), launches=2 if split_size else 1)
 
 
 
@@ -609,15 +640,17 @@ def decode_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
                      positions: torch.Tensor, row_request: torch.Tensor, block_table: torch.Tensor, *,
                      scale: float, window: int, scratch_acc: torch.Tensor, scratch_ml: torch.Tensor,
                      counters: torch.Tensor, error_word: torch.Tensor, max_keys: Optional[int] = None,
-                     chunk: int = 0, sinks: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None) -> None:
-    """Attention of decoded tokens (one row each), bfloat16, head_dim 64 or 128; ``window``, ``chunk``, ``sinks`` and
-    ``gates`` as in :func:`paged_attention` (the sink joins where a row's splits are merged, once).
+                     chunk: int = 0, sinks: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None,
+                     out_scale: float = 1.0) -> None:
+    """Attention of decoded tokens (one row each), bfloat16, head_dim 64 or 128; ``window``, ``chunk``, ``sinks``,
+    ``gates``, ``out_scale`` and the rows of ``out`` as in :func:`paged_attention` (the sink joins where a row's splits are merged, once).
 
     The keys of a (row, kv head) are shared by ``decode_splits(rows, n_kv, max_keys)`` blocks
     (``max_keys``: the most keys any row sees, if known); the block that finishes last merges them.  ``counters``: int32, zero, at least rows * n_kv entries; they
     are zero again afterwards.  Scratch: rows * n_q * splits * head_dim and rows * n_q * splits * 2
     floats."""
-    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16)
+    _need(q, "q", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16)
+    pitch = _head_rows(out, "out", q.dtype)
     _need(v_pool, "v_pool", torch.bfloat16); _need(positions, "positions", torch.int32)
     _need(row_request, "row_request", torch.int32); _need(block_table, "block_table", torch.int32)
     _need(scratch_acc, "scratch_acc", torch.float32); _need(scratch_ml, "scratch_ml", torch.float32)
@@ -647,7 +680,7 @@ def decode_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(scratch_acc), _ptr(scratch_ml), _ptr(counters),
         _ptr(positions), _ptr(row_request), _ptr(block_table), block_table.stride(0), rows, n_q, n_kv, head_dim,
         page_size, num_pages, int(window), int(chunk), splits, ctypes.c_float(scale), _ptr(error_word), _ptr(sinks),
-        _ptr(gates), _stream()))
+        _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale), _stream()))
 
 
 def tiled_attention_takes(dtype: torch.dtype, n_q: int, n_kv: int, head_dim: int) -> bool:
@@ -661,11 +694,12 @@ def tiled_attention_takes(dtype: torch.dtype, n_q: int, n_kv: int, head_dim: int
 def tiled_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
                     tiles: torch.Tensor, block_table: torch.Tensor, *, scale: float, window: int,
                     error_word: torch.Tensor, chunk: int = 0, sinks: Optional[torch.Tensor] = None,
-                    gates: Optional[torch.Tensor] = None) -> None:
-    """Attention of prompt portions, bfloat16 (``sinks``, ``gates``: as in :func:`paged_attention`).  ``tiles`` is int32 [n, 4]: first row of the
+                    gates: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
+    """Attention of prompt portions, bfloat16 (``sinks``, ``gates``, ``out_scale``, rows of ``out``: as in :func:`paged_attention`).  ``tiles`` is int32 [n, 4]: first row of the
     step, rows (at most 64, consecutive rows of one request), request index, first position.
     Rows outside the tiles are left untouched."""
-    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16)
+    _need(q, "q", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16)
+    pitch = _head_rows(out, "out", q.dtype)
     _need(v_pool, "v_pool", torch.bfloat16); _need(tiles, "tiles", torch.int32)
     _need(block_table, "block_table", torch.int32)
     rows, n_q, head_dim = q.shape
@@ -685,7 +719,7 @@ def tiled_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     _check(lib, lib.srb_prefill_attention_gated(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(tiles), tiles.shape[0], _ptr(block_table),
         block_table.stride(0), n_q, n_kv, head_dim, page_size, num_pages, int(window), int(chunk), ctypes.c_float(scale),
-        _ptr(error_word), _ptr(sinks), _ptr(gates), _stream()))
+        _ptr(error_word), _ptr(sinks), _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale), _stream()))
 
 
 TC_TILE_ROWS = 128
@@ -702,10 +736,11 @@ def tiled_attention_tc_takes(dtype: torch.dtype, n_q: int, n_kv: int, head_dim: 
 def tiled_attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
                        tiles: torch.Tensor, block_table: torch.Tensor, *, scale: float, window: int,
                        error_word: torch.Tensor, chunk: int = 0, sinks: Optional[torch.Tensor] = None,
-                       gates: Optional[torch.Tensor] = None) -> None:
+                       gates: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
     """Attention of prompt portions on tcgen05 tensor cores (S, P and O in tensor memory, operands
-    by TMA; ``sinks``, ``gates``: as in :func:`paged_attention`).  ``tiles`` as for :func:`tiled_attention`, with at most 128 rows per tile."""
-    _need(q, "q", torch.bfloat16); _need(out, "out", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16)
+    by TMA; ``sinks``, ``gates``, ``out_scale``, rows of ``out`` (16-byte borders): as in :func:`paged_attention`).  ``tiles`` as for :func:`tiled_attention`, with at most 128 rows per tile."""
+    _need(q, "q", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16)
+    pitch = _head_rows(out, "out", q.dtype)
     _need(v_pool, "v_pool", torch.bfloat16); _need(tiles, "tiles", torch.int32)
     _need(block_table, "block_table", torch.int32)
     rows, n_q, head_dim = q.shape
@@ -725,7 +760,7 @@ def tiled_attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tens
     _check(lib, lib.srb_prefill_attention_tc_gated(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(tiles), tiles.shape[0], rows, _ptr(block_table),
         block_table.stride(0), n_q, n_kv, head_dim, page_size, num_pages, int(window), int(chunk), ctypes.c_float(scale),
-        _ptr(error_word), _ptr(sinks), _ptr(gates), _stream()))
+        _ptr(error_word), _ptr(sinks), _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale), _stream()))
 
 
 # --------------------------------------------------------------------------- latents and per-head products
@@ -999,8 +1034,8 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
     crates/sglang-kernel/src/cublas.rs:383-410); both accumulate in 32-bit.  ``out_dtype``
     float32 keeps the accumulator's precision (used for the logits).  With ``partial_ok`` the
     result may be float32 [parts, rows, out]: partial sums over K that the consumer adds in
-    order (``add_rmsnorm`` and ``qk_norm_rope_kv`` do)."""
-    _need(x, "x"); _need(weight, "weight", x.dtype)
+    order (``add_rmsnorm`` and ``qk_norm_rope_kv`` do).  ``x`` may be columns of a wider matrix (dense rows, any pitch)."""
+    _need_rows(x, "x"); _need(weight, "weight", x.dtype)
     if x.dim() != 2 or weight.dim() != 2 or x.shape[1] != weight.shape[1]:
         raise KernelError(f"linear: x {tuple(x.shape)} and weight {tuple(weight.shape)} do not fit")
     m, k = x.shape
@@ -1013,7 +1048,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
         _check(lib, lib.srb_gemm_f32(_ptr(x), _ptr(weight), _ptr(bias), _ptr(out), m, n, k, x.stride(0),
                                      weight.stride(0), out.stride(0), _stream()))
         return out
-    if m <= OWN_GEMM_MAX_TOKENS and error_word is not None and gemm_bf16_takes(k):
+    if m <= OWN_GEMM_MAX_TOKENS and error_word is not None and gemm_bf16_takes(k) and _rows_on_16_bytes(x):
         splits = gemm_splits(m, n, k) if partial_ok else 1
         if splits > 1:
             out = gemm_bf16(x, weight, error_word, mode="partial", splits=splits)
@@ -1045,22 +1080,24 @@ def library_product(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtyp
 
 @traced("gemm")
 def gated_product(x: torch.Tensor, weight: torch.Tensor, inner: int, error_word: Optional[torch.Tensor] = None,
-                  activation: str = "silu") -> torch.Tensor:
-    """act(x gate^T) * (x up^T) for ``weight`` = gate rows stacked over up rows [2 inner, in].
+                  activation: str = "silu", activation_param: Optional[float] = None) -> torch.Tensor:
+    """act(x gate^T) * (x up^T) for ``weight`` = gate rows stacked over up rows [2 inner, in] (``activation_param``: the
+    parameter of an activation that has one).
 
     bfloat16 with few rows: one tcgen05 kernel whose epilogue takes the product of its two
     accumulators, so the [rows, 2 inner] intermediate never exists; with many rows the CTA-pair
     kernel does the same.  Otherwise the product (``linear``) followed by the activation kernel."""
     if (x.dtype == torch.bfloat16 and x.shape[0] <= OWN_GEMM_MAX_TOKENS and error_word is not None
             and gemm_bf16_takes(x.shape[1])):
-        return gemm_bf16(x, weight, error_word, mode="gated", features=inner, up_row_offset=inner, activation=activation)
+        return gemm_bf16(x, weight, error_word, mode="gated", features=inner, up_row_offset=inner, activation=activation,
+                         activation_param=activation_param)
     if (x.dtype == torch.bfloat16 and error_word is not None and weight.shape[0] == 2 * inner
             and pair_gemm_takes(x.shape[0], inner, x.shape[1])):
         return gemm_bf16_pair(x, weight, error_word, mode="gated", features=inner, up_row_offset=inner,
-                              activation=activation)
+                              activation=activation, activation_param=activation_param)
     gate_up = linear(x, weight, error_word=error_word)
     act = torch.empty((x.shape[0], inner), dtype=x.dtype, device=x.device)
-    gated_mul(gate_up, act, activation)
+    gated_mul(gate_up, act, activation, activation_param)
     return act
 
 
@@ -1072,7 +1109,8 @@ GEMM_CLUSTER_SPLITS = 8
 @traced("gemm")
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, error_word: torch.Tensor, *, mode: str = "bf16",
               features: Optional[int] = None, up_row_offset: int = 0, splits: int = 1,
-              out: Optional[torch.Tensor] = None, activation: str = "silu") -> torch.Tensor:
+              out: Optional[torch.Tensor] = None, activation: str = "silu",
+              activation_param: Optional[float] = None) -> torch.Tensor:
     """y = x @ w^T on tcgen05 tensor cores (bfloat16 in, 32-bit accumulation).
 
     x [tokens, k], w [rows, k], k a multiple of 8.  ``mode``: ``bf16`` / ``f32`` store
@@ -1085,7 +1123,7 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, error_word: torch.Tensor, *, mod
     (The engine's decode steps do not use ``add``: measured at Qwen3-8B sizes, partial sums that the
     next norm kernel adds are quicker, 3.22 / 3.48 / 7.21 ms per step at batch 1 / 8 / 64 against
     3.37 / 3.52 / 7.69 ms, because clusters of 8 blocks start later and end with two cluster barriers.)"""
-    _need(x, "x", torch.bfloat16); _need(w, "w", torch.bfloat16)
+    _need_rows(x, "x", torch.bfloat16); _need(w, "w", torch.bfloat16)
     tokens, k = x.shape
     rows = w.shape[0]
     if w.shape[1] != k:
@@ -1107,15 +1145,17 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, error_word: torch.Tensor, *, mod
         splits = 1
         out = torch.empty((tokens, features), dtype=torch.float32 if mode == "f32" else torch.bfloat16, device=x.device)
     lib = load_library("gemm_bf16")
-    _check(lib, lib.srb_gemm_bf16(_ptr(x), _ptr(w), _ptr(out), tokens, features, k, x.stride(0), w.stride(0), pitch,
-                                  rows, int(up_row_offset), code, int(splits), activation_code(activation),
-                                  _ptr(error_word), _stream()))
+    _check(lib, lib.srb_gemm_bf16_param(_ptr(x), _ptr(w), _ptr(out), tokens, features, k, x.stride(0), w.stride(0), pitch,
+                                        rows, int(up_row_offset), code, int(splits),
+                                        activation_code(activation, activation_param is not None),
+                                        ctypes.c_float(activation_param or 0.0), _ptr(error_word), _stream()))
     return out
 
 
 @traced("gemm")
 def gemm_bf16_pair(x: torch.Tensor, w: torch.Tensor, error_word: torch.Tensor, *, mode: str = "bf16",
-                   features: Optional[int] = None, up_row_offset: int = 0, activation: str = "silu") -> torch.Tensor:
+                   features: Optional[int] = None, up_row_offset: int = 0, activation: str = "silu",
+                   activation_param: Optional[float] = None) -> torch.Tensor:
     """y = x @ w^T for many tokens: 256 x 256 tiles on pairs of CTAs (``tcgen05.mma.cta_group::2``) in a
     persistent kernel.  ``mode`` ``bf16``, ``gated`` or ``act`` as in :func:`gemm_bf16`; the result is bfloat16."""
     _need(x, "x", torch.bfloat16); _need(w, "w", torch.bfloat16)
@@ -1128,9 +1168,10 @@ def gemm_bf16_pair(x: torch.Tensor, w: torch.Tensor, error_word: torch.Tensor, *
     pitch = -(-features // 8) * 8
     out = torch.empty((tokens, pitch), dtype=torch.bfloat16, device=x.device)
     lib = load_library("gemm_bf16_pair")
-    _check(lib, lib.srb_gemm_bf16_pair(_ptr(x), _ptr(w), _ptr(out), tokens, features, k, x.stride(0), w.stride(0), pitch,
-                                       rows, int(up_row_offset), GEMM_MODES[mode], activation_code(activation),
-                                       _ptr(error_word), _stream()))
+    _check(lib, lib.srb_gemm_bf16_pair_param(_ptr(x), _ptr(w), _ptr(out), tokens, features, k, x.stride(0), w.stride(0), pitch,
+                                             rows, int(up_row_offset), GEMM_MODES[mode],
+                                             activation_code(activation, activation_param is not None),
+                                             ctypes.c_float(activation_param or 0.0), _ptr(error_word), _stream()))
     return out if pitch == features else out[:, :features]
 
 
@@ -1381,30 +1422,47 @@ def _mamba_args(proj, state, heads, vdim, nstate, groups, taps):
         raise KernelError("mamba: rows of the in-projection are too short")
 
 
-@traced("mamba_conv")
-def mamba_conv(proj: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, positions: torch.Tensor, row_request: torch.Tensor,
-               cu_rows: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor, num_requests: int, *,
-               heads: int, vdim: int, nstate: int, groups: int, taps: int, read_only: bool = False) -> None:
-    """The causal convolution per channel and SiLU of the x, B and C entries of ``proj``'s rows
-    ([z | x | B | C | dt]); ``out`` [rows, channels], float32 or (beside a bfloat16 ``proj``, for :func:`mamba_chunks`)
-    bfloat16.  Inputs before a request's first row of the step come from
-    its slot of ``state`` (zeros before position 0); unless ``read_only`` the slot then keeps the sequence's last
-    ``taps`` - 1 inputs.  ``weight`` float32 [channels, taps] (the last column is the current token's), ``bias`` [channels]."""
-    _mamba_args(proj, state, heads, vdim, nstate, groups, taps)
-    channels = heads * vdim + 2 * groups * nstate
-    _need(weight, "weight", torch.float32); _need(bias, "bias", torch.float32)
+@traced("short_conv")
+def short_conv(proj: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], positions: torch.Tensor,
+               row_request: torch.Tensor, cu_rows: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+               num_requests: int, *, read_only: bool = False, single_rows: bool = False) -> None:
+    """A causal convolution over time per channel, then SiLU: out[t, c] = silu(bias[c] + sum_j weight[c, j] u[t - taps + 1 + j, c]).
+
+    ``proj`` [rows, channels]: the inputs u, columns of a wider projection (dense rows, any pitch); ``weight`` float32
+    [channels, taps] (the last column is the current token's), ``bias`` float32 [channels] or None; ``out`` [rows, channels],
+    float32 or (beside a bfloat16 ``proj``) bfloat16.  Inputs before a request's first row of the step come from the first
+    (taps - 1) * channels floats of its slot of ``state`` (float32 [slots, floats]; zeros before position 0); unless
+    ``read_only`` the slot then keeps the sequence's last taps - 1 inputs.  ``single_rows``: every request of the step brings
+    exactly one row (decoded tokens): one launch then does both."""
+    _need_rows(proj, "proj"); _need(weight, "weight", torch.float32); _need(state, "state", torch.float32)
     _need(out, "out", torch.float32 if out.dtype != proj.dtype else proj.dtype)
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
     for name, t in (("positions", positions), ("row_request", row_request), ("cu_rows", cu_rows), ("state_slots", state_slots)):
         _need(t, name, torch.int32)
-    rows = proj.shape[0]
-    if weight.shape != (channels, taps) or bias.numel() != channels or out.shape != (rows, channels):
-        raise KernelError("mamba_conv: shapes of the filter, its bias and the output do not agree")
-    lib = load_library("mamba")
-    _check(lib, lib.srb_mamba_conv(_ptr(proj), ctypes.c_longlong(proj.stride(0)), _ptr(weight), _ptr(bias), _ptr(positions),
-                                   _ptr(row_request), _ptr(cu_rows), _ptr(state_slots), _ptr(state),
-                                   ctypes.c_longlong(state.stride(0)), _ptr(out), rows, int(num_requests), heads, vdim, nstate,
-                                   groups, taps, int(not read_only), dtype_code(proj.dtype), dtype_code(out.dtype), _stream()),
-           launches=1 if read_only or taps == 1 else 2)
+    rows, channels = proj.shape
+    if weight.dim() != 2 or weight.shape[0] != channels or (bias is not None and bias.numel() != channels) or out.shape != proj.shape:
+        raise KernelError("short_conv: shapes of the filter, its bias and the output do not agree")
+    if state.dim() != 2 or state.shape[1] < (weight.shape[1] - 1) * channels:
+        raise KernelError("short_conv: the state must be float32 [slots, at least (taps - 1) * channels]")
+    taps = weight.shape[1]
+    lib = load_library("short_conv")
+    _check(lib, lib.srb_short_conv(
+        _ptr(proj), ctypes.c_longlong(proj.stride(0)), _ptr(weight), _ptr(bias), _ptr(positions), _ptr(row_request), _ptr(cu_rows),
+        _ptr(state_slots), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(out), rows, int(num_requests), channels, taps,
+        int(not read_only), int(single_rows), dtype_code(proj.dtype), dtype_code(out.dtype), _stream()),
+        launches=1 if read_only or taps == 1 or single_rows else 2)
+
+
+def mamba_conv(proj: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, positions: torch.Tensor, row_request: torch.Tensor,
+               cu_rows: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor, num_requests: int, *,
+               heads: int, vdim: int, nstate: int, groups: int, taps: int, read_only: bool = False,
+               single_rows: bool = False) -> None:
+    """:func:`short_conv` of the x, B and C entries of ``proj``'s rows ([z | x | B | C | dt])."""
+    _mamba_args(proj, state, heads, vdim, nstate, groups, taps)
+    inner, channels = heads * vdim, heads * vdim + 2 * groups * nstate
+    short_conv(proj[:, inner:inner + channels], weight, bias, positions, row_request, cu_rows, state_slots, state, out,
+               num_requests, read_only=read_only, single_rows=single_rows)
 
 
 @traced("mamba_scan")
@@ -1484,6 +1542,113 @@ def mamba_gate_norm(y: torch.Tensor, proj: torch.Tensor, weight: torch.Tensor, e
     lib = load_library("mamba")
     _check(lib, lib.srb_mamba_gate_norm(_ptr(y), _ptr(proj), ctypes.c_longlong(proj.stride(0)), _ptr(weight), ctypes.c_float(eps),
                                         rows, inner, int(norm_groups), _ptr(out), dtype_code(proj.dtype), _stream()))
+
+
+# --------------------------------------------------------------------------- the gated delta rule over a state per request
+
+def delta_slot_floats(heads: int, kv_heads: int, dim: int, vdim: int, taps: int) -> int:
+    """Floats of state per request: the convolution's last ``taps`` - 1 inputs [taps - 1, channels], then S [heads, vdim,
+    dim], each padded to a multiple of four (srb_delta_slot_floats)."""
+    conv = (taps - 1) * (2 * kv_heads * dim + heads * vdim)
+    return -(-(-(-conv // 4) * 4 + heads * dim * vdim) // 4) * 4
+
+
+def _delta_args(qkv, beta, decay, a_log, dt_bias, positions, cu_rows, state_slots, state, out, heads, kv_heads, dim, vdim, taps,
+                channel_decay):
+    _need(state, "state", torch.float32); _need(out, "out", torch.float32); _need(qkv, "qkv")
+    _need_rows(beta, "beta"); _need_rows(decay, "decay", beta.dtype)
+    rows = qkv.shape[0]
+    columns = heads * dim if channel_decay else heads
+    for name, t, count in (("a_log", a_log, heads), ("dt_bias", dt_bias, columns)):
+        _need(t, name, torch.float32)
+        if t.numel() != count:
+            raise KernelError(f"delta: {name} needs {count} entries")
+    for name, t in (("positions", positions), ("cu_rows", cu_rows), ("state_slots", state_slots)):
+        _need(t, name, torch.int32)
+    if qkv.shape != (rows, 2 * kv_heads * dim + heads * vdim) or beta.shape != (rows, heads) or decay.shape != (rows, columns) \
+            or out.shape != (rows, heads * vdim):
+        raise KernelError("delta: shapes of the convolved inputs, the logits and the output do not agree")
+    if state.dim() != 2 or state.shape[1] != delta_slot_floats(heads, kv_heads, dim, vdim, taps):
+        raise KernelError("delta: the state must be float32 [slots, floats per slot]")
+    return (_ptr(qkv), _ptr(beta), ctypes.c_longlong(beta.stride(0)), _ptr(decay), ctypes.c_longlong(decay.stride(0)), _ptr(a_log),
+            _ptr(dt_bias), _ptr(positions), _ptr(cu_rows), _ptr(state_slots), _ptr(state), ctypes.c_longlong(state.stride(0)))
+
+
+@traced("delta")
+def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+               positions: torch.Tensor, cu_rows: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+               num_requests: int, *, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, channel_decay: bool, unit_eps: float,
+               read_only: bool = False) -> None:
+    """The gated delta rule, token by token from each request's state, all in 32-bit: per head (with unit vectors q, k and
+    q times dim^-1/2) S <- g S, u = sigmoid(beta) (v - S^T k), S <- S + k u^T, out = S^T q, where g =
+    exp(-exp(a_log) softplus(decay + dt_bias)) is one number per head or, with ``channel_decay``, one per row of S.
+
+    ``qkv`` float32 [rows, channels]: q (kv_heads * dim) | k (kv_heads * dim) | v (heads * vdim), as :func:`short_conv` wrote
+    them; ``beta`` [rows, heads] and ``decay`` [rows, heads (* dim)]: columns of projections; ``state`` float32 [slots,
+    ``delta_slot_floats``]; ``out`` float32 [rows, heads * vdim].  ``unit_eps`` stands beside the sum of squares of q and k."""
+    _need(qkv, "qkv", torch.float32)
+    args = _delta_args(qkv, beta, decay, a_log, dt_bias, positions, cu_rows, state_slots, state, out, heads, kv_heads, dim, vdim, taps,
+                       channel_decay)
+    lib = load_library("delta")
+    _check(lib, lib.srb_delta_scan(*args, _ptr(out), qkv.shape[0], int(num_requests), heads, kv_heads, dim, vdim, taps,
+                                   int(channel_decay), ctypes.c_float(unit_eps), int(not read_only), dtype_code(beta.dtype), _stream()))
+
+
+def delta_chunks_takes(dtype: torch.dtype, dim: int, vdim: int) -> bool:
+    """True if the chunk kernels for prompt portions take these sizes (the rule of srb_delta_chunks_supports)."""
+    return False
+
+
+#: tokens per chunk of :func:`delta_chunks` (DC_TOKENS of csrc/delta.cu)
+DELTA_CHUNK_TOKENS = 64
+
+
+@traced("delta_gate_norm")
+def delta_gate_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, *, heads: int,
+                    silu: bool, scale: float = 1.0) -> None:
+    """Per head out = o / sqrt(mean(o^2) + eps) * weight * scale * (silu(gate) or sigmoid(gate)); ``o`` float32 [rows, heads *
+    vdim], ``gate`` and ``out`` [rows, heads * vdim], columns of wider matrices, ``weight`` float32 [vdim]."""
+    _need(o, "o", torch.float32); _need(weight, "weight", torch.float32); _need_rows(gate, "gate"); _need_rows(out, "out", gate.dtype)
+    rows, width = o.shape
+    if width % heads or gate.shape != o.shape or out.shape != o.shape or weight.numel() != width // heads:
+        raise KernelError("delta_gate_norm: shapes do not agree")
+    lib = load_library("delta")
+    _check(lib, lib.srb_delta_gate_norm(_ptr(o), _ptr(gate), ctypes.c_longlong(gate.stride(0)), _ptr(weight), ctypes.c_float(eps),
+                                        ctypes.c_float(scale), int(silu), rows, heads, width // heads, _ptr(out),
+                                        ctypes.c_longlong(out.stride(0)), dtype_code(gate.dtype), _stream()))
+
+
+# --------------------------------------------------------------------------- minGRU over a state per request
+
+#: tokens per chunk of :func:`mingru` (GRU_CHUNK of csrc/mingru.cu)
+MINGRU_CHUNK_TOKENS = 64
+
+
+@traced("mingru")
+def mingru(proj: torch.Tensor, z_at: int, x_at: int, g_at: int, z_bias: torch.Tensor, x_bias: torch.Tensor, positions: torch.Tensor,
+           cu_rows: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor, num_requests: int, chunks: int, *,
+           scale: float = 1.0, single_rows: bool = False, read_only: bool = False) -> None:
+    """Channel by channel S <- (1 - z) S + z c with z = sigmoid(z + z_bias), u = x + x_bias, c = u + 1/2 where u >= 0 and
+    sigmoid(u) elsewhere; out = scale * S silu(g).  z, x, g: the columns ``z_at`` .., ``x_at`` .., ``g_at`` .. of ``proj``;
+    ``state`` float32 [slots, width]; ``out`` [rows, width], columns of a wider matrix.  ``chunks``: the number of chunks of the
+    step, sum over the requests of ceil(rows / MINGRU_CHUNK_TOKENS), or more.  ``single_rows``: every request brings one row."""
+    _need_rows(proj, "proj"); _need(state, "state", torch.float32); _need_rows(out, "out", proj.dtype)
+    rows, width = out.shape
+    for name, t in (("z_bias", z_bias), ("x_bias", x_bias)):
+        _need(t, name, torch.float32)
+        if t.numel() != width:
+            raise KernelError(f"mingru: {name} needs {width} entries")
+    for name, t in (("positions", positions), ("cu_rows", cu_rows), ("state_slots", state_slots)):
+        _need(t, name, torch.int32)
+    if state.dim() != 2 or state.shape[1] != width or proj.shape[0] != rows or max(z_at, x_at, g_at) + width > proj.shape[1]:
+        raise KernelError("mingru: shapes of the projection, the state and the output do not agree")
+    maps = None if single_rows else torch.empty((max(int(chunks), 1), 2, width), dtype=torch.float32, device=proj.device)
+    lib = load_library("mingru")
+    _check(lib, lib.srb_mingru(_ptr(proj), ctypes.c_longlong(proj.stride(0)), int(z_at), int(x_at), int(g_at), width, _ptr(z_bias),
+                               _ptr(x_bias), _ptr(positions), _ptr(cu_rows), _ptr(state_slots), _ptr(state), _ptr(maps), _ptr(out),
+                               ctypes.c_longlong(out.stride(0)), rows, int(num_requests), max(int(chunks), 1), int(single_rows),
+                               int(not read_only), ctypes.c_float(scale), dtype_code(proj.dtype), _stream()),
+           launches=1 if single_rows else 3)
 
 
 # --------------------------------------------------------------------------- sublayers side by side, a token's own input

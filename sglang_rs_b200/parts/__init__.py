@@ -1,7 +1,8 @@
 from .attention import AttentionNames, GroupedQueryAttention
-from .base import (CacheNeed, FeedForward, Mixer, Norm, NormedDelta, PagedKV, Part, PositionEncoding, RequestState,
+from .base import (CacheNeed, FeedForward, JointNeed, Mixer, Norm, NormedDelta, PagedKV, Part, PositionEncoding, RequestState,
                    TensorSpec, matrix_to, scale_to)
-from .block import ParallelBlock, PreNormBlock, SandwichBlock
+from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
+from .delta import DeltaNames, GatedDeltaRule
 from .latent_attention import LatentAttention, LatentAttentionNames
 from .loop import PassEntry, PassSum
 from .moe import RoutedExperts
@@ -10,9 +11,11 @@ from .hyper import StreamBlock, StreamConnection, StreamNames, StreamSumNorm, St
 from .lightning import LightningAttention, LightningNames
 from .mlp import GatedMlp, GatedMlpNames, PlainMlp
 from .mamba import MambaMixer, MambaNames
+from .mingru import MinGru, MinGruNames
+from .parallel import ParallelMixer
 from .norm import GroupedRmsNorm, LayerNorm, RmsNorm
 from .side import TokenSideInput, TokenSideNames
-from .rope import NoPositionEncoding, RotaryEncoding, WavelengthScaling
+from .rope import NoPositionEncoding, RampScaling, RotaryEncoding, WavelengthScaling
 
 __all__ = [
     "AttentionNames", "GroupedQueryAttention", "CacheNeed", "FeedForward", "Mixer", "Norm", "PagedKV", "Part",
@@ -22,4 +25,5 @@ __all__ = [
     "PairTokenEmbedding", "StreamBlock", "StreamConnection", "StreamNames", "StreamSumNorm", "StreamUpdate",
     "LightningAttention", "LightningNames", "PlainMlp", "WavelengthScaling",
     "ParallelBlock", "GroupedRmsNorm", "MambaMixer", "MambaNames", "TokenSideInput", "TokenSideNames",
+    "JointNeed", "PostNormBlock", "DeltaNames", "GatedDeltaRule", "MinGru", "MinGruNames", "ParallelMixer", "RampScaling",
 ]

@@ -14,16 +14,17 @@ holds q and k only, and the fused kernel stores the unrotated key in the value p
 see, of the keys up to its own, only those of its own chunk of ``chunk`` positions (chunks counted from
 position 0 of the sequence, whatever portion of a prompt brought the row).
 
-Four more, also off by default.  ``whole_norm``: q and k are each normed over the WHOLE projection (all heads of the row
+More, also off by default.  ``whole_norm``: q and k are each normed over the WHOLE projection (all heads of the row
 together, before they are split into heads) with a weight per entry of the projection, ``names.q_norm`` [n_q * head_dim]
 and ``names.k_norm`` [n_kv * head_dim], instead of head by head with a shared weight.  ``value_dim``: values of another
 width than queries and keys (W_v is [n_kv * value_dim, hidden], W_o [hidden, n_q * value_dim], the value pool has rows of
 that width).  ``sink``: a number that joins the softmax's denominator as exp(sink) beside the keys' terms, the same for
-every head (0 adds one to the denominator); it has no key and no value.  ``names.gate``: a matrix [n_q, hidden] whose
+every head (0 adds one to the denominator), or, with ``names.sink``, a learned number per head; it has no key and no value.  ``names.gate``: a matrix [n_q, hidden] whose
 product with the mixer's input gives a logit per head; head h's result is multiplied by its sigmoid before the output
 projection (the matrix rides in the q/k/v product, the factor in the attention kernel's last step).  A mixer with any of
 these runs ``ops.proj_norm_rope_kv`` between the product and attention; every attention kernel takes the sink and the
-gates, and the tensor-core ones serve where values are as wide as the keys.
+gates, and the tensor-core ones serve where values are as wide as the keys.  In this arrangement the mixer can stand beside
+another one (``parts/parallel.py``): it reads its columns of a joint product and writes its columns of a joint result.
 """
 from __future__ import annotations
 
@@ -33,7 +34,8 @@ from typing import Dict, Mapping, Optional
 import torch
 
 from .. import ops
-from .base import Mixer, PagedKV, PositionEncoding, TensorSpec, matrix_to, scale_to
+from .base import PagedKV, PositionEncoding, TensorSpec, matrix_to, scale_to
+from .stacking import Stackable, aligned, result_columns, stack_rows
 
 
 @dataclass(frozen=True)
@@ -49,9 +51,10 @@ class AttentionNames:
     v_bias: Optional[str] = None
     o_bias: Optional[str] = None
     gate: Optional[str] = None
+    sink: Optional[str] = None
 
 
-class GroupedQueryAttention(Mixer):
+class GroupedQueryAttention(Stackable):
     graph_safe = True
     #: what the attention kernels take: the generic one gives a warp to each query head of a kv head (at most
     #: 32 warps a block) and keeps up to 16 values of a head per lane
@@ -82,7 +85,10 @@ class GroupedQueryAttention(Mixer):
         #: whether the output product may hand on partial sums along K (a consumer that cannot add them says no)
         self.partial_sums = bool(partial_sums)
         #: the arrangement that ``ops.proj_norm_rope_kv`` prepares
-        self.wide = self.whole_norm or self.vd != self.d or self.sink is not None or names.gate is not None
+        self.wide = (self.whole_norm or self.vd != self.d or self.sink is not None or names.gate is not None
+                     or names.sink is not None)
+        if self.sink is not None and names.sink is not None:
+            raise ValueError("a sink is one number for all heads or a learned one per head, not both")
         if not self.wide and num_heads // num_kv_heads > self.MAX_HEADS_PER_KV_HEAD:
             # (the fused per-head kernel's limit; the other arrangement goes through kernels that take the heads of a kv
             # head in chunks)
@@ -116,6 +122,8 @@ class GroupedQueryAttention(Mixer):
             specs[n.k_norm] = TensorSpec((self.n_kv * self.d if self.whole_norm else self.d,), "scale")
         if n.gate:
             specs[n.gate] = TensorSpec((self.n_q, self.hidden))
+        if n.sink:
+            specs[n.sink] = TensorSpec((self.n_q,))
         for name, width in ((n.q_bias, self.n_q * self.d), (n.k_bias, self.n_kv * self.d),
                             (n.v_bias, self.n_kv * self.d), (n.o_bias, self.hidden)):
             if name:
@@ -124,11 +132,25 @@ class GroupedQueryAttention(Mixer):
         return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor], device, dtype: torch.dtype) -> None:
+        first, last = self.load_inner(tensors, device, dtype)
+        self.w_qkv, self.w_o = matrix_to(first, device, dtype), matrix_to(last, device, dtype)
+
+    @property
+    def in_width(self) -> int:
+        width = self.n_q * self.d + self.n_kv * (self.d + (0 if self.values_from_keys else self.vd)) + (self.n_q if self.names.gate else 0)
+        return aligned(width) if self.wide else width
+
+    @property
+    def out_width(self) -> int:
+        return self.n_q * self.vd
+
+    def load_inner(self, tensors: Mapping[str, torch.Tensor], device, dtype: torch.dtype):
         n = self.names
         stacked = [tensors[n.q], tensors[n.k]] + ([tensors[n.v]] if n.v else []) + ([tensors[n.gate]] if n.gate else [])
         self.sinks = torch.full((self.n_q,), self.sink, dtype=torch.float32, device=device) if self.sink is not None else None
-        self.w_qkv = matrix_to(torch.cat(stacked, dim=0), device, dtype)
-        self.w_o = matrix_to(tensors[n.o], device, dtype)
+        if n.sink:
+            self.sinks = scale_to(tensors[n.sink], device)
+        first = torch.cat(stacked, dim=0)
         self.q_norm = scale_to(tensors[n.q_norm], device) if n.q_norm else None
         self.k_norm = scale_to(tensors[n.k_norm], device) if n.k_norm else None
         if n.q_bias or n.k_bias or n.v_bias:
@@ -139,6 +161,7 @@ class GroupedQueryAttention(Mixer):
             self.b_qkv = scale_to(torch.cat(parts), device)
         self.b_o = scale_to(tensors[n.o_bias], device) if n.o_bias else None
         self.position.load(tensors, device, dtype)
+        return stack_rows([first]) if self.wide else first, tensors[n.o]
 
     def native_record(self):
         """This mixer for the step executor, or None if its position encoding is not of the kind the fused
@@ -162,12 +185,14 @@ class GroupedQueryAttention(Mixer):
         batch = ctx.paged[cache.group]
         rows = x.shape[0]
         qkv = ops.linear(x, self.w_qkv, self.b_qkv, error_word=ctx.error_word, partial_ok=True)
-        q = torch.empty((rows, self.n_q, self.d), dtype=x.dtype, device=x.device)
-        rotary = self.position.fused_rotary() if self.position.fused else None
         if not self.position.fused:
             raise NotImplementedError("a position encoding with kernels of its own is applied by its mixer")
         if self.wide:
-            return self._forward_wide(ctx, cache, batch, qkv, q, rotary)
+            out = result_columns(rows, self.out_width, x.dtype, x.device)
+            self.mix(ctx, cache, qkv, out)
+            return ops.linear(out, self.w_o, self.b_o, error_word=ctx.error_word, partial_ok=self.partial_sums)
+        rotary = self.position.fused_rotary()
+        q = torch.empty((rows, self.n_q, self.d), dtype=x.dtype, device=x.device)
         ops.qk_norm_rope_kv(
             qkv, q, cache.k_pool if cache.writable else None, cache.v_pool if cache.writable else None,
             ctx.positions, batch.slots if cache.writable else None, self.q_norm, self.k_norm,
@@ -181,23 +206,25 @@ class GroupedQueryAttention(Mixer):
         return ops.linear(out.view(rows, self.n_q * self.d), self.w_o, self.b_o, error_word=ctx.error_word,
                           partial_ok=self.partial_sums)
 
-    def _attend(self, ctx, cache, batch, q, out, gates) -> None:
+    def _attend(self, ctx, cache, batch, q, out, gates, scale: float = 1.0) -> None:
         """The step's attention launches: the tensor-core kernels where they take the sizes (values as wide as the keys,
-        heads of 64 or 128), the generic kernel elsewhere; the sink and the gates go to whichever runs."""
+        heads of 64 or 128), the generic kernel elsewhere; the sink, the gates and the factor ``scale`` go to whichever
+        runs."""
         chunk, sinks = self.chunk or 0, self.sinks
-        same_width = self.vd == self.d
+        # (the tensor-core kernels for prompt portions store 16 bytes at a time)
+        same_width = self.vd == self.d and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
         for launch in batch.launches:
             b, e = launch.begin, launch.end
             if same_width and launch.wide_tiles is not None and ops.tiled_attention_tc_takes(
                     q.dtype, self.n_q, self.n_kv, self.d, cache.k_pool.shape[2]):
                 ops.tiled_attention_tc(q, cache.k_pool, cache.v_pool, out, launch.wide_tiles, batch.block_table,
                                        scale=self.scale, window=self.window or 0, error_word=ctx.error_word, chunk=chunk,
-                                       sinks=sinks, gates=gates)
+                                       sinks=sinks, gates=gates, out_scale=scale)
                 continue
             if same_width and launch.tiles is not None and ops.tiled_attention_takes(q.dtype, self.n_q, self.n_kv, self.d):
                 ops.tiled_attention(q, cache.k_pool, cache.v_pool, out, launch.tiles, batch.block_table,
                                     scale=self.scale, window=self.window or 0, error_word=ctx.error_word, chunk=chunk,
-                                    sinks=sinks, gates=gates)
+                                    sinks=sinks, gates=gates, out_scale=scale)
                 continue
             row_gates = None if gates is None else gates[b:e]
             if (same_width and launch.tiles is None and launch.split_size and batch.counters is not None
@@ -208,30 +235,31 @@ class GroupedQueryAttention(Mixer):
                                      window=self.window or 0, scratch_acc=batch.scratch_acc,
                                      scratch_ml=batch.scratch_ml, counters=batch.counters,
                                      error_word=ctx.error_word, max_keys=launch.max_keys, chunk=chunk, sinks=sinks,
-                                     gates=row_gates)
+                                     gates=row_gates, out_scale=scale)
                 continue
             ops.paged_attention(q[b:e], cache.k_pool, cache.v_pool, out[b:e], ctx.positions[b:e],
                                 ctx.row_request[b:e], batch.block_table, scale=self.scale,
                                 window=self.window or 0, split_size=launch.split_size,
                                 max_splits=launch.max_splits, scratch_acc=batch.scratch_acc,
                                 scratch_ml=batch.scratch_ml, error_word=ctx.error_word, chunk=chunk, sinks=sinks,
-                                gates=row_gates)
+                                gates=row_gates, out_scale=scale)
 
-    def _forward_wide(self, ctx, cache, batch, qkv, q, rotary) -> torch.Tensor:
-        """Norms over the whole projections, values of their own width, a sink and a gate per head: one kernel between
-        the product and attention, the attention kernels with the sink in the denominator and the gate in their last
-        step, the output product."""
+    def mix(self, ctx, cache, proj: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
+        """Norms over the whole projections or per head, values of their own width, a sink and a gate per head: one kernel
+        between the product and attention, the attention kernels with the sink in the denominator and the gate and the
+        factor in their last step."""
+        batch, rows = ctx.paged[cache.group], proj.shape[-2]
+        rotary = self.position.fused_rotary()
         if rotary is not None and rotary.angles is not None:
             raise NotImplementedError("angles computed per step are not built for this arrangement")
-        rows = q.shape[0]
+        q = torch.empty((rows, self.n_q, self.d), dtype=out.dtype, device=out.device)
         gates = torch.empty((rows, self.n_q), dtype=torch.float32, device=q.device) if self.names.gate else None
         ops.proj_norm_rope_kv(
-            qkv, q, cache.k_pool, cache.v_pool, ctx.positions, batch.slots if cache.writable else None,
-            self.q_norm if self.whole_norm else None, self.k_norm if self.whole_norm else None,
+            proj, q, cache.k_pool, cache.v_pool, ctx.positions, batch.slots if cache.writable else None,
+            self.q_norm, self.k_norm,
             self.qk_norm_eps if self.qk_norm_eps is not None else 0.0, rotary.inv_freq if rotary else None,
             rotary.rotary_dim if rotary else 0, rotary.interleaved if rotary else False, self.n_q, self.n_kv, self.d,
-            self.vd, ctx.error_word, magnitude=rotary.magnitude if rotary is not None else 1.0, gate_out=gates)
-        out = torch.empty((rows, self.n_q, self.vd), dtype=q.dtype, device=q.device)
-        self._attend(ctx, cache, batch, q, out, gates)
-        return ops.linear(out.view(rows, self.n_q * self.vd), self.w_o, self.b_o, error_word=ctx.error_word,
-                          partial_ok=self.partial_sums)
+            self.vd, ctx.error_word, magnitude=rotary.magnitude if rotary is not None else 1.0, gate_out=gates,
+            per_head=not self.whole_norm)
+        heads = out.as_strided((rows, self.n_q, self.vd), (out.stride(0), self.vd, 1))
+        self._attend(ctx, cache, batch, q, heads, gates, scale)

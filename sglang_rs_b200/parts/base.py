@@ -26,12 +26,25 @@ from typing import Dict, Mapping, Optional, Tuple, Union
 import torch
 
 
+#: a dimension of a :class:`TensorSpec` whose size the checkpoint decides
+FREE = -1
+
+
 @dataclass(frozen=True)
 class TensorSpec:
     """Shape of a checkpoint tensor and how the random-weights mode fills it:
-    ``normal`` N(0, 0.02), ``scale`` 1 + U(-0.1, 0.1), ``zeros``."""
+    ``normal`` N(0, 0.02), ``scale`` 1 + U(-0.1, 0.1), ``zeros``.
+
+    A dimension of ``FREE`` takes whatever size the checkpoint's tensor has there (a rank that no configuration names);
+    the part reads it at load.  ``free_size`` is the size the random-weights mode gives it."""
     shape: Tuple[int, ...]
     init: str = "normal"
+    free_size: int = 1
+
+    @property
+    def sample_shape(self) -> Tuple[int, ...]:
+        """The shape with every free dimension filled in, for weights that are made up."""
+        return tuple(self.free_size if size == FREE else size for size in self.shape)
 
 
 @dataclass(frozen=True)
@@ -59,7 +72,23 @@ class RequestState:
     dtype: Optional[torch.dtype] = None
 
 
-CacheNeed = Union[PagedKV, RequestState, None]
+@dataclass(frozen=True)
+class JointNeed:
+    """Several needs of one layer call: a mixer made of mixers that each keep something of their own (keys and values
+    beside a state, say).  The call is handed one cache whose ``parts`` are the needs' caches in this order."""
+    parts: Tuple[Union[PagedKV, RequestState, None], ...]
+
+
+CacheNeed = Union[PagedKV, RequestState, JointNeed, None]
+
+
+def simple_needs(needs):
+    """The needs of a model with every :class:`JointNeed` replaced by its parts."""
+    for need in needs:
+        if isinstance(need, JointNeed):
+            yield from simple_needs(need.parts)
+        else:
+            yield need
 
 
 class Part:

@@ -4,6 +4,7 @@ Pre-norm residual form (reference: crates/sglang-srt/src/cpu_reference.rs:257-31
 h' = h + mixer(norm_1(h)); h'' = h' + feed_forward(norm_2(h')).  The hidden state travels
 as (residual, delta) with h = residual + delta; each norm takes the pending sum first, in
 32-bit, so no separate add kernel runs.  :class:`SandwichBlock` norms each sublayer on both sides;
+:class:`PostNormBlock` norms only what a sublayer returns;
 :class:`ParallelBlock` runs mixer and feed-forward side by side from one norm.
 """
 from __future__ import annotations
@@ -14,6 +15,7 @@ import torch
 
 from .. import ops
 from .base import FeedForward, Mixer, Norm, NormedDelta, Part, TensorSpec
+from .norm import rounded_sum
 
 
 class PreNormBlock(Part):
@@ -108,6 +110,51 @@ class SandwichBlock(Part):
             return residual, delta
         normed = self.norm_2.add_norm(residual, delta, ctx.dtype)
         return residual, NormedDelta(self.feed_forward.forward(ctx, normed), self.norm_2b)
+
+
+class PostNormBlock(Part):
+    """A norm on each sublayer's output only: h' = h + norm_1(mixer(h)), h'' = h' + norm_2(feed_forward(h')); the sublayers
+    read the stream itself.  Without a feed-forward the block ends after the mixer.
+
+    The hidden state travels as (residual, pending) with the pending term a :class:`NormedDelta`: the norm behind a
+    sublayer, the residual sum and the rounded copy that the next sublayer's product reads are one kernel, also across
+    the border between two blocks and into the final norm."""
+
+    def __init__(self, mixer: Mixer, norm_1: Norm, feed_forward: Optional[FeedForward] = None, norm_2: Optional[Norm] = None):
+        if (feed_forward is None) != (norm_2 is None):
+            raise ValueError("a feed-forward comes with the norm behind it, or not at all")
+        self.mixer, self.norm_1, self.feed_forward, self.norm_2 = mixer, norm_1, feed_forward, norm_2
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(part.graph_safe for part in self.parts())
+
+    def parts(self):
+        return tuple(part for part in (self.mixer, self.norm_1, self.feed_forward, self.norm_2) if part is not None)
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def split_scratch(self):
+        return self.mixer.split_scratch()
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        specs: Dict[str, TensorSpec] = {}
+        for part in self.parts():
+            specs.update(part.tensor_specs())
+        return specs
+
+    def load(self, tensors: Mapping[str, torch.Tensor], device, dtype: torch.dtype) -> None:
+        for part in self.parts():
+            part.load(tensors, device, dtype)
+
+    def forward(self, ctx, cache, residual: torch.Tensor, delta):
+        stream = rounded_sum(residual, delta, ctx.dtype)
+        delta = NormedDelta(self.mixer.forward(ctx, cache, stream), self.norm_1)
+        if self.feed_forward is None:
+            return residual, delta
+        stream = rounded_sum(residual, delta, ctx.dtype)
+        return residual, NormedDelta(self.feed_forward.forward(ctx, stream), self.norm_2)
 
 
 class ParallelBlock(Part):

@@ -97,7 +97,8 @@ class MambaMixer(Mixer):
                    and ops.mamba_chunks_takes(proj.dtype, self.vdim, self.state))
         xbc = torch.empty((rows, self.channels), dtype=proj.dtype if chunked else torch.float32, device=x.device)
         ops.mamba_conv(proj, self.conv, self.conv_bias, ctx.positions, ctx.row_request, ctx.cu_rows, ctx.state_slots,
-                       cache.state, xbc, ctx.num_requests, read_only=not cache.writable, **self.sizes)
+                       cache.state, xbc, ctx.num_requests, read_only=not cache.writable,
+                       single_rows=len(counts) == ctx.num_requests and all(count == 1 for count in counts), **self.sizes)
         y = torch.empty((rows, self.inner), dtype=torch.float32, device=x.device)
         if chunked:
             # prompt portions: chunks in parallel on the tensor cores

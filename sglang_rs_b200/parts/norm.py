@@ -129,3 +129,11 @@ def add_pending(residual: torch.Tensor, delta, outer, out: Optional[torch.Tensor
         inner, delta = delta.norm.spec(), delta.values
     ops.norm_add_norm(residual, delta, inner, outer, out, row_index=row_index, write_residual=row_index is None,
                       extra=extra, addend=addend)
+
+
+def rounded_sum(residual: torch.Tensor, delta, out_dtype: torch.dtype) -> torch.Tensor:
+    """residual += delta (a tensor, a :class:`NormedDelta` or None); returns the sum rounded to ``out_dtype``: what a
+    sublayer that reads the stream itself takes."""
+    out = torch.empty(residual.shape, dtype=out_dtype, device=residual.device)
+    add_pending(residual, delta, None, out)
+    return out

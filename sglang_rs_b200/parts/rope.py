@@ -12,12 +12,16 @@ with d(t) = dims * ln(original / (2 pi t)) / (2 ln theta) (the pair whose wavele
 original context), lo = max(floor(d(fast)), 0), hi = min(ceil(d(slow)), dims - 1) and ramp_i = clamp((i - lo) /
 max(hi - lo, 0.001), 0, 1), pair i turns at f_i / factor * ramp_i + f_i * (1 - ramp_i); cosines and sines are
 multiplied by 0.1 ln(factor) + 1 (``magnitude``).
+
+:class:`RampScaling` stretches them by a rule of the wavelength w = 2 pi / f instead: f stays where w < original / high, becomes
+f / factor where w > original / low, and between the two, with s = (original / w - low) / (high - low), it is
+(1 - s) f / factor + s f; cosines and sines keep their size.
 """
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Callable, Optional
+from typing import Callable, Optional, Union
 
 import torch
 
@@ -64,13 +68,37 @@ class WavelengthScaling:
         return frequencies / self.factor * ramp + frequencies * (1.0 - ramp)
 
 
+@dataclass(frozen=True)
+class RampScaling:
+    """Stretching of the long wavelengths of a rotary table by a ramp over wavelengths (see the module's text)."""
+    factor: float
+    low: float               # waves that fit the original context fewer times than this are slowed by ``factor``
+    high: float              # waves that fit it more often than this keep their frequency
+    original: float          # positions of the original context
+
+    #: cosines and sines are left as they are
+    magnitude = 1.0
+
+    def __post_init__(self):
+        if not (self.factor > 0 and self.original > 0 and self.low > 0 and self.high >= self.low):
+            raise ValueError("rotary scaling needs a positive factor and context and 0 < low <= high")
+
+    def apply(self, frequencies: torch.Tensor, rotary_dim: int, theta: float) -> torch.Tensor:
+        """``frequencies`` float64 [rotary_dim / 2] -> the stretched ones."""
+        wave = 2.0 * math.pi / frequencies
+        s = torch.clamp((self.original / wave - self.low) / max(self.high - self.low, 1e-30), 0.0, 1.0)
+        between = (1.0 - s) * frequencies / self.factor + s * frequencies
+        slowed = torch.where(wave > self.original / self.low, frequencies / self.factor, between)
+        return torch.where(wave < self.original / self.high, frequencies, slowed)
+
+
 class RotaryEncoding(PositionEncoding):
     graph_safe = True
 
     fused = True
 
     def __init__(self, head_dim: int, theta: float, rotary_dim: Optional[int] = None, interleaved: bool = False,
-                 scaling: Optional[WavelengthScaling] = None):
+                 scaling: Union[WavelengthScaling, RampScaling, None] = None):
         self.head_dim = int(head_dim)
         self.scaling = scaling
         self.rotary_dim = int(rotary_dim if rotary_dim is not None else head_dim)
@@ -80,7 +108,7 @@ class RotaryEncoding(PositionEncoding):
             raise ValueError(f"rotary width {self.rotary_dim} must be even, positive and at most {self.head_dim}")
         if not self.theta > 0:
             raise ValueError("RoPE theta must be finite and positive")
-        if scaling is not None and not self.theta > 1:
+        if isinstance(scaling, WavelengthScaling) and not self.theta > 1:
             raise ValueError("rotary scaling needs a base above 1")
         self._table: Optional[FusedRotary] = None
 

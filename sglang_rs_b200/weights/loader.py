@@ -24,6 +24,7 @@ from typing import Dict, Mapping, Sequence, Tuple
 
 import torch
 
+from ..parts.base import FREE
 from .safetensors_io import read_model_dir
 
 
@@ -62,6 +63,12 @@ def stored_form(tensor: torch.Tensor) -> torch.Tensor:
     return tensor
 
 
+def shape_fits(expected: Sequence[int], found: Sequence[int]) -> bool:
+    """True if the shapes agree; a dimension of ``FREE`` takes any positive size."""
+    return len(expected) == len(found) and all(
+        have > 0 if want == FREE else want == have for want, have in zip(expected, found))
+
+
 def validate(expected: Mapping[str, Tuple[int, ...]], tensors: Mapping[str, torch.Tensor],
              ignored: Sequence[str] = ()) -> None:
     """``ignored``: shell-style patterns of tensor names that may be present and are not read."""
@@ -69,7 +76,7 @@ def validate(expected: Mapping[str, Tuple[int, ...]], tensors: Mapping[str, torc
     unexpected = [name for name in tensors if name not in expected
                   and not any(fnmatch.fnmatchcase(name, pattern) for pattern in ignored)]
     wrong = [(name, tuple(shape), tuple(tensors[name].shape)) for name, shape in expected.items()
-             if name in tensors and tuple(tensors[name].shape) != tuple(shape)]
+             if name in tensors and not shape_fits(shape, tensors[name].shape)]
     wrong_dtype = [(name, str(tensors[name].dtype)) for name in expected
                    if name in tensors and tensors[name].dtype in (torch.complex64, torch.complex128)]
     if missing or unexpected or wrong or wrong_dtype:

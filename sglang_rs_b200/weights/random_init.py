@@ -26,11 +26,11 @@ def random_tensor(name: str, spec: TensorSpec, seed: int, device="cpu", dtype: t
     generator = torch.Generator(device=device)
     generator.manual_seed((int(seed) * 1_000_003 + zlib.crc32(name.encode("utf-8"))) % (2 ** 63 - 1))
     if spec.init == "normal":
-        values = torch.randn(spec.shape, generator=generator, device=device, dtype=torch.float32) * NORMAL_STD
+        values = torch.randn(spec.sample_shape, generator=generator, device=device, dtype=torch.float32) * NORMAL_STD
     elif spec.init == "scale":
-        values = 1.0 + (torch.rand(spec.shape, generator=generator, device=device, dtype=torch.float32) * 2 - 1) * SCALE_SPREAD
+        values = 1.0 + (torch.rand(spec.sample_shape, generator=generator, device=device, dtype=torch.float32) * 2 - 1) * SCALE_SPREAD
     elif spec.init == "zeros":
-        values = torch.zeros(spec.shape, device=device, dtype=torch.float32)
+        values = torch.zeros(spec.sample_shape, device=device, dtype=torch.float32)
     else:
         raise ValueError(f"tensor {name}: unknown init {spec.init}")
     return values.to(dtype)
