@@ -159,7 +159,7 @@ def main() -> int:
     parser.add_argument("--warmup", type=int, default=3)
     parser.add_argument("--impl", default="ours", choices=("ours", "reference"))
     parser.add_argument("--shape", default="qwen3-8b", choices=sorted(SHAPES))
-    parser.add_argument("--mode", default="decode", choices=("decode", "prefill", "serve", "compare-cublas", "kernels", "ablate", "probe-overlap", "timeline", "gegepel", "tosivik", "desarax", "titatar"))
+    parser.add_argument("--mode", default="decode", choices=("decode", "prefill", "serve", "compare-cublas", "kernels", "ablate", "probe-overlap", "timeline", "gegepel", "tosivik", "desarax", "titatar", "sogodra"))
     parser.add_argument("--rows", default="1,8,64,2048", help="--mode compare-cublas: the row counts, comma-separated")
     parser.add_argument("--layers", type=int, default=None, help="fewer than the shape has, only where memory or time needs it")
     parser.add_argument("--batch", type=int, default=8)
@@ -172,7 +172,7 @@ def main() -> int:
     parser.add_argument("--requests", type=int, default=128, help="--mode serve: number of requests")
     parser.add_argument("--seed", type=int, default=0)
     parser.add_argument("--width", type=int, default=2048, choices=(1024, 2048, 4096),
-                        help="--mode tosivik and --mode desarax: the model's width; heads, feed-forwards and the shape beside it follow")
+                        help="--mode tosivik, --mode desarax and --mode sogodra: the model's width; heads, feed-forwards and the shape beside it follow")
     args = parser.parse_args()
 
     if args.impl == "reference":
@@ -193,6 +193,8 @@ def main() -> int:
         return desarax_beside_tosivik(args, warmup)
     if args.mode == "titatar":
         return titatar_beside_gegepel(args, warmup)
+    if args.mode == "sogodra":
+        return sogodra_beside_tosivik(args, warmup)
 
     if args.mode == "timeline":
         # the kernels of a decode step, built with marks that record when each block starts, stops waiting for the
@@ -942,6 +944,40 @@ def titatar_beside_gegepel(args, warmup) -> int:
     note = {"layers": layers, "width": GEGEPEL_WIDTH, "vocab": vocab, "titatar_layers": designs["titatar"]["layers"][:4],
             "gegepel_mixer": GEGEPEL_MIXER, "gegepel_mlp": GEGEPEL_MLP, "layer_runs": {"titatar": runs, "gegepel": runs}}
     return designs_side_by_side(args, warmup, "titatar", designs, vocab, note)
+
+
+def sogodra_layers(width: int, count: int):
+    """Layers of a real model's size at ``width``: the gated delta rule with heads of 128 over states of 128 x 128 and a convolution
+    over four tokens; beside it, in parallel layers, attention with four query heads per kv head, half of each head rotated with
+    stretched wavelengths and a window of 1,024 positions; minGRU as wide as the stream; a clamped feed-forward of three widths.
+    The kinds repeat as delta, parallel, minGRU, delta."""
+    heads = width // 128
+    rule = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4}
+    attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 1.0 / math.sqrt(128),
+                 "mask": {"size": 1024}, "rot": {"base": 50000.0, "dims": 64, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    dense = {"kind": "dense", "ff": 3 * width, "limit": 7.0}
+    kinds = [("delta", rule), ("parallel", {"left": attention, "right": rule, "left_scale": 0.8, "right_scale": 1.2}),
+             ("mingru", {"width": width}), ("delta", rule)]
+    return [{"type": kind, "mixer": mixer, "mlp": dense} for kind, mixer in (kinds[i % 4] for i in range(count))]
+
+
+def sogodra_beside_tosivik(args, warmup) -> int:
+    """``--mode sogodra``: prefill and decode of a Sogodra model with layers of a real model's size (random weights) beside a Tosivik
+    model of equal width and depth with dense feed-forwards of equal size and one copy of the stream (the closest design: linear
+    attention over a state per request beside softmax attention).  ``--width`` 1024, 2048 or 4096."""
+    layers = args.layers if args.layers is not None else 4
+    vocab = 32768
+    lightning, _, attention, _ = tosivik_layers(args.width, 4)
+    plain = [lightning, {**attention, "mlp": lightning["mlp"]}, lightning, lightning]
+    designs = {
+        "sogodra": {"architecture": "Sogodra", "vocab": vocab, "width": args.width, "norm": {"eps": 1e-5},
+                    "layers": sogodra_layers(args.width, layers)},
+        "tosivik": {"architecture": "Tosivik", "vocab": vocab, "width": args.width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5},
+                    "layers": [plain[i % 4] for i in range(layers)]},
+    }
+    note = {"layers": layers, "width": args.width, "vocab": vocab, "sogodra_layers": designs["sogodra"]["layers"][:4],
+            "tosivik_layers": designs["tosivik"]["layers"][:4]}
+    return designs_side_by_side(args, warmup, "sogodra", designs, vocab, note)
 
 
 def designs_side_by_side(args, warmup, mode, designs, vocab, note) -> int:

@@ -317,3 +317,811 @@ extern "C" int srb_delta_gate_norm(const float* o, const void* g, long long g_pi
   SRB_LAUNCH_CHECK("delta_gate_norm");
   return SRB_OK;
 }
+
+// ---- prompt portions in bfloat16: chunks of tokens on the tensor cores ---------------------------------------------------
+// The rows of every request are cut into chunks of DC_TOKENS (64) tokens (from the request's first row of the step).  Inside a
+// chunk that starts from state S and holds tokens 0 .. n-1, with c_t the sum of the logarithms of the decays up to t (a number,
+// or one per row of S; never positive, and never rising), k' and q' the unit vectors, and (k e^c) meaning entry by entry:
+//     L[t, j] = beta_t sum_d k'_t k'_j e^(c_t - c_j)   for j < t           A[t, j] = sum_d q'_t k'_j e^(c_t - c_j)   for j <= t
+//     (1 + L) U = beta (V - (K' e^c) S)                                    o_t = (q'_t e^(c_t)) S + sum_j A[t, j] u_j
+//     S <- e^(c_(n-1)) S + sum_j (k'_j e^(c_(n-1) - c_j)) u_j^T
+// so U = T beta V - W S with T = (1 + L)^-1 and W = T beta (K' e^c).  Every exponential is of a number that is not positive.
+// With a decay per row of S the sums behind L and A do not factor into e^(c_t) and e^(-c_j), which could overflow: they are taken
+// block by block of 16 tokens, the blocks left of the diagonal with both factors relative to c just before the row block (both
+// exponents are then not positive), the diagonal blocks pair by pair.  Two kernels:
+//   1. delta_chunk_prepare: per (chunk, head), in parallel: A, T, W, T beta V and the scaled q' and k'
+//   2. delta_chunk_walk: per (request, head, VS value columns) the chunks in order, S in registers: U, the results, the next S
+// x goes in as bfloat16 (what the convolution wrote); whatever is 32-bit by the design and has to be an operand of a product
+// goes in as the sum of two bfloat16 numbers, its rounding and the rounding of the rest (16 bits of mantissa), in two products,
+// or three where both operands are such sums; accumulation is 32-bit (mma.sync m16n8k16).
+// Heads of up to 128 entries (padded to 64 or 128 with zeros), widths that are multiples of eight.
+#include "mma_helpers.cuh"
+
+#define DC_TOKENS 64
+#define DC_PREPARE_THREADS 256
+#define DC_PAD 8
+#define DC_LOG2E 1.4426950408889634f
+#define DC_FASTEST -40.0f        // log2 of the smallest decay: below 2^-40 of a state nothing is left beside a 32-bit sum, and the
+                                 // sums of logarithms down a chunk, whose differences are taken, keep their last bits
+
+__device__ __forceinline__ unsigned dc_word(const __nv_bfloat16* p) { return *reinterpret_cast<const unsigned*>(p); }
+// (a, b) as two packed pairs: the roundings and the roundings of what they left
+__device__ __forceinline__ void dc_split2(float a, float b, unsigned& hi, unsigned& lo) {
+  hi = pack_bf16(a, b);
+  const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(&hi);
+  const float2 f = __bfloat1622float2(h);
+  lo = pack_bf16(a - f.x, b - f.y);
+}
+__device__ __forceinline__ float2 dc_pair(const __nv_bfloat16* p) {
+  return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+}
+
+// What kernel 1 hands to kernel 2, per (chunk, head); all pieces start on 16-byte borders.
+template <int DP, bool CHANNEL>
+struct DeltaChunkLayout {
+  static constexpr int ROWS = DC_TOKENS * DP * 2;                          // bytes of a [64][DP] operand
+  static constexpr int W = 0;                                              // -W: roundings, then the rest
+  static constexpr int Q = 2 * ROWS;                                       // CHANNEL: q' e^c, k' e^(c_last - c), each in two
+  static constexpr int K = Q + (CHANNEL ? 2 * ROWS : 0);
+  static constexpr int A = K + (CHANNEL ? 2 * ROWS : 0);                   // [64][64] in two
+  static constexpr int F = A + 2 * DC_TOKENS * DC_TOKENS * 2;              // floats: CHANNEL e^(c_last) [DP]; else q's and k's
+  static constexpr int FLOATS = CHANNEL ? DP : 2 * DC_TOKENS + 4;          // factors per token and e^(c_last)
+  static constexpr int V = F + FLOATS * 4;                                 // T beta V, transposed: float [vp][64]
+  static __host__ __device__ long long bytes(int vp) { return V + (long long)vp * DC_TOKENS * 4; }
+};
+
+// the request and the chunk of it that block `index` works on; false: there is no such chunk
+__device__ __forceinline__ bool dc_find(const DeltaArgs& a, int index, int& request, int& row0, int& n) {
+  int first = 0;
+  for (request = 0; request < a.requests; ++request) {
+    const int begin = a.cu_rows[request], rows = a.cu_rows[request + 1] - begin;
+    const int chunks = (rows + DC_TOKENS - 1) / DC_TOKENS;
+    if (index < first + chunks) {
+      row0 = begin + (index - first) * DC_TOKENS;
+      n = min(DC_TOKENS, begin + rows - row0);
+      return true;
+    }
+    first += chunks;
+  }
+  return false;
+}
+
+template <int DP, bool CHANNEL>
+struct DeltaPrepareSmem {
+  static constexpr int XP = DP + DC_PAD, CP = DP + 2, TP = DC_TOKENS + DC_PAD, LP = DC_TOKENS + 1;
+  static constexpr int K = 0;                                              // bfloat16 [64][XP]
+  static constexpr int Q = K + DC_TOKENS * XP * 2;                         // bfloat16 [64][XP]; later T scaled, in two [64][TP]
+  static constexpr int T_BYTES = 2 * DC_TOKENS * TP * 2;
+  static constexpr int QB = DC_TOKENS * XP * 2 > T_BYTES ? DC_TOKENS * XP * 2 : T_BYTES;
+  static constexpr int LT = Q + QB;                                        // L and T, float [64][LP] each; later k' e^c in two
+  static constexpr int LT_BYTES_A = 2 * DC_TOKENS * LP * 4, LT_BYTES_B = CHANNEL ? 2 * DC_TOKENS * XP * 2 : T_BYTES;
+  static constexpr int LT_BYTES = LT_BYTES_A > LT_BYTES_B ? LT_BYTES_A : LT_BYTES_B;
+  static constexpr int C = LT + LT_BYTES;                                  // CHANNEL: c, float [64][CP]; later v
+  static constexpr int C_BYTES = CHANNEL ? DC_TOKENS * CP * 4 : 0;
+  static constexpr int small(int vp) {
+    const int v = DC_TOKENS * (vp + DC_PAD) * 2;
+    return C + (C_BYTES > v ? C_BYTES : v);
+  }
+  static constexpr int SMALL_FLOATS = 4 * DC_TOKENS + 4 * DP + 16;          // per token: beta, 1/|k|, scale/|q|, c; totals
+  static constexpr int bytes(int vp) { return small(vp) + SMALL_FLOATS * 4; }
+};
+
+template <int DP, bool CHANNEL>
+__global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_kernel(DeltaArgs a, unsigned char* scratch, int vp) {
+  using M = DeltaPrepareSmem<DP, CHANNEL>;
+  using P = DeltaChunkLayout<DP, CHANNEL>;
+  constexpr int XP = M::XP, CP = M::CP, TP = M::TP, LP = M::LP, NTH = DC_PREPARE_THREADS;
+  extern __shared__ __align__(16) unsigned char dp_smem[];
+  __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(dp_smem + M::K);
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(dp_smem + M::Q);
+  float* ls = reinterpret_cast<float*>(dp_smem + M::LT);                   // [64][LP]
+  float* ts = ls + DC_TOKENS * LP;                                         // [64][LP]: A first, then T
+  float* cs = reinterpret_cast<float*>(dp_smem + M::C);                    // [64][CP], in units of log2 (CHANNEL)
+  float* beta_s = reinterpret_cast<float*>(dp_smem + M::small(vp));
+  float* ik_s = beta_s + DC_TOKENS;
+  float* iq_s = ik_s + DC_TOKENS;
+  float* cum_s = iq_s + DC_TOKENS;                                         // one decay per head: c, in units of log2
+  float* part_s = cum_s + DC_TOKENS;                                       // [4][DP]
+  srb_launch_dependents();
+  srb_grid_dependency_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int head = blockIdx.y, dim = a.dim, vdim = a.vdim;
+  int request, row0, n;
+  if (!dc_find(a, blockIdx.x, request, row0, n)) return;
+  const int qk_head = head / (a.heads / a.kv_heads);
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x) + (size_t)row0 * a.channels;
+  const __nv_bfloat16* beta = reinterpret_cast<const __nv_bfloat16*>(a.beta);
+  const __nv_bfloat16* decay = reinterpret_cast<const __nv_bfloat16*>(a.decay);
+  unsigned char* place = scratch + ((size_t)blockIdx.x * a.heads + head) * P::bytes(vp);
+
+  // q and k as they lie, zeros beyond the chunk's tokens and the head's entries
+  for (int i = tid; i < DC_TOKENS * DP / 8; i += NTH) {
+    const int t = i / (DP / 8), d = i % (DP / 8) * 8;
+    const bool live = t < n && d < dim;
+    const __nv_bfloat16* from = x + (size_t)(live ? t : 0) * a.channels + qk_head * dim + (live ? d : 0);
+    cp_async_16(qs + t * XP + d, from, live ? 16 : 0);
+    cp_async_16(ks + t * XP + d, from + a.kv_heads * dim, live ? 16 : 0);
+  }
+  cp_async_commit();
+  const float rate = expf(a.a_log[head]) * DC_LOG2E;
+  if (tid < DC_TOKENS) beta_s[tid] = tid < n ? delta_sigmoid(__bfloat162float(beta[(size_t)(row0 + tid) * a.beta_pitch + head])) : 0.f;
+  if (CHANNEL) {
+    // running sums down the tokens: a thread takes one row of the state for a part of the tokens, then adds the parts before
+    constexpr int PARTS = NTH / DP, PER = DC_TOKENS / PARTS;
+    const int d = tid % DP, part = tid / DP;
+    float sum = 0.f;
+    if (d < dim) {
+      const float bias = a.dt_bias[head * dim + d];
+      const __nv_bfloat16* from = decay + (size_t)row0 * a.decay_pitch + head * dim + d;
+      for (int t0 = part * PER; t0 < (part + 1) * PER; t0 += 8) {
+        float v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = t0 + j < n ? __bfloat162float(from[(size_t)(t0 + j) * a.decay_pitch]) : 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          if (t0 + j < n) sum += fmaxf(-rate * delta_softplus(v[j] + bias), DC_FASTEST);
+          cs[(t0 + j) * CP + d] = sum;
+        }
+      }
+    } else {
+      for (int t = part * PER; t < (part + 1) * PER; ++t) cs[t * CP + d] = 0.f;
+    }
+    part_s[part * DP + d] = sum;
+    __syncthreads();
+    float before = 0.f;
+    for (int p = 0; p < part; ++p) before += part_s[p * DP + d];
+    if (part)
+      for (int t = part * PER; t < (part + 1) * PER; ++t) cs[t * CP + d] += before;
+  } else if (warp == 0) {
+    float v0 = 0.f, v1 = 0.f;                              // a lane takes tokens 2 lane and 2 lane + 1
+    const float bias = a.dt_bias[head];
+    const int t = 2 * lane;
+    if (t < n) v0 = fmaxf(-rate * delta_softplus(__bfloat162float(decay[(size_t)(row0 + t) * a.decay_pitch + head]) + bias), DC_FASTEST);
+    if (t + 1 < n) v1 = fmaxf(-rate * delta_softplus(__bfloat162float(decay[(size_t)(row0 + t + 1) * a.decay_pitch + head]) + bias), DC_FASTEST);
+    float total = v0 + v1;
+#pragma unroll
+    for (int offset = 1; offset < 32; offset <<= 1) {
+      const float other = __shfl_up_sync(0xffffffffu, total, offset);
+      if (lane >= offset) total += other;
+    }
+    cum_s[t + 1] = total;
+    cum_s[t] = total - v1;
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  // lengths: a warp takes eight tokens
+  for (int t = warp * 8; t < warp * 8 + 8; ++t) {
+    float kk = 0.f, qq = 0.f;
+    for (int d = lane * 2; d < DP; d += 64) {
+      const float2 k = dc_pair(ks + t * XP + d), q = dc_pair(qs + t * XP + d);
+      kk = fmaf(k.x, k.x, fmaf(k.y, k.y, kk));
+      qq = fmaf(q.x, q.x, fmaf(q.y, q.y, qq));
+    }
+    kk = srb_warp_sum(kk);
+    qq = srb_warp_sum(qq);
+    if (lane == 0) {
+      ik_s[t] = 1.0f / sqrtf(kk + a.unit_eps);
+      iq_s[t] = a.q_scale / sqrtf(qq + a.unit_eps);
+    }
+  }
+  __syncthreads();
+
+  // ---- L and A.  Warps 0-3 take the rows of K, 4-7 those of Q, a block of 16 rows each
+  const int rb = warp & 3, kind = warp >> 2;
+  const int r0 = rb * 16 + g, r1 = r0 + 8;
+  const __nv_bfloat16* rows_s = kind ? qs : ks;
+  float* into = kind ? ts : ls;
+  if (!CHANNEL) {
+    float acc[8][4];
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
+#pragma unroll
+    for (int kk = 0; kk < DP / 16; ++kk) {
+      const int col = kk * 16 + 2 * t4;
+      unsigned ra[4] = {dc_word(rows_s + r0 * XP + col), dc_word(rows_s + r1 * XP + col), dc_word(rows_s + r0 * XP + col + 8),
+                        dc_word(rows_s + r1 * XP + col + 8)};
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt)
+        if (nt < 2 * rb + 2) {
+          const __nv_bfloat16* b = ks + (nt * 8 + g) * XP + col;
+          mma_bf16(acc[nt], ra, dc_word(b), dc_word(b + 8));
+        }
+    }
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+      if (nt < 2 * rb + 2) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int t = e < 2 ? r0 : r1, j = nt * 8 + 2 * t4 + (e & 1);
+          float v = 0.f;
+          if (j < t || (kind && j == t))
+            v = acc[nt][e] * (kind ? iq_s[t] : beta_s[t] * ik_s[t]) * ik_s[j] * exp2f(cum_s[t] - cum_s[j]);
+          into[t * LP + j] = v;
+        }
+      }
+  } else {
+    if (rb > 0) {
+      const float* ref = cs + (rb * 16 - 1) * CP;          // c just before the row block
+      float acc[6][4];
+#pragma unroll
+      for (int nt = 0; nt < 6; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
+      const float s0 = kind ? iq_s[r0] : beta_s[r0] * ik_s[r0], s1 = kind ? iq_s[r1] : beta_s[r1] * ik_s[r1];
+#pragma unroll 1
+      for (int kk = 0; kk < DP / 16; ++kk) {
+        const int d = kk * 16 + 2 * t4;
+        const float2 rlo = *reinterpret_cast<const float2*>(ref + d), rhi = *reinterpret_cast<const float2*>(ref + d + 8);
+        auto scaled = [&](const __nv_bfloat16* v, const float* c, float2 from, float sign, float scale) -> float2 {
+          const float2 x2 = dc_pair(v), c2 = *reinterpret_cast<const float2*>(c);
+          return make_float2(x2.x * scale * exp2f(sign * (c2.x - from.x)), x2.y * scale * exp2f(sign * (c2.y - from.y)));
+        };
+        unsigned hi[4], lo[4];
+        float2 v;
+        v = scaled(rows_s + r0 * XP + d, cs + r0 * CP + d, rlo, 1.f, s0);          dc_split2(v.x, v.y, hi[0], lo[0]);
+        v = scaled(rows_s + r1 * XP + d, cs + r1 * CP + d, rlo, 1.f, s1);          dc_split2(v.x, v.y, hi[1], lo[1]);
+        v = scaled(rows_s + r0 * XP + d + 8, cs + r0 * CP + d + 8, rhi, 1.f, s0);  dc_split2(v.x, v.y, hi[2], lo[2]);
+        v = scaled(rows_s + r1 * XP + d + 8, cs + r1 * CP + d + 8, rhi, 1.f, s1);  dc_split2(v.x, v.y, hi[3], lo[3]);
+#pragma unroll
+        for (int nt = 0; nt < 6; ++nt)
+          if (nt < 2 * rb) {
+            const int j = nt * 8 + g;
+            unsigned bh[2], bl[2];
+            v = scaled(ks + j * XP + d, cs + j * CP + d, rlo, -1.f, ik_s[j]);          dc_split2(v.x, v.y, bh[0], bl[0]);
+            v = scaled(ks + j * XP + d + 8, cs + j * CP + d + 8, rhi, -1.f, ik_s[j]);  dc_split2(v.x, v.y, bh[1], bl[1]);
+            mma_bf16(acc[nt], hi, bh[0], bh[1]);
+            mma_bf16(acc[nt], hi, bl[0], bl[1]);
+            mma_bf16(acc[nt], lo, bh[0], bh[1]);
+          }
+      }
+#pragma unroll
+      for (int nt = 0; nt < 6; ++nt)
+        if (nt < 2 * rb) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) into[(e < 2 ? r0 : r1) * LP + nt * 8 + 2 * t4 + (e & 1)] = acc[nt][e];
+        }
+    }
+    // the diagonal blocks, pair by pair (t >= j): 136 pairs in each of the four
+    for (int item = tid; item < 4 * 136; item += NTH) {
+      const int block = item / 136, pair = item - block * 136;
+      int t = (int)((sqrtf(8.0f * pair + 1.0f) - 1.0f) * 0.5f);
+      while ((t + 1) * (t + 2) / 2 <= pair) ++t;           // (the root may be off by one)
+      while (t * (t + 1) / 2 > pair) --t;
+      const int j = block * 16 + pair - t * (t + 1) / 2;
+      t += block * 16;
+      float kk = 0.f, qk = 0.f;
+      for (int d = 0; d < DP; d += 2) {
+        const float2 ct = *reinterpret_cast<const float2*>(cs + t * CP + d), cj = *reinterpret_cast<const float2*>(cs + j * CP + d);
+        const float2 kj = dc_pair(ks + j * XP + d), kt = dc_pair(ks + t * XP + d), qt = dc_pair(qs + t * XP + d);
+        const float e0 = kj.x * exp2f(ct.x - cj.x), e1 = kj.y * exp2f(ct.y - cj.y);
+        kk = fmaf(kt.x, e0, fmaf(kt.y, e1, kk));
+        qk = fmaf(qt.x, e0, fmaf(qt.y, e1, qk));
+      }
+      ls[t * LP + j] = j < t ? kk * beta_s[t] * ik_s[t] * ik_s[j] : 0.f;
+      ts[t * LP + j] = qk * iq_s[t] * ik_s[j];
+    }
+  }
+  __syncthreads();
+
+  // ---- A leaves in two; so do the scaled q' and k' (CHANNEL) or their factors
+  {
+    __nv_bfloat16* ah = reinterpret_cast<__nv_bfloat16*>(place + P::A);
+    __nv_bfloat16* al = ah + DC_TOKENS * DC_TOKENS;
+    for (int i = tid; i < DC_TOKENS * DC_TOKENS / 2; i += NTH) {
+      const int t = i / (DC_TOKENS / 2), j = i % (DC_TOKENS / 2) * 2;
+      unsigned hi, lo;
+      dc_split2(j <= t ? ts[t * LP + j] : 0.f, j + 1 <= t ? ts[t * LP + j + 1] : 0.f, hi, lo);
+      *reinterpret_cast<unsigned*>(ah + t * DC_TOKENS + j) = hi;
+      *reinterpret_cast<unsigned*>(al + t * DC_TOKENS + j) = lo;
+    }
+  }
+  float* factors = reinterpret_cast<float*>(place + P::F);
+  if (CHANNEL) {
+    __nv_bfloat16* qh = reinterpret_cast<__nv_bfloat16*>(place + P::Q);
+    __nv_bfloat16* kh = reinterpret_cast<__nv_bfloat16*>(place + P::K);
+    const float* last = cs + (DC_TOKENS - 1) * CP;
+    for (int i = tid; i < DC_TOKENS * DP / 2; i += NTH) {
+      const int t = i / (DP / 2), d = i % (DP / 2) * 2;
+      const float2 c = *reinterpret_cast<const float2*>(cs + t * CP + d), end = *reinterpret_cast<const float2*>(last + d);
+      const float2 q = dc_pair(qs + t * XP + d), k = dc_pair(ks + t * XP + d);
+      unsigned hi, lo;
+      dc_split2(q.x * iq_s[t] * exp2f(c.x), q.y * iq_s[t] * exp2f(c.y), hi, lo);
+      *reinterpret_cast<unsigned*>(qh + t * DP + d) = hi;
+      *reinterpret_cast<unsigned*>(qh + DC_TOKENS * DP + t * DP + d) = lo;
+      dc_split2(k.x * ik_s[t] * exp2f(end.x - c.x), k.y * ik_s[t] * exp2f(end.y - c.y), hi, lo);
+      *reinterpret_cast<unsigned*>(kh + t * DP + d) = hi;
+      *reinterpret_cast<unsigned*>(kh + DC_TOKENS * DP + t * DP + d) = lo;
+    }
+    for (int d = tid; d < DP; d += NTH) factors[d] = exp2f(last[d]);
+  } else if (tid < DC_TOKENS) {
+    factors[tid] = iq_s[tid] * exp2f(cum_s[tid]);
+    factors[DC_TOKENS + tid] = ik_s[tid] * exp2f(cum_s[DC_TOKENS - 1] - cum_s[tid]);
+    if (tid == 0) factors[2 * DC_TOKENS] = exp2f(cum_s[DC_TOKENS - 1]);
+  }
+  __syncthreads();
+
+  // ---- T = (1 + L)^-1: the four diagonal blocks by forward substitution (a lane takes a column), then the blocks below them
+  if (warp < 4 && lane < 16) {
+    const int b = warp * 16;
+    float col[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      float v = i == lane ? 1.f : 0.f;
+#pragma unroll
+      for (int m = 0; m < 16; ++m)
+        if (m < i) v = fmaf(-ls[(b + i) * LP + b + m], col[m], v);
+      col[i] = v;
+    }
+#pragma unroll
+    for (int i = 0; i < 16; ++i) ts[(b + i) * LP + b + lane] = col[i];
+  }
+  __syncthreads();
+  {
+    const int i = tid >> 4, j = tid & 15;                  // an entry of a 16 x 16 block
+    for (int gap = 1; gap < 4; ++gap) {
+      // P = sum over the blocks between of L T, kept where the result goes; then T_ii P.  (the places are not read before)
+      for (int cb = 0; cb + gap < 4; ++cb) {
+        const int b = (cb + gap) * 16, c = cb * 16;
+        float v = 0.f;
+        for (int m = c; m < b; ++m) v = fmaf(ls[(b + i) * LP + m], ts[m * LP + c + j], v);
+        ts[(b + i) * LP + c + j] = v;
+      }
+      __syncthreads();
+      float v[3];
+#pragma unroll
+      for (int cb = 0; cb < 3; ++cb)
+        if (cb + gap < 4) {
+          const int b = (cb + gap) * 16, c = cb * 16;
+          v[cb] = 0.f;
+          for (int m = 0; m <= i; ++m) v[cb] = fmaf(-ts[(b + i) * LP + b + m], ts[(b + m) * LP + c + j], v[cb]);
+        }
+      __syncthreads();
+#pragma unroll
+      for (int cb = 0; cb < 3; ++cb)
+        if (cb + gap < 4) ts[((cb + gap) * 16 + i) * LP + cb * 16 + j] = v[cb];
+      __syncthreads();
+    }
+  }
+  // ---- T with its columns scaled, in two: times beta (for V), and without channels times beta |k|^-1 e^c (for K as it lies)
+  __nv_bfloat16* th = qs;                                  // [64][TP], then the rest
+  __nv_bfloat16* tl = th + DC_TOKENS * TP;
+  for (int i = tid; i < DC_TOKENS * DC_TOKENS / 2; i += NTH) {
+    const int t = i / (DC_TOKENS / 2), j = i % (DC_TOKENS / 2) * 2;
+    unsigned hi, lo;
+    dc_split2(j <= t ? ts[t * LP + j] * beta_s[j] : 0.f, j + 1 <= t ? ts[t * LP + j + 1] * beta_s[j + 1] : 0.f, hi, lo);
+    *reinterpret_cast<unsigned*>(th + t * TP + j) = hi;
+    *reinterpret_cast<unsigned*>(tl + t * TP + j) = lo;
+  }
+  __syncthreads();
+  __nv_bfloat16* second = reinterpret_cast<__nv_bfloat16*>(dp_smem + M::LT);
+  if (CHANNEL) {
+    // k' e^c in two, over L and T
+    for (int i = tid; i < DC_TOKENS * DP / 2; i += NTH) {
+      const int t = i / (DP / 2), d = i % (DP / 2) * 2;
+      const float2 c = *reinterpret_cast<const float2*>(cs + t * CP + d), k = dc_pair(ks + t * XP + d);
+      unsigned hi, lo;
+      dc_split2(k.x * ik_s[t] * exp2f(c.x), k.y * ik_s[t] * exp2f(c.y), hi, lo);
+      *reinterpret_cast<unsigned*>(second + t * XP + d) = hi;
+      *reinterpret_cast<unsigned*>(second + DC_TOKENS * XP + t * XP + d) = lo;
+    }
+  } else {
+    // T once more, its columns scaled for K (from the scaled copy: T itself lies where this goes)
+    for (int i = tid; i < DC_TOKENS * DC_TOKENS / 2; i += NTH) {
+      const int t = i / (DC_TOKENS / 2), j = i % (DC_TOKENS / 2) * 2;
+      const float2 h = dc_pair(th + t * TP + j), l = dc_pair(tl + t * TP + j);
+      unsigned hi, lo;
+      dc_split2((h.x + l.x) * ik_s[j] * exp2f(cum_s[j]), (h.y + l.y) * ik_s[j + 1] * exp2f(cum_s[j + 1]), hi, lo);
+      *reinterpret_cast<unsigned*>(second + t * TP + j) = hi;
+      *reinterpret_cast<unsigned*>(second + DC_TOKENS * TP + t * TP + j) = lo;
+    }
+  }
+  __syncthreads();
+  // ---- v over c
+  const int VP = vp + DC_PAD;
+  __nv_bfloat16* vs = reinterpret_cast<__nv_bfloat16*>(cs);
+  for (int i = tid; i < DC_TOKENS * vp / 8; i += NTH) {
+    const int t = i / (vp / 8), c = i % (vp / 8) * 8;
+    const bool live = t < n && c < vdim;
+    cp_async_16(vs + t * VP + c, x + (size_t)(live ? t : 0) * a.channels + 2 * a.kv_heads * dim + head * vdim + (live ? c : 0), live ? 16 : 0);
+  }
+  cp_async_commit();
+
+  // ---- -W [64][DP]: warps take 16 tokens and half of the columns
+  {
+    constexpr int NT = DP / 16;
+    float acc[NT][4];
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
+    const __nv_bfloat16* lh = CHANNEL ? th : second;
+    const __nv_bfloat16* ll = CHANNEL ? tl : second + DC_TOKENS * TP;
+    const int matrix = lane >> 3, inner = lane & 7;
+#pragma unroll
+    for (int kk = 0; kk < DC_TOKENS / 16; ++kk) {
+      if (kk > rb) break;                                  // T is zero above the diagonal
+      unsigned hi[4], lo[4];
+      const int at = (rb * 16 + (matrix & 1) * 8 + inner) * TP + kk * 16 + (matrix >> 1) * 8;
+      ldmatrix_x4(hi[0], hi[1], hi[2], hi[3], lh + at);
+      ldmatrix_x4(lo[0], lo[1], lo[2], lo[3], ll + at);
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        const int d = kind * (DP / 2) + nt * 8;
+        if (CHANNEL) {
+          unsigned b0, b1, b2, b3;
+          ldmatrix_x4_trans(b0, b1, b2, b3, second + (matrix >> 1) * DC_TOKENS * XP + (kk * 16 + (matrix & 1) * 8 + inner) * XP + d);
+          mma_bf16(acc[nt], hi, b0, b1);
+          mma_bf16(acc[nt], hi, b2, b3);
+          mma_bf16(acc[nt], lo, b0, b1);
+        } else {
+          if (nt & 1) continue;                            // two tiles of eight columns at a time
+          unsigned b0, b1, b2, b3;
+          ldmatrix_x4_trans(b0, b1, b2, b3, ks + (kk * 16 + (matrix & 1) * 8 + inner) * XP + d + (matrix >> 1) * 8);
+          mma_bf16(acc[nt], hi, b0, b1);
+          mma_bf16(acc[nt], lo, b0, b1);
+          mma_bf16(acc[nt + 1], hi, b2, b3);
+          mma_bf16(acc[nt + 1], lo, b2, b3);
+        }
+      }
+    }
+    __nv_bfloat16* wh = reinterpret_cast<__nv_bfloat16*>(place + P::W);
+    __nv_bfloat16* wl = wh + DC_TOKENS * DP;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      const int d = kind * (DP / 2) + nt * 8 + 2 * t4;
+      unsigned hi, lo;
+      dc_split2(-acc[nt][0], -acc[nt][1], hi, lo);
+      *reinterpret_cast<unsigned*>(wh + r0 * DP + d) = hi;
+      *reinterpret_cast<unsigned*>(wl + r0 * DP + d) = lo;
+      dc_split2(-acc[nt][2], -acc[nt][3], hi, lo);
+      *reinterpret_cast<unsigned*>(wh + r1 * DP + d) = hi;
+      *reinterpret_cast<unsigned*>(wl + r1 * DP + d) = lo;
+    }
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  // ---- (T beta V)^T [vp][64]: a warp takes 16 value columns at a time; the left operand is V read across its rows
+  {
+    float* vt = reinterpret_cast<float*>(place + P::V);
+    const int matrix = lane >> 3, inner = lane & 7;
+    for (int c0 = warp * 16; c0 < vp; c0 += 8 * 16) {
+      float acc[8][4];
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
+#pragma unroll
+      for (int kk = 0; kk < DC_TOKENS / 16; ++kk) {
+        unsigned va[4];                                    // rows: value columns, inner index: tokens
+        ldmatrix_x4_trans(va[0], va[1], va[2], va[3], vs + (kk * 16 + (matrix >> 1) * 8 + inner) * VP + c0 + (matrix & 1) * 8);
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt) {
+          if (nt < 2 * kk) continue;                       // tokens before these give nothing
+          unsigned b0, b1, b2, b3;
+          ldmatrix_x4(b0, b1, b2, b3, th + (matrix >> 1) * DC_TOKENS * TP + (nt * 8 + inner) * TP + kk * 16 + (matrix & 1) * 8);
+          mma_bf16(acc[nt], va, b0, b1);
+          mma_bf16(acc[nt], va, b2, b3);
+        }
+      }
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) {
+        *reinterpret_cast<float2*>(vt + (c0 + g) * DC_TOKENS + nt * 8 + 2 * t4) = make_float2(acc[nt][0], acc[nt][1]);
+        *reinterpret_cast<float2*>(vt + (c0 + g + 8) * DC_TOKENS + nt * 8 + 2 * t4) = make_float2(acc[nt][2], acc[nt][3]);
+      }
+    }
+  }
+}
+
+// MT: tiles of 16 value columns per block; four warps per tile share the tokens (U, results) and the rows of S (next S).
+template <int DP, bool CHANNEL, int MT>
+struct DeltaWalkSmem {
+  static constexpr int XP = DP + DC_PAD, TP = DC_TOKENS + DC_PAD, VS = 16 * MT, QK = CHANNEL ? 2 : 1;
+  static constexpr int ROWS = DC_TOKENS * XP * 2;
+  static constexpr int W = 0, Q = W + 2 * ROWS, K = Q + QK * ROWS, A = K + QK * ROWS, A_HALF = DC_TOKENS * TP * 2;
+  static constexpr int S = A + 2 * A_HALF, S_HALF = VS * XP * 2;
+  static constexpr int U = S + 2 * S_HALF, U_HALF = VS * TP * 2;           // U in two; without channels also U times k's factors
+  static constexpr int F = U + (CHANNEL ? 2 : 4) * U_HALF;
+  static constexpr int BYTES = F + (CHANNEL ? DP : 2 * DC_TOKENS + 4) * 4;
+};
+
+template <int DP, bool CHANNEL, int MT>
+__global__ void __launch_bounds__(128 * MT) delta_chunk_walk_kernel(DeltaArgs a, const unsigned char* scratch, int vp) {
+  using M = DeltaWalkSmem<DP, CHANNEL, MT>;
+  using P = DeltaChunkLayout<DP, CHANNEL>;
+  constexpr int XP = M::XP, TP = M::TP, NTH = 128 * MT, DT = DP / 32;      // DT: tiles of eight rows of S that a warp owns
+  extern __shared__ __align__(16) unsigned char dw_smem[];
+  __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(dw_smem + M::W);
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(dw_smem + M::Q);
+  __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(dw_smem + M::K);
+  __nv_bfloat16* as = reinterpret_cast<__nv_bfloat16*>(dw_smem + M::A);
+  __nv_bfloat16* ss = reinterpret_cast<__nv_bfloat16*>(dw_smem + M::S);
+  __nv_bfloat16* us = reinterpret_cast<__nv_bfloat16*>(dw_smem + M::U);
+  float* fs = reinterpret_cast<float*>(dw_smem + M::F);
+  srb_launch_dependents();
+  srb_grid_dependency_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int tile = warp >> 2, part = warp & 3, matrix = lane >> 3, inner = lane & 7;
+  const int head = blockIdx.y, request = blockIdx.z, dim = a.dim, vdim = a.vdim;
+  const int begin = a.cu_rows[request], rows = a.cu_rows[request + 1] - begin;
+  if (rows <= 0) return;
+  const int start = a.positions[begin];
+  if (start < 0) return;
+  int first = 0;
+  for (int r = 0; r < request; ++r) first += (a.cu_rows[r + 1] - a.cu_rows[r] + DC_TOKENS - 1) / DC_TOKENS;
+  const int chunks = (rows + DC_TOKENS - 1) / DC_TOKENS;
+  const int c_tile = blockIdx.x * M::VS + tile * 16;                       // the warp's value columns: c_tile + g, c_tile + g + 8
+  const int c_lo = c_tile + g, c_hi = c_lo + 8;
+  const int qk_head = head / (a.heads / a.kv_heads);
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x);
+  float* state = a.state + (size_t)a.state_slots[request] * a.slot_floats + a.conv_floats + (size_t)head * vdim * dim;
+
+  // the warp's part of S^T: columns c_lo, c_hi, rows d = part * DP / 4 + nt * 8 + 2 t4, + 1
+  float s[DT][4];
+#pragma unroll
+  for (int nt = 0; nt < DT; ++nt) {
+    const int d = part * (DP / 4) + nt * 8 + 2 * t4;
+    s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+    if (start > 0 && d < dim) {                            // (dim is even)
+      if (c_lo < vdim) { const float2 v = *reinterpret_cast<const float2*>(state + (size_t)c_lo * dim + d); s[nt][0] = v.x; s[nt][1] = v.y; }
+      if (c_hi < vdim) { const float2 v = *reinterpret_cast<const float2*>(state + (size_t)c_hi * dim + d); s[nt][2] = v.x; s[nt][3] = v.y; }
+    }
+  }
+  auto place_of = [&](int chunk) { return scratch + ((size_t)(first + chunk) * a.heads + head) * P::bytes(vp); };
+  auto keep_state = [&]() {
+#pragma unroll
+    for (int nt = 0; nt < DT; ++nt) {
+      const int d = part * (DP / 4) + nt * 8 + 2 * t4;
+      unsigned hi, lo;
+      dc_split2(s[nt][0], s[nt][1], hi, lo);
+      __nv_bfloat16* at = ss + (tile * 16 + g) * XP + d;
+      *reinterpret_cast<unsigned*>(at) = hi;
+      *reinterpret_cast<unsigned*>(at + M::S_HALF / 2) = lo;
+      dc_split2(s[nt][2], s[nt][3], hi, lo);
+      *reinterpret_cast<unsigned*>(at + 8 * XP) = hi;
+      *reinterpret_cast<unsigned*>(at + 8 * XP + M::S_HALF / 2) = lo;
+    }
+  };
+  auto fetch_rows = [&](__nv_bfloat16* to, const unsigned char* from, int halves) {      // operands in two: [halves * 64][DP]
+    for (int i = tid; i < halves * DC_TOKENS * DP / 8; i += NTH) {
+      const int t = i / (DP / 8), d = i % (DP / 8) * 8;
+      cp_async_16(to + t * XP + d, from + (size_t)i * 16, 16);
+    }
+  };
+  auto fetch_x = [&](__nv_bfloat16* to, int column, int chunk) {                         // q or k as they lie
+    for (int i = tid; i < DC_TOKENS * DP / 8; i += NTH) {
+      const int t = i / (DP / 8), d = i % (DP / 8) * 8;
+      const bool live = chunk * DC_TOKENS + t < rows && d < dim;
+      cp_async_16(to + t * XP + d, x + (size_t)(begin + (live ? chunk * DC_TOKENS + t : 0)) * a.channels + column + (live ? d : 0), live ? 16 : 0);
+    }
+  };
+  auto fetch_wq = [&](int chunk) {
+    const unsigned char* place = place_of(chunk);
+    fetch_rows(ws, place + P::W, 2);
+    if (CHANNEL) fetch_rows(qs, place + P::Q, 2); else fetch_x(qs, qk_head * dim, chunk);
+    cp_async_commit();
+  };
+  auto fetch_ak = [&](int chunk) {
+    const unsigned char* place = place_of(chunk);
+    for (int i = tid; i < 2 * DC_TOKENS * DC_TOKENS / 8; i += NTH) {
+      const int t = i / (DC_TOKENS / 8), j = i % (DC_TOKENS / 8) * 8;
+      cp_async_16(as + t * TP + j, place + P::A + (size_t)i * 16, 16);
+    }
+    if (CHANNEL) fetch_rows(ks, place + P::K, 2); else fetch_x(ks, (a.kv_heads + qk_head) * dim, chunk);
+    for (int i = tid; i < P::FLOATS / 4; i += NTH) cp_async_16(fs + i * 4, place + P::F + (size_t)i * 16, 16);
+    cp_async_commit();
+  };
+  float uv[2][4];                                          // the warp's 16 tokens of T beta V, for the chunk to come
+  auto fetch_v = [&](int chunk) {
+    const float* vt = reinterpret_cast<const float*>(place_of(chunk) + P::V);
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      const int t = part * 16 + nt * 8 + 2 * t4;
+      float2 lo = make_float2(0.f, 0.f), hi = lo;
+      if (c_lo < vp) lo = *reinterpret_cast<const float2*>(vt + (size_t)c_lo * DC_TOKENS + t);
+      if (c_hi < vp) hi = *reinterpret_cast<const float2*>(vt + (size_t)c_hi * DC_TOKENS + t);
+      uv[nt][0] = lo.x; uv[nt][1] = lo.y; uv[nt][2] = hi.x; uv[nt][3] = hi.y;
+    }
+  };
+  fetch_wq(0);
+  fetch_v(0);
+  keep_state();
+  for (int chunk = 0; chunk < chunks; ++chunk) {
+    cp_async_wait<0>();
+    __syncthreads();                                       // W, q and the state are there; A, k and U are no longer read
+    fetch_ak(chunk);
+    float u[2][4], o[2][4];
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { u[nt][e] = uv[nt][e]; o[nt][e] = 0.f; }
+    // U = T beta V - W S and (q e^c) S for the warp's 16 tokens
+#pragma unroll 2
+    for (int kk = 0; kk < DP / 16; ++kk) {
+      unsigned sh[4], sl[4];
+      const __nv_bfloat16* at = ss + (tile * 16 + (matrix & 1) * 8 + inner) * XP + kk * 16 + (matrix >> 1) * 8;
+      ldmatrix_x4(sh[0], sh[1], sh[2], sh[3], at);
+      ldmatrix_x4(sl[0], sl[1], sl[2], sl[3], at + M::S_HALF / 2);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) {
+        unsigned b0, b1, b2, b3;
+        const int row = part * 16 + nt * 8 + inner;
+        ldmatrix_x4(b0, b1, b2, b3, ws + (matrix >> 1) * DC_TOKENS * XP + row * XP + kk * 16 + (matrix & 1) * 8);
+        mma_bf16(u[nt], sh, b0, b1);
+        mma_bf16(u[nt], sh, b2, b3);
+        mma_bf16(u[nt], sl, b0, b1);
+      }
+      if (CHANNEL) {
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          unsigned b0, b1, b2, b3;
+          const int row = part * 16 + nt * 8 + inner;
+          ldmatrix_x4(b0, b1, b2, b3, qs + (matrix >> 1) * DC_TOKENS * XP + row * XP + kk * 16 + (matrix & 1) * 8);
+          mma_bf16(o[nt], sh, b0, b1);
+          mma_bf16(o[nt], sh, b2, b3);
+          mma_bf16(o[nt], sl, b0, b1);
+        }
+      } else {
+        unsigned b0, b1, b2, b3;                           // both tiles of eight tokens at once
+        ldmatrix_x4(b0, b1, b2, b3, qs + (part * 16 + (matrix >> 1) * 8 + inner) * XP + kk * 16 + (matrix & 1) * 8);
+        mma_bf16(o[0], sh, b0, b1);
+        mma_bf16(o[0], sl, b0, b1);
+        mma_bf16(o[1], sh, b2, b3);
+        mma_bf16(o[1], sl, b2, b3);
+      }
+    }
+    cp_async_wait<0>();                                    // A, k and the factors (each thread its own copies; the barrier below joins them)
+    if (!CHANNEL) __syncthreads();                         // the factors are read below by every thread
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      const int t = part * 16 + nt * 8 + 2 * t4;
+      unsigned hi, lo;
+      __nv_bfloat16* at = us + (tile * 16 + g) * TP + t;
+      dc_split2(u[nt][0], u[nt][1], hi, lo);
+      *reinterpret_cast<unsigned*>(at) = hi;
+      *reinterpret_cast<unsigned*>(at + M::U_HALF / 2) = lo;
+      dc_split2(u[nt][2], u[nt][3], hi, lo);
+      *reinterpret_cast<unsigned*>(at + 8 * TP) = hi;
+      *reinterpret_cast<unsigned*>(at + 8 * TP + M::U_HALF / 2) = lo;
+      if (!CHANNEL) {
+        const float k0 = fs[DC_TOKENS + t], k1 = fs[DC_TOKENS + t + 1];
+        at += M::U_HALF;                                   // U times k's factors, behind the two halves of U
+        dc_split2(u[nt][0] * k0, u[nt][1] * k1, hi, lo);
+        *reinterpret_cast<unsigned*>(at) = hi;
+        *reinterpret_cast<unsigned*>(at + M::U_HALF / 2) = lo;
+        dc_split2(u[nt][2] * k0, u[nt][3] * k1, hi, lo);
+        *reinterpret_cast<unsigned*>(at + 8 * TP) = hi;
+        *reinterpret_cast<unsigned*>(at + 8 * TP + M::U_HALF / 2) = lo;
+        const float q0 = fs[t], q1 = fs[t + 1];
+        o[nt][0] *= q0; o[nt][1] *= q1; o[nt][2] *= q0; o[nt][3] *= q1;
+      }
+    }
+    __syncthreads();                                       // U, A, k are there; W, q and the state before are no longer read
+    if (chunk + 1 < chunks) {
+      fetch_wq(chunk + 1);
+      fetch_v(chunk + 1);
+    }
+    // the next S: the decay, then U^T k over the chunk's tokens
+    const float whole = CHANNEL ? 1.f : fs[2 * DC_TOKENS];
+#pragma unroll
+    for (int nt = 0; nt < DT; ++nt) {
+      float e0 = whole, e1 = whole;
+      if (CHANNEL) { const int d = part * (DP / 4) + nt * 8 + 2 * t4; e0 = fs[d]; e1 = fs[d + 1]; }
+      s[nt][0] *= e0; s[nt][1] *= e1; s[nt][2] *= e0; s[nt][3] *= e1;
+    }
+#pragma unroll
+    for (int kk = 0; kk < DC_TOKENS / 16; ++kk) {
+      const __nv_bfloat16* at = us + (tile * 16 + (matrix & 1) * 8 + inner) * TP + kk * 16 + (matrix >> 1) * 8;
+      unsigned uh[4], ul[4];
+      ldmatrix_x4(uh[0], uh[1], uh[2], uh[3], at);
+      ldmatrix_x4(ul[0], ul[1], ul[2], ul[3], at + M::U_HALF / 2);
+      if (kk <= part) {                                    // A is zero above the diagonal
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          unsigned b0, b1, b2, b3;
+          ldmatrix_x4(b0, b1, b2, b3, as + (matrix >> 1) * DC_TOKENS * TP + (part * 16 + nt * 8 + inner) * TP + kk * 16 + (matrix & 1) * 8);
+          mma_bf16(o[nt], uh, b0, b1);
+          mma_bf16(o[nt], uh, b2, b3);
+          mma_bf16(o[nt], ul, b0, b1);
+        }
+      }
+      if (!CHANNEL) {
+        ldmatrix_x4(uh[0], uh[1], uh[2], uh[3], at + M::U_HALF);
+        ldmatrix_x4(ul[0], ul[1], ul[2], ul[3], at + M::U_HALF + M::U_HALF / 2);
+      }
+      if (CHANNEL) {
+#pragma unroll
+        for (int nt = 0; nt < DT; ++nt) {
+          unsigned b0, b1, b2, b3;
+          const int d = part * (DP / 4) + nt * 8;
+          ldmatrix_x4_trans(b0, b1, b2, b3, ks + (matrix >> 1) * DC_TOKENS * XP + (kk * 16 + (matrix & 1) * 8 + inner) * XP + d);
+          mma_bf16(s[nt], uh, b0, b1);
+          mma_bf16(s[nt], uh, b2, b3);
+          mma_bf16(s[nt], ul, b0, b1);
+        }
+      } else {
+#pragma unroll
+        for (int nt = 0; nt < DT; nt += 2) {
+          unsigned b0, b1, b2, b3;
+          const int d = part * (DP / 4) + nt * 8;
+          ldmatrix_x4_trans(b0, b1, b2, b3, ks + (kk * 16 + (matrix & 1) * 8 + inner) * XP + d + (matrix >> 1) * 8);
+          mma_bf16(s[nt], uh, b0, b1);
+          mma_bf16(s[nt], ul, b0, b1);
+          mma_bf16(s[nt + 1], uh, b2, b3);
+          mma_bf16(s[nt + 1], ul, b2, b3);
+        }
+      }
+    }
+    if (chunk + 1 < chunks) keep_state();
+    const int left = rows - chunk * DC_TOKENS;
+    float* out = a.out + (size_t)(begin + chunk * DC_TOKENS) * a.heads * vdim + (size_t)head * vdim;
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      const int t = part * 16 + nt * 8 + 2 * t4;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int token = t + (e & 1), c = e < 2 ? c_lo : c_hi;
+        if (token < left && c < vdim) out[(size_t)token * a.heads * vdim + c] = o[nt][e];
+      }
+    }
+  }
+  if (!a.write_state) return;
+#pragma unroll
+  for (int nt = 0; nt < DT; ++nt) {
+    const int d = part * (DP / 4) + nt * 8 + 2 * t4;
+    if (d >= dim) continue;
+    if (c_lo < vdim) *reinterpret_cast<float2*>(state + (size_t)c_lo * dim + d) = make_float2(s[nt][0], s[nt][1]);
+    if (c_hi < vdim) *reinterpret_cast<float2*>(state + (size_t)c_hi * dim + d) = make_float2(s[nt][2], s[nt][3]);
+  }
+}
+
+static int delta_padded_columns(int vdim) { return (vdim + 15) / 16 * 16; }
+
+template <int DP, bool CHANNEL>
+static int launch_delta_chunks(const DeltaArgs& a, unsigned char* scratch, int chunks, cudaStream_t s) {
+  const int vp = delta_padded_columns(a.vdim);
+  const int smem1 = DeltaPrepareSmem<DP, CHANNEL>::bytes(vp);
+  if (smem1 > 227 * 1024) SRB_FAIL("delta_chunks: %d bytes of shared memory exceed 232448", smem1);
+  SRB_CUDA_CALL(cudaFuncSetAttribute(delta_chunk_prepare_kernel<DP, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
+  SRB_CUDA_CALL(srb_launch(delta_chunk_prepare_kernel<DP, CHANNEL>, dim3(chunks, a.heads), dim3(DC_PREPARE_THREADS), smem1, s, a, scratch, vp));
+  SRB_LAUNCH_CHECK("delta_chunk_prepare");
+  if (vp % 32 == 0) {
+    const int smem2 = DeltaWalkSmem<DP, CHANNEL, 2>::BYTES;
+    SRB_CUDA_CALL(cudaFuncSetAttribute(delta_chunk_walk_kernel<DP, CHANNEL, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
+    SRB_CUDA_CALL(srb_launch(delta_chunk_walk_kernel<DP, CHANNEL, 2>, dim3(vp / 32, a.heads, a.requests), dim3(256), smem2, s, a,
+                             (const unsigned char*)scratch, vp));
+  } else {
+    const int smem2 = DeltaWalkSmem<DP, CHANNEL, 1>::BYTES;
+    SRB_CUDA_CALL(cudaFuncSetAttribute(delta_chunk_walk_kernel<DP, CHANNEL, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
+    SRB_CUDA_CALL(srb_launch(delta_chunk_walk_kernel<DP, CHANNEL, 1>, dim3(vp / 16, a.heads, a.requests), dim3(128), smem2, s, a,
+                             (const unsigned char*)scratch, vp));
+  }
+  SRB_LAUNCH_CHECK("delta_chunk_walk");
+  return SRB_OK;
+}
+
+// Tokens of a chunk, whether these sizes are taken, and the scratch a chunk needs per head.
+extern "C" int srb_delta_chunk_tokens() { return DC_TOKENS; }
+extern "C" int srb_delta_chunks_supports(int dim, int vdim, int dtype) {
+  return dtype == SRB_DTYPE_BF16 && dim >= 8 && dim <= 128 && dim % 8 == 0 && vdim >= 8 && vdim <= 256 && vdim % 8 == 0;
+}
+extern "C" long long srb_delta_chunk_bytes(int dim, int vdim, int channel_decay) {
+  const int vp = delta_padded_columns(vdim);
+  if (dim <= 64) return channel_decay ? DeltaChunkLayout<64, true>::bytes(vp) : DeltaChunkLayout<64, false>::bytes(vp);
+  return channel_decay ? DeltaChunkLayout<128, true>::bytes(vp) : DeltaChunkLayout<128, false>::bytes(vp);
+}
+
+// What srb_delta_scan computes, for prompt portions in bfloat16.  x: bfloat16 [rows, channels] (srb_short_conv with a bfloat16
+// result); `chunks`: at least the number of chunks of the step, sum over the requests of ceil(rows / srb_delta_chunk_tokens());
+// `scratch`: chunks * heads * srb_delta_chunk_bytes() bytes on a 16-byte border.
+extern "C" int srb_delta_chunks(const void* x, const void* beta, long long beta_pitch, const void* decay, long long decay_pitch,
+                                const float* a_log, const float* dt_bias, const int* positions, const int* cu_rows,
+                                const int* state_slots, float* state, long long slot_floats, void* scratch, float* out, int rows,
+                                int requests, int chunks, int heads, int kv_heads, int dim, int vdim, int taps, int channel_decay,
+                                float unit_eps, int write_state, void* stream) {
+  if (rows <= 0 || requests <= 0 || chunks <= 0) return SRB_OK;
+  if (!srb_delta_chunks_supports(dim, vdim, SRB_DTYPE_BF16)) SRB_FAIL("delta_chunks: heads of %d x %d entries are not taken", dim, vdim);
+  if (heads > 65535) SRB_FAIL("delta_chunks: %d heads exceed one launch", heads);
+  DeltaArgs a;
+  if (delta_args(a, x, beta, beta_pitch, decay, decay_pitch, a_log, dt_bias, positions, cu_rows, state_slots, state, slot_floats, out,
+                 requests, heads, kv_heads, dim, vdim, taps, channel_decay, unit_eps, write_state) != SRB_OK)
+    return SRB_ERR_INVALID;
+  if (((uintptr_t)x & 15) || ((uintptr_t)scratch & 15)) SRB_FAIL("delta_chunks: the convolved inputs and the scratch must start on 16-byte borders");
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dim <= 64)
+    return channel_decay ? launch_delta_chunks<64, true>(a, (unsigned char*)scratch, chunks, s) : launch_delta_chunks<64, false>(a, (unsigned char*)scratch, chunks, s);
+  return channel_decay ? launch_delta_chunks<128, true>(a, (unsigned char*)scratch, chunks, s) : launch_delta_chunks<128, false>(a, (unsigned char*)scratch, chunks, s);
+}

@@ -1596,11 +1596,37 @@ def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log
 
 def delta_chunks_takes(dtype: torch.dtype, dim: int, vdim: int) -> bool:
     """True if the chunk kernels for prompt portions take these sizes (the rule of srb_delta_chunks_supports)."""
-    return False
+    return dtype == torch.bfloat16 and 8 <= dim <= 128 and dim % 8 == 0 and 8 <= vdim <= 256 and vdim % 8 == 0
 
 
 #: tokens per chunk of :func:`delta_chunks` (DC_TOKENS of csrc/delta.cu)
 DELTA_CHUNK_TOKENS = 64
+
+
+@traced("delta")
+def delta_chunks(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                 positions: torch.Tensor, cu_rows: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+                 num_requests: int, chunks: int, *, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, channel_decay: bool,
+                 unit_eps: float, read_only: bool = False) -> None:
+    """What :func:`delta_scan` computes, for prompt portions in bfloat16: the rows of every request are cut into chunks of
+    ``DELTA_CHUNK_TOKENS`` tokens; what a chunk needs that does not depend on the state before it is made for all chunks in
+    parallel, then a request's chunks are walked in order, the tokens of a chunk together, on the tensor cores.  ``qkv``:
+    bfloat16, as :func:`short_conv` wrote it; ``chunks``: the number of chunks of the step, sum over the requests of ceil(rows /
+    DELTA_CHUNK_TOKENS), or more."""
+    _need(qkv, "qkv", torch.bfloat16); _need_rows(beta, "beta", torch.bfloat16)
+    args = _delta_args(qkv, beta, decay, a_log, dt_bias, positions, cu_rows, state_slots, state, out, heads, kv_heads, dim, vdim, taps,
+                       channel_decay)
+    if not delta_chunks_takes(qkv.dtype, dim, vdim):
+        raise KernelError(f"delta_chunks: heads of {dim} x {vdim} entries are not taken")
+    lib = load_library("delta")
+    if lib.srb_delta_chunk_bytes.restype is not ctypes.c_longlong:
+        lib.srb_delta_chunk_bytes.restype = ctypes.c_longlong
+    chunks = max(int(chunks), 1)
+    scratch = torch.empty((chunks * heads * lib.srb_delta_chunk_bytes(dim, vdim, int(channel_decay)),), dtype=torch.uint8,
+                          device=qkv.device)
+    _check(lib, lib.srb_delta_chunks(*args, _ptr(scratch), _ptr(out), qkv.shape[0], int(num_requests), chunks, heads, kv_heads, dim,
+                                     vdim, taps, int(channel_decay), ctypes.c_float(unit_eps), int(not read_only), _stream()),
+           launches=2)
 
 
 @traced("delta_gate_norm")
