@@ -294,6 +294,41 @@ __global__ void delta_gate_norm_kernel(const float* __restrict__ o, const T* __r
   }
 }
 
+// The same in bfloat16 with four consecutive entries a lane: LANES lanes take a head of 4 LANES entries (32, 64 or 128), so a warp
+// takes 32 / LANES heads; rows and columns on 8-byte borders.
+template <int LANES>
+__global__ void __launch_bounds__(128)
+delta_gate_norm_quad_kernel(const float* __restrict__ o, const __nv_bfloat16* __restrict__ g, long long g_pitch,
+                            const float* __restrict__ weight, float eps, float scale, int silu, int rows, int heads,
+                            __nv_bfloat16* __restrict__ out, long long out_pitch) {
+  srb_launch_dependents();
+  const int lane = threadIdx.x % LANES;
+  const float4 w = *reinterpret_cast<const float4*>(weight + lane * 4);
+  srb_grid_dependency_wait();
+  const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / LANES;
+  const bool live = item < (long long)rows * heads;
+  const int row = live ? (int)(item / heads) : 0, head = live ? (int)(item - (long long)row * heads) : 0;
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  uint2 raw = make_uint2(0u, 0u);
+  if (live) {
+    v = *reinterpret_cast<const float4*>(o + (size_t)item * (4 * LANES) + lane * 4);
+    raw = *reinterpret_cast<const uint2*>(g + (size_t)row * g_pitch + (size_t)head * (4 * LANES) + lane * 4);
+  }
+  float squares = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+#pragma unroll
+  for (int offset = LANES / 2; offset > 0; offset >>= 1) squares += __shfl_xor_sync(0xffffffffu, squares, offset);
+  if (!live) return;
+  const float inv = scale / sqrtf(squares / (float)(4 * LANES) + eps);
+  const float2 za = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 zb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  auto gate = [&](float z) { return silu ? z * delta_sigmoid(z) : delta_sigmoid(z); };
+  const __nv_bfloat162 ya = __floats2bfloat162_rn(v.x * inv * w.x * gate(za.x), v.y * inv * w.y * gate(za.y));
+  const __nv_bfloat162 yb = __floats2bfloat162_rn(v.z * inv * w.z * gate(zb.x), v.w * inv * w.w * gate(zb.y));
+  raw.x = *reinterpret_cast<const unsigned*>(&ya);
+  raw.y = *reinterpret_cast<const unsigned*>(&yb);
+  *reinterpret_cast<uint2*>(out + (size_t)row * out_pitch + (size_t)head * (4 * LANES) + lane * 4) = raw;
+}
+
 // o: float [rows, heads * vdim]; g: heads * vdim columns of a projection; weight float [vdim]; out: rows `out_pitch` apart;
 // silu 0: the gate is sigmoid(g), 1: silu(g); `scale`: a factor on everything
 extern "C" int srb_delta_gate_norm(const float* o, const void* g, long long g_pitch, const float* weight, float eps, float scale,
@@ -306,6 +341,14 @@ extern "C" int srb_delta_gate_norm(const float* o, const void* g, long long g_pi
   const int warps = 4;
   const dim3 grid((unsigned)((items + warps - 1) / warps));
   cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == SRB_DTYPE_BF16 && (vdim == 32 || vdim == 64 || vdim == 128) && g_pitch % 4 == 0 && out_pitch % 4 == 0 &&
+      (((uintptr_t)o | (uintptr_t)weight) & 15) == 0 && (((uintptr_t)g | (uintptr_t)out) & 7) == 0) {
+    auto kernel = vdim == 128 ? delta_gate_norm_quad_kernel<32> : (vdim == 64 ? delta_gate_norm_quad_kernel<16> : delta_gate_norm_quad_kernel<8>);
+    SRB_CUDA_CALL(srb_launch(kernel, dim3((unsigned)((items * (vdim / 4) + 127) / 128)), dim3(128), 0, s, o, (const __nv_bfloat16*)g, g_pitch,
+                             weight, eps, scale, silu, rows, heads, (__nv_bfloat16*)out, out_pitch));
+    SRB_LAUNCH_CHECK("delta_gate_norm");
+    return SRB_OK;
+  }
   if (dtype == SRB_DTYPE_F32)
     SRB_CUDA_CALL(srb_launch(delta_gate_norm_kernel<float>, grid, dim3(warps * 32), 0, s, o, (const float*)g, g_pitch, weight, eps,
                              scale, silu, rows, heads, vdim, (float*)out, out_pitch));
@@ -327,8 +370,8 @@ extern "C" int srb_delta_gate_norm(const float* o, const void* g, long long g_pi
 //     S <- e^(c_(n-1)) S + sum_j (k'_j e^(c_(n-1) - c_j)) u_j^T
 // so U = T beta V - W S with T = (1 + L)^-1 and W = T beta (K' e^c).  Every exponential is of a number that is not positive.
 // With a decay per row of S the sums behind L and A do not factor into e^(c_t) and e^(-c_j), which could overflow: they are taken
-// block by block of 16 tokens, the blocks left of the diagonal with both factors relative to c just before the row block (both
-// exponents are then not positive), the diagonal blocks pair by pair.  Two kernels:
+// block by block of 16 tokens with both factors relative to c just before the row block: left of the diagonal both exponents are
+// then not positive; a diagonal block whose c falls by more than 2^100 in some row of S is taken pair by pair.  Two kernels:
 //   1. delta_chunk_prepare: per (chunk, head), in parallel: A, T, W, T beta V and the scaled q' and k'
 //   2. delta_chunk_walk: per (request, head, VS value columns) the chunks in order, S in registers: U, the results, the next S
 // x goes in as bfloat16 (what the convolution wrote); whatever is 32-bit by the design and has to be an operand of a product
@@ -351,6 +394,12 @@ __device__ __forceinline__ void dc_split2(float a, float b, unsigned& hi, unsign
   const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(&hi);
   const float2 f = __bfloat1622float2(h);
   lo = pack_bf16(a - f.x, b - f.y);
+}
+// 2^x for the factors of a chunk: the hardware's exponential (2 units in the last place), results below 2^-126 are zero
+__device__ __forceinline__ float dc_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 __device__ __forceinline__ float2 dc_pair(const __nv_bfloat16* p) {
   return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
@@ -388,7 +437,7 @@ __device__ __forceinline__ bool dc_find(const DeltaArgs& a, int index, int& requ
 
 template <int DP, bool CHANNEL>
 struct DeltaPrepareSmem {
-  static constexpr int XP = DP + DC_PAD, CP = DP + 2, TP = DC_TOKENS + DC_PAD, LP = DC_TOKENS + 1;
+  static constexpr int XP = DP + DC_PAD, CP = DP + 2, TP = DC_TOKENS + DC_PAD, LP = DC_TOKENS + 4;
   static constexpr int K = 0;                                              // bfloat16 [64][XP]
   static constexpr int Q = K + DC_TOKENS * XP * 2;                         // bfloat16 [64][XP]; later T scaled, in two [64][TP]
   static constexpr int T_BYTES = 2 * DC_TOKENS * TP * 2;
@@ -421,7 +470,9 @@ __global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_ker
   float* ik_s = beta_s + DC_TOKENS;
   float* iq_s = ik_s + DC_TOKENS;
   float* cum_s = iq_s + DC_TOKENS;                                         // one decay per head: c, in units of log2
-  float* part_s = cum_s + DC_TOKENS;                                       // [4][DP]
+  float* part_s = cum_s + DC_TOKENS;                                       // [4][DP]; then the first DP floats are zeros
+  const float* zero_s = part_s;
+  int* mild_s = reinterpret_cast<int*>(part_s + 4 * DP);                   // [4]
   srb_launch_dependents();
   srb_grid_dependency_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
@@ -489,6 +540,8 @@ __global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_ker
   }
   cp_async_wait<0>();
   __syncthreads();
+  if (CHANNEL)
+    for (int d = tid; d < DP; d += NTH) part_s[d] = 0.f;   // (every thread has taken its parts' totals)
   // lengths: a warp takes eight tokens
   for (int t = warp * 8; t < warp * 8 + 8; ++t) {
     float kk = 0.f, qq = 0.f;
@@ -507,7 +560,8 @@ __global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_ker
   __syncthreads();
 
   // ---- L and A.  Warps 0-3 take the rows of K, 4-7 those of Q, a block of 16 rows each
-  const int rb = warp & 3, kind = warp >> 2;
+  // (the second four count their blocks backwards, so that the long rows are spread over the SM's quarters)
+  const int kind = warp >> 2, rb = kind ? 3 - (warp & 3) : warp & 3;
   const int r0 = rb * 16 + g, r1 = r0 + 8;
   const __nv_bfloat16* rows_s = kind ? qs : ks;
   float* into = kind ? ts : ls;
@@ -535,53 +589,87 @@ __global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_ker
           const int t = e < 2 ? r0 : r1, j = nt * 8 + 2 * t4 + (e & 1);
           float v = 0.f;
           if (j < t || (kind && j == t))
-            v = acc[nt][e] * (kind ? iq_s[t] : beta_s[t] * ik_s[t]) * ik_s[j] * exp2f(cum_s[t] - cum_s[j]);
+            v = acc[nt][e] * (kind ? iq_s[t] : beta_s[t] * ik_s[t]) * ik_s[j] * dc_exp2(cum_s[t] - cum_s[j]);
           into[t * LP + j] = v;
         }
       }
   } else {
-    if (rb > 0) {
-      const float* ref = cs + (rb * 16 - 1) * CP;          // c just before the row block
-      float acc[6][4];
+    // c falls by what inside the row block?  Up to 2^100 both factors of a diagonal block can be taken relative to c just
+    // before it, too (what the mask discards stays finite)
+    const float* ref = rb ? cs + (rb * 16 - 1) * CP : zero_s;
+    float fall = 0.f;
+    for (int d = lane; d < DP; d += 32) fall = fmaxf(fall, ref[d] - cs[(rb * 16 + 15) * CP + d]);
+    const bool mild = srb_warp_max(fall) <= 100.f;
+    if (lane == 0 && kind == 0) mild_s[rb] = mild;
+    const int tiles = mild ? 2 * rb + 2 : 2 * rb;
+    // the two warps of a row block take every second tile of eight columns, for the rows of K and of Q together
+    float acc_k[4][4], acc_q[4][4];
 #pragma unroll
-      for (int nt = 0; nt < 6; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
-      const float s0 = kind ? iq_s[r0] : beta_s[r0] * ik_s[r0], s1 = kind ? iq_s[r1] : beta_s[r1] * ik_s[r1];
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc_k[i][e] = acc_q[i][e] = 0.f;
+    const float k0 = beta_s[r0] * ik_s[r0], k1 = beta_s[r1] * ik_s[r1], q0 = iq_s[r0], q1 = iq_s[r1];
+    if (kind < tiles) {
 #pragma unroll 1
       for (int kk = 0; kk < DP / 16; ++kk) {
-        const int d = kk * 16 + 2 * t4;
-        const float2 rlo = *reinterpret_cast<const float2*>(ref + d), rhi = *reinterpret_cast<const float2*>(ref + d + 8);
-        auto scaled = [&](const __nv_bfloat16* v, const float* c, float2 from, float sign, float scale) -> float2 {
-          const float2 x2 = dc_pair(v), c2 = *reinterpret_cast<const float2*>(c);
-          return make_float2(x2.x * scale * exp2f(sign * (c2.x - from.x)), x2.y * scale * exp2f(sign * (c2.y - from.y)));
-        };
-        unsigned hi[4], lo[4];
-        float2 v;
-        v = scaled(rows_s + r0 * XP + d, cs + r0 * CP + d, rlo, 1.f, s0);          dc_split2(v.x, v.y, hi[0], lo[0]);
-        v = scaled(rows_s + r1 * XP + d, cs + r1 * CP + d, rlo, 1.f, s1);          dc_split2(v.x, v.y, hi[1], lo[1]);
-        v = scaled(rows_s + r0 * XP + d + 8, cs + r0 * CP + d + 8, rhi, 1.f, s0);  dc_split2(v.x, v.y, hi[2], lo[2]);
-        v = scaled(rows_s + r1 * XP + d + 8, cs + r1 * CP + d + 8, rhi, 1.f, s1);  dc_split2(v.x, v.y, hi[3], lo[3]);
+        unsigned kh[4], kl[4], qh[4], ql[4];
+        float2 from[2];
 #pragma unroll
-        for (int nt = 0; nt < 6; ++nt)
-          if (nt < 2 * rb) {
+        for (int half = 0; half < 2; ++half) {
+          const int d = kk * 16 + 2 * t4 + 8 * half;
+          from[half] = *reinterpret_cast<const float2*>(ref + d);
+          const float2 c0 = *reinterpret_cast<const float2*>(cs + r0 * CP + d), c1 = *reinterpret_cast<const float2*>(cs + r1 * CP + d);
+          const float2 e0 = make_float2(dc_exp2(c0.x - from[half].x), dc_exp2(c0.y - from[half].y));
+          const float2 e1 = make_float2(dc_exp2(c1.x - from[half].x), dc_exp2(c1.y - from[half].y));
+          float2 v = dc_pair(ks + r0 * XP + d);
+          dc_split2(v.x * k0 * e0.x, v.y * k0 * e0.y, kh[2 * half], kl[2 * half]);
+          v = dc_pair(ks + r1 * XP + d);
+          dc_split2(v.x * k1 * e1.x, v.y * k1 * e1.y, kh[2 * half + 1], kl[2 * half + 1]);
+          v = dc_pair(qs + r0 * XP + d);
+          dc_split2(v.x * q0 * e0.x, v.y * q0 * e0.y, qh[2 * half], ql[2 * half]);
+          v = dc_pair(qs + r1 * XP + d);
+          dc_split2(v.x * q1 * e1.x, v.y * q1 * e1.y, qh[2 * half + 1], ql[2 * half + 1]);
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int nt = 2 * i + kind;
+          if (nt < tiles) {
             const int j = nt * 8 + g;
+            const float scale = ik_s[j];
             unsigned bh[2], bl[2];
-            v = scaled(ks + j * XP + d, cs + j * CP + d, rlo, -1.f, ik_s[j]);          dc_split2(v.x, v.y, bh[0], bl[0]);
-            v = scaled(ks + j * XP + d + 8, cs + j * CP + d + 8, rhi, -1.f, ik_s[j]);  dc_split2(v.x, v.y, bh[1], bl[1]);
-            mma_bf16(acc[nt], hi, bh[0], bh[1]);
-            mma_bf16(acc[nt], hi, bl[0], bl[1]);
-            mma_bf16(acc[nt], lo, bh[0], bh[1]);
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+              const int d = kk * 16 + 2 * t4 + 8 * half;
+              const float2 v = dc_pair(ks + j * XP + d), c = *reinterpret_cast<const float2*>(cs + j * CP + d);
+              dc_split2(v.x * scale * dc_exp2(from[half].x - c.x), v.y * scale * dc_exp2(from[half].y - c.y), bh[half], bl[half]);
+            }
+            mma_bf16(acc_k[i], kh, bh[0], bh[1]);
+            mma_bf16(acc_q[i], qh, bh[0], bh[1]);
+            mma_bf16(acc_k[i], kh, bl[0], bl[1]);
+            mma_bf16(acc_q[i], qh, bl[0], bl[1]);
+            mma_bf16(acc_k[i], kl, bh[0], bh[1]);
+            mma_bf16(acc_q[i], ql, bh[0], bh[1]);
           }
+        }
       }
 #pragma unroll
-      for (int nt = 0; nt < 6; ++nt)
-        if (nt < 2 * rb) {
+      for (int i = 0; i < 4; ++i) {
+        const int nt = 2 * i + kind;
+        if (nt < tiles) {
 #pragma unroll
-          for (int e = 0; e < 4; ++e) into[(e < 2 ? r0 : r1) * LP + nt * 8 + 2 * t4 + (e & 1)] = acc[nt][e];
+          for (int e = 0; e < 4; ++e) {
+            const int t = e < 2 ? r0 : r1, j = nt * 8 + 2 * t4 + (e & 1);
+            ls[t * LP + j] = j < t ? acc_k[i][e] : 0.f;
+            ts[t * LP + j] = j <= t ? acc_q[i][e] : 0.f;
+          }
         }
+      }
     }
-    // the diagonal blocks, pair by pair (t >= j): 136 pairs in each of the four
+    __syncthreads();
+    // diagonal blocks in which some decay falls faster, pair by pair (t >= j): 136 pairs each
     for (int item = tid; item < 4 * 136; item += NTH) {
       const int block = item / 136, pair = item - block * 136;
+      if (mild_s[block]) continue;
       int t = (int)((sqrtf(8.0f * pair + 1.0f) - 1.0f) * 0.5f);
       while ((t + 1) * (t + 2) / 2 <= pair) ++t;           // (the root may be off by one)
       while (t * (t + 1) / 2 > pair) --t;
@@ -591,7 +679,7 @@ __global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_ker
       for (int d = 0; d < DP; d += 2) {
         const float2 ct = *reinterpret_cast<const float2*>(cs + t * CP + d), cj = *reinterpret_cast<const float2*>(cs + j * CP + d);
         const float2 kj = dc_pair(ks + j * XP + d), kt = dc_pair(ks + t * XP + d), qt = dc_pair(qs + t * XP + d);
-        const float e0 = kj.x * exp2f(ct.x - cj.x), e1 = kj.y * exp2f(ct.y - cj.y);
+        const float e0 = kj.x * dc_exp2(ct.x - cj.x), e1 = kj.y * dc_exp2(ct.y - cj.y);
         kk = fmaf(kt.x, e0, fmaf(kt.y, e1, kk));
         qk = fmaf(qt.x, e0, fmaf(qt.y, e1, qk));
       }
@@ -623,60 +711,67 @@ __global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_ker
       const float2 c = *reinterpret_cast<const float2*>(cs + t * CP + d), end = *reinterpret_cast<const float2*>(last + d);
       const float2 q = dc_pair(qs + t * XP + d), k = dc_pair(ks + t * XP + d);
       unsigned hi, lo;
-      dc_split2(q.x * iq_s[t] * exp2f(c.x), q.y * iq_s[t] * exp2f(c.y), hi, lo);
+      dc_split2(q.x * iq_s[t] * dc_exp2(c.x), q.y * iq_s[t] * dc_exp2(c.y), hi, lo);
       *reinterpret_cast<unsigned*>(qh + t * DP + d) = hi;
       *reinterpret_cast<unsigned*>(qh + DC_TOKENS * DP + t * DP + d) = lo;
-      dc_split2(k.x * ik_s[t] * exp2f(end.x - c.x), k.y * ik_s[t] * exp2f(end.y - c.y), hi, lo);
+      dc_split2(k.x * ik_s[t] * dc_exp2(end.x - c.x), k.y * ik_s[t] * dc_exp2(end.y - c.y), hi, lo);
       *reinterpret_cast<unsigned*>(kh + t * DP + d) = hi;
       *reinterpret_cast<unsigned*>(kh + DC_TOKENS * DP + t * DP + d) = lo;
     }
-    for (int d = tid; d < DP; d += NTH) factors[d] = exp2f(last[d]);
+    for (int d = tid; d < DP; d += NTH) factors[d] = dc_exp2(last[d]);
   } else if (tid < DC_TOKENS) {
-    factors[tid] = iq_s[tid] * exp2f(cum_s[tid]);
-    factors[DC_TOKENS + tid] = ik_s[tid] * exp2f(cum_s[DC_TOKENS - 1] - cum_s[tid]);
-    if (tid == 0) factors[2 * DC_TOKENS] = exp2f(cum_s[DC_TOKENS - 1]);
+    factors[tid] = iq_s[tid] * dc_exp2(cum_s[tid]);
+    factors[DC_TOKENS + tid] = ik_s[tid] * dc_exp2(cum_s[DC_TOKENS - 1] - cum_s[tid]);
+    if (tid == 0) factors[2 * DC_TOKENS] = dc_exp2(cum_s[DC_TOKENS - 1]);
   }
   __syncthreads();
 
-  // ---- T = (1 + L)^-1: the four diagonal blocks by forward substitution (a lane takes a column), then the blocks below them
-  if (warp < 4 && lane < 16) {
-    const int b = warp * 16;
-    float col[16];
+  // ---- T = (1 + L)^-1: two diagonal blocks of 32 by forward substitution (a lane takes a column), then the block below them,
+  // T_10 = -T_11 L_10 T_00
+  if (warp < 2) {
+    const int b = warp * 32;
+    float col[32];
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      float v = i == lane ? 1.f : 0.f;
+    for (int i = 0; i < 32; ++i) {
+      const float4* row = reinterpret_cast<const float4*>(ls + (b + i) * LP + b);
+      float v[4] = {i == lane ? 1.f : 0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int m = 0; m < 16; ++m)
-        if (m < i) v = fmaf(-ls[(b + i) * LP + b + m], col[m], v);
-      col[i] = v;
+      for (int m = 0; m < i; m += 4) {
+        const float4 l = row[m / 4];
+        v[0] = fmaf(-l.x, col[m], v[0]);
+        if (m + 1 < i) v[1] = fmaf(-l.y, col[m + 1], v[1]);
+        if (m + 2 < i) v[2] = fmaf(-l.z, col[m + 2], v[2]);
+        if (m + 3 < i) v[3] = fmaf(-l.w, col[m + 3], v[3]);
+      }
+      col[i] = (v[0] + v[1]) + (v[2] + v[3]);
     }
 #pragma unroll
-    for (int i = 0; i < 16; ++i) ts[(b + i) * LP + b + lane] = col[i];
+    for (int i = 0; i < 32; ++i) ts[(b + i) * LP + b + lane] = col[i];
   }
   __syncthreads();
   {
-    const int i = tid >> 4, j = tid & 15;                  // an entry of a 16 x 16 block
-    for (int gap = 1; gap < 4; ++gap) {
-      // P = sum over the blocks between of L T, kept where the result goes; then T_ii P.  (the places are not read before)
-      for (int cb = 0; cb + gap < 4; ++cb) {
-        const int b = (cb + gap) * 16, c = cb * 16;
-        float v = 0.f;
-        for (int m = c; m < b; ++m) v = fmaf(ls[(b + i) * LP + m], ts[m * LP + c + j], v);
-        ts[(b + i) * LP + c + j] = v;
-      }
-      __syncthreads();
-      float v[3];
+    const int i = tid >> 3, j = (tid & 7) * 4;             // four entries of a row of a 32 x 32 block
+    const float4* left[2] = {reinterpret_cast<const float4*>(ls + (32 + i) * LP), reinterpret_cast<const float4*>(ts + (32 + i) * LP + 32)};
+    float* mine = ts + (32 + i) * LP + j;
 #pragma unroll
-      for (int cb = 0; cb < 3; ++cb)
-        if (cb + gap < 4) {
-          const int b = (cb + gap) * 16, c = cb * 16;
-          v[cb] = 0.f;
-          for (int m = 0; m <= i; ++m) v[cb] = fmaf(-ts[(b + i) * LP + b + m], ts[(b + m) * LP + c + j], v[cb]);
+    for (int pass = 0; pass < 2; ++pass) {                 // L_10 T_00, kept where the result goes; then -T_11 times that
+      const float* right = ts + (pass ? 32 * LP : 0) + j;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int m = 0; m < 32; m += 4) {
+        const float4 l = left[pass][m / 4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float4 r = *reinterpret_cast<const float4*>(right + (m + k) * LP);
+          const float f = k == 0 ? l.x : (k == 1 ? l.y : (k == 2 ? l.z : l.w));
+          v.x = fmaf(f, r.x, v.x); v.y = fmaf(f, r.y, v.y); v.z = fmaf(f, r.z, v.z); v.w = fmaf(f, r.w, v.w);
         }
-      __syncthreads();
-#pragma unroll
-      for (int cb = 0; cb < 3; ++cb)
-        if (cb + gap < 4) ts[((cb + gap) * 16 + i) * LP + cb * 16 + j] = v[cb];
+      }
+      if (pass) {
+        __syncthreads();                                   // every thread has read the product before
+        v = make_float4(-v.x, -v.y, -v.z, -v.w);
+      }
+      *reinterpret_cast<float4*>(mine) = v;
       __syncthreads();
     }
   }
@@ -698,7 +793,7 @@ __global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_ker
       const int t = i / (DP / 2), d = i % (DP / 2) * 2;
       const float2 c = *reinterpret_cast<const float2*>(cs + t * CP + d), k = dc_pair(ks + t * XP + d);
       unsigned hi, lo;
-      dc_split2(k.x * ik_s[t] * exp2f(c.x), k.y * ik_s[t] * exp2f(c.y), hi, lo);
+      dc_split2(k.x * ik_s[t] * dc_exp2(c.x), k.y * ik_s[t] * dc_exp2(c.y), hi, lo);
       *reinterpret_cast<unsigned*>(second + t * XP + d) = hi;
       *reinterpret_cast<unsigned*>(second + DC_TOKENS * XP + t * XP + d) = lo;
     }
@@ -708,7 +803,7 @@ __global__ void __launch_bounds__(DC_PREPARE_THREADS, 2) delta_chunk_prepare_ker
       const int t = i / (DC_TOKENS / 2), j = i % (DC_TOKENS / 2) * 2;
       const float2 h = dc_pair(th + t * TP + j), l = dc_pair(tl + t * TP + j);
       unsigned hi, lo;
-      dc_split2((h.x + l.x) * ik_s[j] * exp2f(cum_s[j]), (h.y + l.y) * ik_s[j + 1] * exp2f(cum_s[j + 1]), hi, lo);
+      dc_split2((h.x + l.x) * ik_s[j] * dc_exp2(cum_s[j]), (h.y + l.y) * ik_s[j + 1] * dc_exp2(cum_s[j + 1]), hi, lo);
       *reinterpret_cast<unsigned*>(second + t * TP + j) = hi;
       *reinterpret_cast<unsigned*>(second + DC_TOKENS * TP + t * TP + j) = lo;
     }
@@ -923,46 +1018,53 @@ __global__ void __launch_bounds__(128 * MT) delta_chunk_walk_kernel(DeltaArgs a,
     cp_async_wait<0>();
     __syncthreads();                                       // W, q and the state are there; A, k and U are no longer read
     fetch_ak(chunk);
-    float u[2][4], o[2][4];
+    // U = T beta V - W S and (q e^c) S for the warp's 16 tokens; the products of the roundings and of the rests go into sums of
+    // their own, so that consecutive products do not wait for each other
+    float u[2][4], o[2][4], u_rest[2][2][4], o_rest[2][2][4];
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) { u[nt][e] = uv[nt][e]; o[nt][e] = 0.f; }
-    // U = T beta V - W S and (q e^c) S for the warp's 16 tokens
+      for (int e = 0; e < 4; ++e) {
+        u[nt][e] = uv[nt][e];
+        o[nt][e] = u_rest[0][nt][e] = u_rest[1][nt][e] = o_rest[0][nt][e] = o_rest[1][nt][e] = 0.f;
+      }
 #pragma unroll 2
     for (int kk = 0; kk < DP / 16; ++kk) {
-      unsigned sh[4], sl[4];
+      unsigned sh[4], sl[4], w[2][4], q[2][4];
       const __nv_bfloat16* at = ss + (tile * 16 + (matrix & 1) * 8 + inner) * XP + kk * 16 + (matrix >> 1) * 8;
       ldmatrix_x4(sh[0], sh[1], sh[2], sh[3], at);
       ldmatrix_x4(sl[0], sl[1], sl[2], sl[3], at + M::S_HALF / 2);
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) {
-        unsigned b0, b1, b2, b3;
-        const int row = part * 16 + nt * 8 + inner;
-        ldmatrix_x4(b0, b1, b2, b3, ws + (matrix >> 1) * DC_TOKENS * XP + row * XP + kk * 16 + (matrix & 1) * 8);
-        mma_bf16(u[nt], sh, b0, b1);
-        mma_bf16(u[nt], sh, b2, b3);
-        mma_bf16(u[nt], sl, b0, b1);
+        const int row = part * 16 + nt * 8 + inner, column = kk * 16 + (matrix & 1) * 8;
+        ldmatrix_x4(w[nt][0], w[nt][1], w[nt][2], w[nt][3], ws + (matrix >> 1) * DC_TOKENS * XP + row * XP + column);
+        if (CHANNEL) ldmatrix_x4(q[nt][0], q[nt][1], q[nt][2], q[nt][3], qs + (matrix >> 1) * DC_TOKENS * XP + row * XP + column);
       }
+      if (!CHANNEL)                                        // both tiles of eight tokens at once
+        ldmatrix_x4(q[0][0], q[0][1], q[1][0], q[1][1], qs + (part * 16 + (matrix >> 1) * 8 + inner) * XP + kk * 16 + (matrix & 1) * 8);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) mma_bf16(u[nt], sh, w[nt][0], w[nt][1]);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) mma_bf16(o[nt], sh, q[nt][0], q[nt][1]);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) mma_bf16(u_rest[0][nt], sh, w[nt][2], w[nt][3]);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) mma_bf16(u_rest[1][nt], sl, w[nt][0], w[nt][1]);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) mma_bf16(o_rest[1][nt], sl, q[nt][0], q[nt][1]);
       if (CHANNEL) {
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          unsigned b0, b1, b2, b3;
-          const int row = part * 16 + nt * 8 + inner;
-          ldmatrix_x4(b0, b1, b2, b3, qs + (matrix >> 1) * DC_TOKENS * XP + row * XP + kk * 16 + (matrix & 1) * 8);
-          mma_bf16(o[nt], sh, b0, b1);
-          mma_bf16(o[nt], sh, b2, b3);
-          mma_bf16(o[nt], sl, b0, b1);
-        }
-      } else {
-        unsigned b0, b1, b2, b3;                           // both tiles of eight tokens at once
-        ldmatrix_x4(b0, b1, b2, b3, qs + (part * 16 + (matrix >> 1) * 8 + inner) * XP + kk * 16 + (matrix & 1) * 8);
-        mma_bf16(o[0], sh, b0, b1);
-        mma_bf16(o[0], sl, b0, b1);
-        mma_bf16(o[1], sh, b2, b3);
-        mma_bf16(o[1], sl, b2, b3);
+        for (int nt = 0; nt < 2; ++nt) mma_bf16(o_rest[0][nt], sh, q[nt][2], q[nt][3]);
       }
     }
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        u[nt][e] += u_rest[0][nt][e] + u_rest[1][nt][e];
+        o[nt][e] += o_rest[0][nt][e] + o_rest[1][nt][e];
+        o_rest[0][nt][e] = o_rest[1][nt][e] = 0.f;
+      }
     cp_async_wait<0>();                                    // A, k and the factors (each thread its own copies; the barrier below joins them)
     if (!CHANNEL) __syncthreads();                         // the factors are read below by every thread
 #pragma unroll
@@ -1005,46 +1107,50 @@ __global__ void __launch_bounds__(128 * MT) delta_chunk_walk_kernel(DeltaArgs a,
 #pragma unroll
     for (int kk = 0; kk < DC_TOKENS / 16; ++kk) {
       const __nv_bfloat16* at = us + (tile * 16 + (matrix & 1) * 8 + inner) * TP + kk * 16 + (matrix >> 1) * 8;
-      unsigned uh[4], ul[4];
+      unsigned uh[4], ul[4], k[DT][4];
       ldmatrix_x4(uh[0], uh[1], uh[2], uh[3], at);
       ldmatrix_x4(ul[0], ul[1], ul[2], ul[3], at + M::U_HALF / 2);
-      if (kk <= part) {                                    // A is zero above the diagonal
+      if (CHANNEL) {
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          unsigned b0, b1, b2, b3;
-          ldmatrix_x4(b0, b1, b2, b3, as + (matrix >> 1) * DC_TOKENS * TP + (part * 16 + nt * 8 + inner) * TP + kk * 16 + (matrix & 1) * 8);
-          mma_bf16(o[nt], uh, b0, b1);
-          mma_bf16(o[nt], uh, b2, b3);
-          mma_bf16(o[nt], ul, b0, b1);
-        }
+        for (int nt = 0; nt < DT; ++nt)
+          ldmatrix_x4_trans(k[nt][0], k[nt][1], k[nt][2], k[nt][3], ks + (matrix >> 1) * DC_TOKENS * XP +
+                            (kk * 16 + (matrix & 1) * 8 + inner) * XP + part * (DP / 4) + nt * 8);
+      } else {
+#pragma unroll
+        for (int nt = 0; nt < DT; nt += 2)                 // two tiles of eight rows of S at once
+          ldmatrix_x4_trans(k[nt][0], k[nt][1], k[nt + 1][0], k[nt + 1][1], ks + (kk * 16 + (matrix & 1) * 8 + inner) * XP +
+                            part * (DP / 4) + nt * 8 + (matrix >> 1) * 8);
+      }
+      if (kk <= part) {                                    // A is zero above the diagonal
+        unsigned b[2][4];
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+          ldmatrix_x4(b[nt][0], b[nt][1], b[nt][2], b[nt][3], as + (matrix >> 1) * DC_TOKENS * TP +
+                      (part * 16 + nt * 8 + inner) * TP + kk * 16 + (matrix & 1) * 8);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) mma_bf16(o[nt], uh, b[nt][0], b[nt][1]);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) mma_bf16(o_rest[0][nt], uh, b[nt][2], b[nt][3]);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) mma_bf16(o_rest[1][nt], ul, b[nt][0], b[nt][1]);
       }
       if (!CHANNEL) {
         ldmatrix_x4(uh[0], uh[1], uh[2], uh[3], at + M::U_HALF);
         ldmatrix_x4(ul[0], ul[1], ul[2], ul[3], at + M::U_HALF + M::U_HALF / 2);
       }
+#pragma unroll
+      for (int nt = 0; nt < DT; ++nt) mma_bf16(s[nt], uh, k[nt][0], k[nt][1]);
       if (CHANNEL) {
 #pragma unroll
-        for (int nt = 0; nt < DT; ++nt) {
-          unsigned b0, b1, b2, b3;
-          const int d = part * (DP / 4) + nt * 8;
-          ldmatrix_x4_trans(b0, b1, b2, b3, ks + (matrix >> 1) * DC_TOKENS * XP + (kk * 16 + (matrix & 1) * 8 + inner) * XP + d);
-          mma_bf16(s[nt], uh, b0, b1);
-          mma_bf16(s[nt], uh, b2, b3);
-          mma_bf16(s[nt], ul, b0, b1);
-        }
-      } else {
-#pragma unroll
-        for (int nt = 0; nt < DT; nt += 2) {
-          unsigned b0, b1, b2, b3;
-          const int d = part * (DP / 4) + nt * 8;
-          ldmatrix_x4_trans(b0, b1, b2, b3, ks + (kk * 16 + (matrix & 1) * 8 + inner) * XP + d + (matrix >> 1) * 8);
-          mma_bf16(s[nt], uh, b0, b1);
-          mma_bf16(s[nt], ul, b0, b1);
-          mma_bf16(s[nt + 1], uh, b2, b3);
-          mma_bf16(s[nt + 1], ul, b2, b3);
-        }
+        for (int nt = 0; nt < DT; ++nt) mma_bf16(s[nt], uh, k[nt][2], k[nt][3]);
       }
+#pragma unroll
+      for (int nt = 0; nt < DT; ++nt) mma_bf16(s[nt], ul, k[nt][0], k[nt][1]);
     }
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[nt][e] += o_rest[0][nt][e] + o_rest[1][nt][e];
     if (chunk + 1 < chunks) keep_state();
     const int left = rows - chunk * DC_TOKENS;
     float* out = a.out + (size_t)(begin + chunk * DC_TOKENS) * a.heads * vdim + (size_t)head * vdim;
@@ -1078,7 +1184,10 @@ static int launch_delta_chunks(const DeltaArgs& a, unsigned char* scratch, int c
   SRB_CUDA_CALL(cudaFuncSetAttribute(delta_chunk_prepare_kernel<DP, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
   SRB_CUDA_CALL(srb_launch(delta_chunk_prepare_kernel<DP, CHANNEL>, dim3(chunks, a.heads), dim3(DC_PREPARE_THREADS), smem1, s, a, scratch, vp));
   SRB_LAUNCH_CHECK("delta_chunk_prepare");
-  if (vp % 32 == 0) {
+  // two tiles of value columns per block share the fetched operands; with a decay per row of S (more to fetch and to multiply per
+  // column) one tile per block is quicker while that fills no more SMs than there are
+  const int mt = (vp % 32 != 0 || (CHANNEL && (long long)vp / 16 * a.heads * a.requests <= srb_sm_count())) ? 1 : 2;
+  if (mt == 2) {
     const int smem2 = DeltaWalkSmem<DP, CHANNEL, 2>::BYTES;
     SRB_CUDA_CALL(cudaFuncSetAttribute(delta_chunk_walk_kernel<DP, CHANNEL, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
     SRB_CUDA_CALL(srb_launch(delta_chunk_walk_kernel<DP, CHANNEL, 2>, dim3(vp / 32, a.heads, a.requests), dim3(256), smem2, s, a,

@@ -396,6 +396,121 @@ __global__ void norm_add_norm_kernel(float* __restrict__ residual, const T* __re
     for (int i = threadIdx.x; i < width; i += blockDim.x) dst[width + i] = srb_from_float<T>(extra[src + i]);
 }
 
+// The same for RMS norms over the whole row (or none), with the row in registers: four consecutive entries per thread and item,
+// ITEMS of them, all loads of a thread in flight together.  Widths that are multiples of four, rows on 16-byte borders (of
+// floats), no `extra`.
+template <typename T, int ITEMS, bool PARTS>
+__global__ void __launch_bounds__(256, ITEMS <= 2 ? 4 : 1)
+norm_add_norm_vec_kernel(float* __restrict__ residual, const T* __restrict__ delta, const float* __restrict__ delta_f32,
+                         NormSpec inner, NormSpec outer, T* __restrict__ out, size_t out_pitch, const int* __restrict__ row_index,
+                         int width, int write_residual, const float* __restrict__ addend, int num_parts, size_t part_stride) {
+  __shared__ float scratch[33];
+  srb_launch_dependents();
+  const int step = blockDim.x * 4;
+  float4 wi[ITEMS], wo[ITEMS];
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {                     // the weights are constants: ahead of the wait
+    const int i = threadIdx.x * 4 + it * step;
+    wi[it] = wo[it] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < width && inner.kind != SRB_NORM_NONE) wi[it] = *reinterpret_cast<const float4*>(inner.weight + i);
+    if (i < width && out && outer.kind != SRB_NORM_NONE) wo[it] = *reinterpret_cast<const float4*>(outer.weight + i);
+  }
+  srb_grid_dependency_wait();
+  const size_t src = (size_t)(row_index ? row_index[blockIdx.x] : blockIdx.x) * width;
+  const bool pending = delta || delta_f32;
+  float4 x[ITEMS], d[ITEMS];
+  float squares = 0.f;
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int i = threadIdx.x * 4 + it * step;
+    x[it] = d[it] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < width) {
+      x[it] = *reinterpret_cast<const float4*>(residual + src + i);
+      if (delta) d[it] = load4(delta + src + i);
+      else if (!PARTS && delta_f32) d[it] = load4(delta_f32 + src + i);
+    }
+  }
+  if (PARTS) {
+    // partial sums of a product cut along K, added in part order, the loads of four parts in flight
+    for (int first = 0; first < num_parts; first += 4) {
+#pragma unroll
+      for (int it = 0; it < ITEMS; ++it) {
+        const int i = threadIdx.x * 4 + it * step;
+        if (i >= width) break;
+        float4 p[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (first + j < num_parts) p[j] = load4(delta_f32 + (first + j) * part_stride + src + i);
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (first + j < num_parts) { d[it].x += p[j].x; d[it].y += p[j].y; d[it].z += p[j].z; d[it].w += p[j].w; }
+      }
+    }
+  }
+  if (pending) {
+    float factor = 1.f;
+    if (inner.kind != SRB_NORM_NONE) {
+#pragma unroll
+      for (int it = 0; it < ITEMS; ++it) squares += d[it].x * d[it].x + d[it].y * d[it].y + d[it].z * d[it].z + d[it].w * d[it].w;
+      factor = 1.0f / sqrtf(srb_block_sum(squares, scratch) / (float)width + inner.eps);
+    }
+#pragma unroll
+    for (int it = 0; it < ITEMS; ++it) {
+      if (inner.kind != SRB_NORM_NONE) {
+        d[it].x = d[it].x * factor * wi[it].x * inner.scale; d[it].y = d[it].y * factor * wi[it].y * inner.scale;
+        d[it].z = d[it].z * factor * wi[it].z * inner.scale; d[it].w = d[it].w * factor * wi[it].w * inner.scale;
+      }
+      x[it].x += d[it].x; x[it].y += d[it].y; x[it].z += d[it].z; x[it].w += d[it].w;
+    }
+  }
+  squares = 0.f;
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int i = threadIdx.x * 4 + it * step;
+    if (i >= width) break;
+    if (addend) {
+      const float4 a = load4(addend + src + i);
+      x[it].x += a.x; x[it].y += a.y; x[it].z += a.z; x[it].w += a.w;
+    }
+    if (write_residual && (pending || addend)) *reinterpret_cast<float4*>(residual + src + i) = x[it];
+    squares += x[it].x * x[it].x + x[it].y * x[it].y + x[it].z * x[it].z + x[it].w * x[it].w;
+  }
+  if (!out) return;
+  float factor = 1.f;
+  if (outer.kind != SRB_NORM_NONE) factor = 1.0f / sqrtf(srb_block_sum(squares, scratch) / (float)width + outer.eps);
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int i = threadIdx.x * 4 + it * step;
+    if (i >= width) break;
+    if (outer.kind != SRB_NORM_NONE) {
+      x[it].x = x[it].x * factor * wo[it].x * outer.scale; x[it].y = x[it].y * factor * wo[it].y * outer.scale;
+      x[it].z = x[it].z * factor * wo[it].z * outer.scale; x[it].w = x[it].w * factor * wo[it].w * outer.scale;
+    }
+    store4(out + (size_t)blockIdx.x * out_pitch + i, x[it]);
+  }
+}
+
+template <typename T>
+static int launch_norm_add_norm_vec(float* residual, const void* delta, const float* delta_f32, const NormSpec& inner, const NormSpec& outer,
+                                    void* out, long long out_pitch, const int* row_index, int rows, int width, int write_residual,
+                                    const float* addend, int num_parts, long long part_stride, cudaStream_t s) {
+  const int quads = width / 4;
+  // few rows: as many threads as the row has pieces; many: two pieces a thread
+  int items = quads <= 256 && rows <= 64 ? 1 : (quads <= 512 ? 2 : (quads <= 1024 ? 4 : 8));
+  const int threads = ((quads + items - 1) / items + 31) / 32 * 32;
+#define SRB_NORM_VEC(ITEMS)                                                                                                    \
+  SRB_CUDA_CALL(srb_launch(num_parts > 0 ? norm_add_norm_vec_kernel<T, ITEMS, true> : norm_add_norm_vec_kernel<T, ITEMS, false>, dim3(rows), dim3(threads), 0, s, residual, (const T*)delta,    \
+                           delta_f32, inner, outer, (T*)out, (size_t)out_pitch, row_index, width, write_residual, addend,     \
+                           num_parts, (size_t)part_stride))
+  if (items == 1) SRB_NORM_VEC(1);
+  else if (items == 2) SRB_NORM_VEC(2);
+  else if (items == 4) SRB_NORM_VEC(4);
+  else SRB_NORM_VEC(8);
+#undef SRB_NORM_VEC
+  SRB_LAUNCH_CHECK("norm_add_norm");
+  return SRB_OK;
+}
+
 // `*_groups` (RMS norms only; 1: the whole row) and `*_scale` (1: none) as NormSpec says.  `addend` (optional, float,
 // shaped like the residual): a second term of the sum, added after the pending one: x = residual + inner(delta) + addend.
 // `num_parts` > 0: `delta_f32` holds that many partial sums of the pending term, `part_stride` floats apart, which are
@@ -425,6 +540,17 @@ extern "C" int srb_norm_add_norm_parts(float* residual, const void* delta, const
   const NormSpec outer{outer_kind, outer_weight, outer_bias, outer_eps, outer_groups, outer_scale};
   const int block = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
   cudaStream_t s = (cudaStream_t)stream;
+  const size_t element = dtype == SRB_DTYPE_BF16 ? 2 : 4;
+  const bool plain = inner_kind != SRB_NORM_LAYER && outer_kind != SRB_NORM_LAYER && inner_groups == 1 && outer_groups == 1 && !extra &&
+                     width % 4 == 0 && width <= 8192 && out_pitch % 4 == 0 && part_stride % 4 == 0 &&
+                     (((uintptr_t)residual | (uintptr_t)delta_f32 | (uintptr_t)addend | (uintptr_t)inner_weight | (uintptr_t)outer_weight) & 15) == 0 &&
+                     (((uintptr_t)delta | (uintptr_t)out) & (4 * element - 1)) == 0;
+  if (plain && dtype == SRB_DTYPE_F32)
+    return launch_norm_add_norm_vec<float>(residual, delta, delta_f32, inner, outer, out, out_pitch, row_index, rows, width, write_residual,
+                                           addend, num_parts, part_stride, s);
+  if (plain && dtype == SRB_DTYPE_BF16)
+    return launch_norm_add_norm_vec<__nv_bfloat16>(residual, delta, delta_f32, inner, outer, out, out_pitch, row_index, rows, width,
+                                                   write_residual, addend, num_parts, part_stride, s);
   if (dtype == SRB_DTYPE_F32) {
     if (smem > 48 * 1024)
       SRB_CUDA_CALL(cudaFuncSetAttribute(norm_add_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));

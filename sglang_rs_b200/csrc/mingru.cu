@@ -5,7 +5,7 @@
 //   S_t = (1 - z_t) S_(t-1) + z_t c_t                out_t = S_t silu(g)
 //
 // Every channel runs by itself, so a step is bound by reading the projection.  Steps in which every request brings one row
-// (decoded tokens) are one pass.  Other steps cut each request's rows into chunks of 64: (1) per (chunk, channel) the chunk as
+// (decoded tokens) are one pass.  Other steps cut each request's rows into chunks of 32: (1) per (chunk, channel) the chunk as
 // an affine map S -> A S + B, (2) per (request, channel) the states before every chunk, in order, the slot receiving the last
 // one, (3) per (chunk, channel) the rows again from the state before the chunk.  Everything between the projection and the
 // result is 32-bit in both dtypes.  A request whose first row of the step is at position 0 starts from zero whatever its slot
@@ -16,7 +16,7 @@
 SRB_DEFINE_LAST_ERROR()
 SRB_DEFINE_PDL_SWITCH()
 
-#define GRU_CHUNK 64
+#define GRU_CHUNK 32
 #define GRU_THREADS 128
 #define GRU_BATCH 8              // rows whose loads are in flight together
 
@@ -39,11 +39,11 @@ struct GruArgs {
 
 // (1 - z, z c) of a row: S <- keep S + add
 __device__ __forceinline__ float2 gru_row(float z, float x) {
-  const float gate = 1.0f / (1.0f + expf(-z));
-  const float candidate = x >= 0.f ? x + 0.5f : 1.0f / (1.0f + expf(-x));
+  const float gate = __fdividef(1.0f, 1.0f + expf(-z));   // (a quotient to 2 units in the last place)
+  const float candidate = x >= 0.f ? x + 0.5f : __fdividef(1.0f, 1.0f + expf(-x));
   return make_float2(1.0f - gate, gate * candidate);
 }
-__device__ __forceinline__ float gru_silu(float g) { return g / (1.0f + expf(-g)); }
+__device__ __forceinline__ float gru_silu(float g) { return __fdividef(g, 1.0f + expf(-g)); }
 
 template <typename T>
 __global__ void __launch_bounds__(GRU_THREADS) gru_single_kernel(GruArgs a) {
@@ -82,40 +82,70 @@ __device__ __forceinline__ bool gru_find(const GruArgs& a, int index, int& reque
   return false;
 }
 
-// OUTPUT false: the chunk's map; true: the rows from the state before the chunk
-template <typename T, bool OUTPUT>
+// V neighbouring channels of a row: one load, or (two bfloat16) four bytes
+template <typename T, int V> struct GruPiece { T v[V]; };
+template <typename T, int V> __device__ __forceinline__ GruPiece<T, V> gru_load(const T* p) {
+  GruPiece<T, V> r;
+  if constexpr (sizeof(T) * V == 4) *reinterpret_cast<unsigned*>(r.v) = *reinterpret_cast<const unsigned*>(p);
+  else r.v[0] = *p;
+  return r;
+}
+template <typename T, int V> __device__ __forceinline__ void gru_store(T* p, const GruPiece<T, V>& r) {
+  if constexpr (sizeof(T) * V == 4) *reinterpret_cast<unsigned*>(p) = *reinterpret_cast<const unsigned*>(r.v);
+  else *p = r.v[0];
+}
+
+// OUTPUT false: the chunk's map; true: the rows from the state before the chunk.  A thread takes V channels.
+template <typename T, int V, bool OUTPUT>
 __global__ void __launch_bounds__(GRU_THREADS) gru_chunk_kernel(GruArgs a) {
   srb_launch_dependents();
-  const int c = blockIdx.y * GRU_THREADS + threadIdx.x;
-  const float zb = c < a.width ? a.z_bias[c] : 0.f, xb = c < a.width ? a.x_bias[c] : 0.f;
+  const int c = (blockIdx.x * GRU_THREADS + threadIdx.x) * V;
+  float zb[V], xb[V];
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    zb[k] = c < a.width ? a.z_bias[c + k] : 0.f;
+    xb[k] = c < a.width ? a.x_bias[c + k] : 0.f;
+  }
   srb_grid_dependency_wait();
   int request, row0, n;
-  if (!gru_find(a, blockIdx.x, request, row0, n) || c >= a.width) return;
+  if (!gru_find(a, blockIdx.y, request, row0, n) || c >= a.width) return;
   const T* p = reinterpret_cast<const T*>(a.proj) + (size_t)row0 * a.pitch + c;
-  float* map = a.maps + (size_t)blockIdx.x * 2 * a.width + c;
-  float keep = 1.f, s = OUTPUT ? map[0] : 0.f;
+  T* out = reinterpret_cast<T*>(a.out) + (size_t)row0 * a.out_pitch + c;
+  float* map = a.maps + (size_t)blockIdx.y * 2 * a.width + c;
+  float keep[V], s[V];
+#pragma unroll
+  for (int k = 0; k < V; ++k) { keep[k] = 1.f; s[k] = OUTPUT ? map[k] : 0.f; }
+#pragma unroll 1
   for (int t0 = 0; t0 < n; t0 += GRU_BATCH) {
-    float z[GRU_BATCH], x[GRU_BATCH], g[GRU_BATCH];
+    GruPiece<T, V> z[GRU_BATCH], x[GRU_BATCH], g[GRU_BATCH];
 #pragma unroll
     for (int j = 0; j < GRU_BATCH; ++j)
       if (t0 + j < n) {
         const T* row = p + (size_t)(t0 + j) * a.pitch;
-        z[j] = srb_to_float(row[a.z_at]);
-        x[j] = srb_to_float(row[a.x_at]);
-        if (OUTPUT) g[j] = srb_to_float(row[a.g_at]);
+        z[j] = gru_load<T, V>(row + a.z_at);
+        x[j] = gru_load<T, V>(row + a.x_at);
+        if (OUTPUT) g[j] = gru_load<T, V>(row + a.g_at);
       }
 #pragma unroll
     for (int j = 0; j < GRU_BATCH; ++j)
       if (t0 + j < n) {
-        const float2 m = gru_row(z[j] + zb, x[j] + xb);
-        s = fmaf(m.x, s, m.y);
-        if (OUTPUT) reinterpret_cast<T*>(a.out)[(size_t)(row0 + t0 + j) * a.out_pitch + c] = srb_from_float<T>(s * gru_silu(g[j]) * a.scale);
-        else keep *= m.x;
+        GruPiece<T, V> y;
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+          const float2 m = gru_row(srb_to_float(z[j].v[k]) + zb[k], srb_to_float(x[j].v[k]) + xb[k]);
+          s[k] = fmaf(m.x, s[k], m.y);
+          if (OUTPUT) y.v[k] = srb_from_float<T>(s[k] * gru_silu(srb_to_float(g[j].v[k])) * a.scale);
+          else keep[k] *= m.x;
+        }
+        if (OUTPUT) gru_store<T, V>(out + (size_t)(t0 + j) * a.out_pitch, y);
       }
   }
   if (!OUTPUT) {
-    map[0] = keep;
-    map[a.width] = s;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      map[k] = keep[k];
+      map[a.width + k] = s[k];
+    }
   }
 }
 
@@ -161,9 +191,15 @@ static int launch_gru(const GruArgs& a, int single_rows, int chunks, cudaStream_
     SRB_LAUNCH_CHECK("mingru_single");
     return SRB_OK;
   }
-  SRB_CUDA_CALL(srb_launch(gru_chunk_kernel<T, false>, dim3(chunks, blocks), dim3(GRU_THREADS), 0, s, a));
+  if (chunks > 65535) SRB_FAIL("mingru: %d chunks exceed one launch", chunks);
+  constexpr int PAIR = sizeof(T) == 2 ? 2 : 1;
+  const bool pair = PAIR == 2 && ((a.width | a.z_at | a.x_at | a.g_at | a.pitch | a.out_pitch) & 1) == 0 &&
+                    (((uintptr_t)a.proj | (uintptr_t)a.out) & 3) == 0;
+  const int v = pair ? 2 : 1;
+  const dim3 grid((a.width / v + GRU_THREADS - 1) / GRU_THREADS, chunks);
+  SRB_CUDA_CALL(srb_launch(pair ? gru_chunk_kernel<T, PAIR, false> : gru_chunk_kernel<T, 1, false>, grid, dim3(GRU_THREADS), 0, s, a));
   SRB_CUDA_CALL(srb_launch(gru_prefix_kernel, dim3(blocks, a.requests), dim3(GRU_THREADS), 0, s, a));
-  SRB_CUDA_CALL(srb_launch(gru_chunk_kernel<T, true>, dim3(chunks, blocks), dim3(GRU_THREADS), 0, s, a));
+  SRB_CUDA_CALL(srb_launch(pair ? gru_chunk_kernel<T, PAIR, true> : gru_chunk_kernel<T, 1, true>, grid, dim3(GRU_THREADS), 0, s, a));
   SRB_LAUNCH_CHECK("mingru");
   return SRB_OK;
 }

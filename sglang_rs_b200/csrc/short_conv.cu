@@ -211,6 +211,78 @@ __global__ void short_conv_single_kernel(const T* __restrict__ proj, const float
     if (j < taps - 1) kept[(size_t)j * s.channels] = u[j + 1];
 }
 
+// bfloat16 to bfloat16 in steps of many rows: a thread takes two neighbouring channels of CONV_ROWS rows, 4 bytes a load.
+template <int TAPS>
+__global__ void __launch_bounds__(128)
+short_conv_pair_kernel(const __nv_bfloat16* __restrict__ proj, const float* __restrict__ weight, const float* __restrict__ bias,
+                       const int* __restrict__ positions, const int* __restrict__ row_request, const int* __restrict__ cu_rows,
+                       const int* __restrict__ state_slots, const float* __restrict__ state, __nv_bfloat16* __restrict__ out, int rows,
+                       ConvShape s) {
+  constexpr int ROWS = CONV_ROWS;
+  srb_launch_dependents();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 2;
+  float w0[TAPS], w1[TAPS], b0 = 0.f, b1 = 0.f;
+  if (c < s.channels) {                                    // constants: ahead of the wait
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) { w0[j] = weight[(size_t)c * TAPS + j]; w1[j] = weight[(size_t)(c + 1) * TAPS + j]; }
+    if (bias) { b0 = bias[c]; b1 = bias[c + 1]; }
+  }
+  srb_grid_dependency_wait();
+  if (c >= s.channels) return;
+  const int row0 = blockIdx.y * ROWS;
+  __nv_bfloat162 u[ROWS + TAPS - 1];                        // the inputs of rows row0 - (TAPS - 1) .. row0 + ROWS - 1
+#pragma unroll
+  for (int k = 0; k < ROWS + TAPS - 1; ++k) {
+    const int row = row0 + k - (TAPS - 1);
+    u[k] = (row >= 0 && row < rows) ? *reinterpret_cast<const __nv_bfloat162*>(proj + (size_t)row * s.proj_pitch + c)
+                                    : __floats2bfloat162_rn(0.f, 0.f);
+  }
+  int pos[ROWS], request[ROWS];
+#pragma unroll
+  for (int r = 0; r < ROWS; ++r) {
+    const bool live = row0 + r < rows;
+    pos[r] = live ? positions[row0 + r] : -1;
+    request[r] = live ? row_request[row0 + r] : 0;
+  }
+  // rows in the middle of a request's rows of the step: every input is one of the step's
+  const bool inside = row0 + ROWS <= rows && pos[0] >= TAPS - 1 && request[0] == request[ROWS - 1] &&
+                      row0 - cu_rows[request[0]] >= TAPS - 1;
+#pragma unroll
+  for (int r = 0; r < ROWS; ++r) {
+    if (row0 + r >= rows) break;
+    float y0 = b0, y1 = b1;
+    if (inside) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const float2 v = __bfloat1622float2(u[r + j]);
+        y0 = fmaf(w0[j], v.x, y0);
+        y1 = fmaf(w1[j], v.y, y1);
+      }
+    } else if (pos[r] >= 0) {
+      const int ahead = row0 + r - cu_rows[request[r]];
+      const float* kept = state + (size_t)state_slots[request[r]] * s.slot_floats + c;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const int back = TAPS - 1 - j;
+        if (pos[r] - back < 0) continue;                   // zeros before the start of the sequence
+        float2 v = __bfloat1622float2(u[r + j]);
+        if (back > ahead) {
+          const float* at = kept + (size_t)(TAPS - 1 - (back - ahead)) * s.channels;
+          v = make_float2(at[0], at[1]);
+        }
+        y0 = fmaf(w0[j], v.x, y0);
+        y1 = fmaf(w1[j], v.y, y1);
+      }
+    } else {
+      y0 = y1 = 0.f;
+    }
+    __nv_bfloat162 y;
+    y.x = conv_result<__nv_bfloat16>(y0);
+    y.y = conv_result<__nv_bfloat16>(y1);
+    *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(row0 + r) * s.channels + c) = y;
+  }
+}
+
 template <typename T, typename O>
 static int launch_short_conv(const void* proj, const float* weight, const float* bias, const int* positions,
                              const int* row_request, const int* cu_rows, const int* state_slots, float* state, void* out,
@@ -236,7 +308,17 @@ static int launch_short_conv(const void* proj, const float* weight, const float*
 #define CONV_LAUNCH(TAPS, ROWS)                                                                                              \
   SRB_CUDA_CALL(srb_launch(short_conv_kernel<T, O, TAPS, ROWS>, grid, dim3(block), 0, st, (const T*)proj, weight, bias,     \
                            positions, row_request, cu_rows, state_slots, (const float*)state, (O*)out, rows, s))
-  if (s.taps == 4 && many) CONV_LAUNCH(4, CONV_ROWS);
+  bool pairs = false;
+  if constexpr (sizeof(T) == 2 && sizeof(O) == 2) {
+    pairs = many && s.taps >= 2 && s.taps <= 4 && s.channels % 2 == 0 && s.proj_pitch % 2 == 0 && (((uintptr_t)proj | (uintptr_t)out) & 3) == 0;
+    if (pairs) {
+      auto kernel = s.taps == 4 ? short_conv_pair_kernel<4> : (s.taps == 3 ? short_conv_pair_kernel<3> : short_conv_pair_kernel<2>);
+      SRB_CUDA_CALL(srb_launch(kernel, dim3((s.channels / 2 + block - 1) / block, grid.y), dim3(block), 0, st, (const __nv_bfloat16*)proj,
+                               weight, bias, positions, row_request, cu_rows, state_slots, (const float*)state, (__nv_bfloat16*)out, rows, s));
+    }
+  }
+  if (pairs) {}
+  else if (s.taps == 4 && many) CONV_LAUNCH(4, CONV_ROWS);
   else if (s.taps == 4) CONV_LAUNCH(4, 1);
   else if (s.taps == 3 && many) CONV_LAUNCH(3, CONV_ROWS);
   else if (s.taps == 2 && many) CONV_LAUNCH(2, CONV_ROWS);

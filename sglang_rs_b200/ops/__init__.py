@@ -1647,7 +1647,7 @@ def delta_gate_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, e
 # --------------------------------------------------------------------------- minGRU over a state per request
 
 #: tokens per chunk of :func:`mingru` (GRU_CHUNK of csrc/mingru.cu)
-MINGRU_CHUNK_TOKENS = 64
+MINGRU_CHUNK_TOKENS = 32
 
 
 @traced("mingru")
