@@ -57,9 +57,9 @@ __device__ __forceinline__ float delta_sigmoid(float v) { return 1.0f / (1.0f + 
 
 // grid (heads * column blocks, requests); NS lanes share a column of the state, each with NR of its entries (groups of four
 // consecutive ones, the groups dealt out over the lanes)
-template <typename T, typename X, int NS, int NR, bool CHANNEL>
-__global__ void __launch_bounds__(DELTA_THREADS) delta_scan_kernel(DeltaArgs a) {
-  constexpr int PB = DELTA_THREADS / NS, DP = NS * NR, WARPS = DELTA_THREADS / 32;
+template <typename T, typename X, int NS, int NR, bool CHANNEL, int THREADS>
+__global__ void __launch_bounds__(THREADS) delta_scan_kernel(DeltaArgs a) {
+  constexpr int PB = THREADS / NS, DP = NS * NR, WARPS = THREADS / 32;
   extern __shared__ __align__(16) float delta_smem[];
   float* q_s = delta_smem;                               // [DELTA_TOKENS][DP]
   float* k_s = q_s + DELTA_TOKENS * DP;
@@ -120,12 +120,12 @@ __global__ void __launch_bounds__(DELTA_THREADS) delta_scan_kernel(DeltaArgs a) 
       const float scale = (is_k ? 1.0f : a.q_scale) / sqrtf(srb_warp_sum(squares) + a.unit_eps);
       for (int d = lane; d < DP; d += 32) dst[d] *= scale;      // each lane its own entries
     }
-    for (int i = tid; i < tc * PB; i += DELTA_THREADS) {
+    for (int i = tid; i < tc * PB; i += THREADS) {
       const int t = i / PB, p = i - t * PB;
       v_s[i] = c0 + p < vdim ? srb_to_float(x[(size_t)(first + t0 + t) * a.channels + v_at + head * vdim + c0 + p]) : 0.f;
     }
     if (CHANNEL) {
-      for (int i = tid; i < tc * DP; i += DELTA_THREADS) {
+      for (int i = tid; i < tc * DP; i += THREADS) {
         const int t = i / DP, d = i - t * DP;
         float g = 1.f;
         if (d < dim)
@@ -217,41 +217,47 @@ static int delta_args(DeltaArgs& a, const void* x, const void* beta, long long b
   return SRB_OK;
 }
 
-template <typename T, typename X, int NS, int NR, bool CHANNEL>
+template <typename T, typename X, int NS, int NR, bool CHANNEL, int THREADS>
 static int launch_delta_scan(const DeltaArgs& a, cudaStream_t s) {
-  constexpr int PB = DELTA_THREADS / NS, DP = NS * NR;
+  constexpr int PB = THREADS / NS, DP = NS * NR;
   const dim3 grid(a.heads * ((a.vdim + PB - 1) / PB), a.requests);
   const size_t smem = (size_t)DELTA_TOKENS * (2 * DP + (CHANNEL ? DP : 1) + PB + 1) * sizeof(float);
-  auto kernel = delta_scan_kernel<T, X, NS, NR, CHANNEL>;
+  auto kernel = delta_scan_kernel<T, X, NS, NR, CHANNEL, THREADS>;
   if (smem > 48 * 1024) SRB_CUDA_CALL(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  SRB_CUDA_CALL(srb_launch(kernel, grid, dim3(DELTA_THREADS), smem, s, a));
+  SRB_CUDA_CALL(srb_launch(kernel, grid, dim3(THREADS), smem, s, a));
   SRB_LAUNCH_CHECK("delta_scan");
   return SRB_OK;
 }
 
+// `single_rows`: steps of decoded tokens read and write each state once, so more and smaller blocks, which all fit the chip
+// together at small batches, are quicker
 template <typename T, typename X>
-static int dispatch_delta_scan(const DeltaArgs& a, cudaStream_t s) {
+static int dispatch_delta_scan(const DeltaArgs& a, int single_rows, cudaStream_t s) {
   if (a.dim > 512) SRB_FAIL("delta_scan: heads of %d entries exceed 512", a.dim);
-  if (a.dim > 256) return a.channel_decay ? launch_delta_scan<T, X, 32, 16, true>(a, s) : launch_delta_scan<T, X, 32, 16, false>(a, s);
-  if (a.dim > 128) return a.channel_decay ? launch_delta_scan<T, X, 16, 16, true>(a, s) : launch_delta_scan<T, X, 16, 16, false>(a, s);
-  if (a.dim > 64) return a.channel_decay ? launch_delta_scan<T, X, 8, 16, true>(a, s) : launch_delta_scan<T, X, 8, 16, false>(a, s);
-  return a.channel_decay ? launch_delta_scan<T, X, 8, 8, true>(a, s) : launch_delta_scan<T, X, 8, 8, false>(a, s);
+#define DELTA_SCAN(NS, NR)                                                                                                  \
+  (a.channel_decay ? (single_rows ? launch_delta_scan<T, X, NS, NR, true, 128>(a, s) : launch_delta_scan<T, X, NS, NR, true, DELTA_THREADS>(a, s)) \
+                   : (single_rows ? launch_delta_scan<T, X, NS, NR, false, 128>(a, s) : launch_delta_scan<T, X, NS, NR, false, DELTA_THREADS>(a, s)))
+  if (a.dim > 256) return DELTA_SCAN(32, 16);
+  if (a.dim > 128) return DELTA_SCAN(16, 16);
+  if (a.dim > 64) return DELTA_SCAN(8, 16);
+  return DELTA_SCAN(8, 8);
+#undef DELTA_SCAN
 }
 
 // x: float [rows, channels] (what srb_short_conv wrote); beta, decay: columns of projections of `dtype`; out: float [rows,
-// heads * vdim]
+// heads * vdim]; `single_rows`: every request of the step brings one row (a hint; the results are the same)
 extern "C" int srb_delta_scan(const float* x, const void* beta, long long beta_pitch, const void* decay, long long decay_pitch,
                               const float* a_log, const float* dt_bias, const int* positions, const int* cu_rows,
                               const int* state_slots, float* state, long long slot_floats, float* out, int rows, int requests,
                               int heads, int kv_heads, int dim, int vdim, int taps, int channel_decay, float unit_eps,
-                              int write_state, int dtype, void* stream) {
+                              int write_state, int single_rows, int dtype, void* stream) {
   if (rows <= 0 || requests <= 0) return SRB_OK;
   DeltaArgs a;
   if (delta_args(a, x, beta, beta_pitch, decay, decay_pitch, a_log, dt_bias, positions, cu_rows, state_slots, state, slot_floats, out,
                  requests, heads, kv_heads, dim, vdim, taps, channel_decay, unit_eps, write_state) != SRB_OK)
     return SRB_ERR_INVALID;
-  if (dtype == SRB_DTYPE_F32) return dispatch_delta_scan<float, float>(a, (cudaStream_t)stream);
-  if (dtype == SRB_DTYPE_BF16) return dispatch_delta_scan<__nv_bfloat16, float>(a, (cudaStream_t)stream);
+  if (dtype == SRB_DTYPE_F32) return dispatch_delta_scan<float, float>(a, single_rows, (cudaStream_t)stream);
+  if (dtype == SRB_DTYPE_BF16) return dispatch_delta_scan<__nv_bfloat16, float>(a, single_rows, (cudaStream_t)stream);
   SRB_FAIL("delta_scan: unknown dtype %d", dtype);
 }
 

@@ -400,7 +400,7 @@ __global__ void norm_add_norm_kernel(float* __restrict__ residual, const T* __re
 // ITEMS of them, all loads of a thread in flight together.  Widths that are multiples of four, rows on 16-byte borders (of
 // floats), no `extra`.
 template <typename T, int ITEMS, bool PARTS>
-__global__ void __launch_bounds__(256, ITEMS <= 2 ? 4 : 1)
+__global__ void __launch_bounds__(ITEMS == 1 ? 1024 : 256, ITEMS == 1 ? 1 : (ITEMS == 2 ? 4 : 1))
 norm_add_norm_vec_kernel(float* __restrict__ residual, const T* __restrict__ delta, const float* __restrict__ delta_f32,
                          NormSpec inner, NormSpec outer, T* __restrict__ out, size_t out_pitch, const int* __restrict__ row_index,
                          int width, int write_residual, const float* __restrict__ addend, int num_parts, size_t part_stride) {
@@ -431,18 +431,19 @@ norm_add_norm_vec_kernel(float* __restrict__ residual, const T* __restrict__ del
     }
   }
   if (PARTS) {
-    // partial sums of a product cut along K, added in part order, the loads of four parts in flight
-    for (int first = 0; first < num_parts; first += 4) {
+    // partial sums of a product cut along K, added in part order, the loads of several parts in flight
+    constexpr int AHEAD = ITEMS == 1 ? 8 : 4;
+    for (int first = 0; first < num_parts; first += AHEAD) {
 #pragma unroll
       for (int it = 0; it < ITEMS; ++it) {
         const int i = threadIdx.x * 4 + it * step;
         if (i >= width) break;
-        float4 p[4];
+        float4 p[AHEAD];
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+        for (int j = 0; j < AHEAD; ++j)
           if (first + j < num_parts) p[j] = load4(delta_f32 + (first + j) * part_stride + src + i);
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+        for (int j = 0; j < AHEAD; ++j)
           if (first + j < num_parts) { d[it].x += p[j].x; d[it].y += p[j].y; d[it].z += p[j].z; d[it].w += p[j].w; }
       }
     }
@@ -496,7 +497,7 @@ static int launch_norm_add_norm_vec(float* residual, const void* delta, const fl
                                     const float* addend, int num_parts, long long part_stride, cudaStream_t s) {
   const int quads = width / 4;
   // few rows: as many threads as the row has pieces; many: two pieces a thread
-  int items = quads <= 256 && rows <= 64 ? 1 : (quads <= 512 ? 2 : (quads <= 1024 ? 4 : 8));
+  const int items = quads <= 1024 && rows <= 64 ? 1 : (quads <= 512 ? 2 : (quads <= 1024 ? 4 : 8));
   const int threads = ((quads + items - 1) / items + 31) / 32 * 32;
 #define SRB_NORM_VEC(ITEMS)                                                                                                    \
   SRB_CUDA_CALL(srb_launch(num_parts > 0 ? norm_add_norm_vec_kernel<T, ITEMS, true> : norm_add_norm_vec_kernel<T, ITEMS, false>, dim3(rows), dim3(threads), 0, s, residual, (const T*)delta,    \

@@ -1578,20 +1578,21 @@ def _delta_args(qkv, beta, decay, a_log, dt_bias, positions, cu_rows, state_slot
 def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
                positions: torch.Tensor, cu_rows: torch.Tensor, state_slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
                num_requests: int, *, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, channel_decay: bool, unit_eps: float,
-               read_only: bool = False) -> None:
+               read_only: bool = False, single_rows: bool = False) -> None:
     """The gated delta rule, token by token from each request's state, all in 32-bit: per head (with unit vectors q, k and
     q times dim^-1/2) S <- g S, u = sigmoid(beta) (v - S^T k), S <- S + k u^T, out = S^T q, where g =
     exp(-exp(a_log) softplus(decay + dt_bias)) is one number per head or, with ``channel_decay``, one per row of S.
 
     ``qkv`` float32 [rows, channels]: q (kv_heads * dim) | k (kv_heads * dim) | v (heads * vdim), as :func:`short_conv` wrote
     them; ``beta`` [rows, heads] and ``decay`` [rows, heads (* dim)]: columns of projections; ``state`` float32 [slots,
-    ``delta_slot_floats``]; ``out`` float32 [rows, heads * vdim].  ``unit_eps`` stands beside the sum of squares of q and k."""
+    ``delta_slot_floats``]; ``out`` float32 [rows, heads * vdim].  ``unit_eps`` stands beside the sum of squares of q and k.
+    ``single_rows``: every request brings one row (smaller blocks, the same results)."""
     _need(qkv, "qkv", torch.float32)
     args = _delta_args(qkv, beta, decay, a_log, dt_bias, positions, cu_rows, state_slots, state, out, heads, kv_heads, dim, vdim, taps,
                        channel_decay)
     lib = load_library("delta")
     _check(lib, lib.srb_delta_scan(*args, _ptr(out), qkv.shape[0], int(num_requests), heads, kv_heads, dim, vdim, taps,
-                                   int(channel_decay), ctypes.c_float(unit_eps), int(not read_only), dtype_code(beta.dtype), _stream()))
+                                   int(channel_decay), ctypes.c_float(unit_eps), int(not read_only), int(single_rows), dtype_code(beta.dtype), _stream()))
 
 
 def delta_chunks_takes(dtype: torch.dtype, dim: int, vdim: int) -> bool:

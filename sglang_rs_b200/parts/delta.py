@@ -177,9 +177,10 @@ class GatedDeltaRule(Stackable):
         known = len(counts) == ctx.num_requests
         chunked = known and max(counts, default=0) > self.CHUNKED_FROM and ops.delta_chunks_takes(proj.dtype, self.dim, self.vdim)
         qkv = torch.empty((rows, self.channels), dtype=proj.dtype if chunked else torch.float32, device=proj.device)
+        single = known and all(count == 1 for count in counts)
         ops.short_conv(proj[:, :self.channels], self.conv, None, ctx.positions, ctx.row_request, ctx.cu_rows, ctx.state_slots,
                        cache.state, qkv, ctx.num_requests, read_only=not cache.writable,
-                       single_rows=known and all(count == 1 for count in counts))
+                       single_rows=single)
         o = torch.empty((rows, vv), dtype=torch.float32, device=proj.device)
         args = (qkv, beta, decay, self.a_log, self.dt_bias, ctx.positions, ctx.cu_rows, ctx.state_slots, cache.state, o,
                 ctx.num_requests)
@@ -187,5 +188,5 @@ class GatedDeltaRule(Stackable):
         if chunked:
             ops.delta_chunks(*args, sum(-(-count // ops.DELTA_CHUNK_TOKENS) for count in counts), **options)
         else:
-            ops.delta_scan(*args, **options)
+            ops.delta_scan(*args, single_rows=single, **options)
         ops.delta_gate_norm(o, gate, self.norm, self.eps, out, silu=self.gate == "silu", scale=scale, heads=self.heads)

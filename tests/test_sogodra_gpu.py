@@ -79,7 +79,7 @@ def test_short_convolution_over_inputs_in_slots(dtype, taps):
         for i, s in enumerate(slots):
             proj[cu[i]:cu[i + 1], at:at + channels] = sequences[s][starts[i]:starts[i] + counts[i]]
         on = proj.to(DEV, dtype)
-        for out_dtype in {torch.float32, dtype}:
+        for out_dtype in [torch.float32] + [dtype] * (dtype != torch.float32):      # (the one that keeps the inputs last)
             for read_only in (True, False):
                 if not read_only and out_dtype != dtype:
                     continue
@@ -141,7 +141,10 @@ def run_delta(kernel, w, rows, counts, starts, slots, state, sizes, channels, dt
             dev(slots), state, out, len(counts)]
     if kernel is ops.delta_chunks:
         args.append(sum(-(-c // ops.DELTA_CHUNK_TOKENS) for c in counts))
-    kernel(*args, channel_decay=channels, unit_eps=1e-6, read_only=read_only, **sizes)
+    options = dict(channel_decay=channels, unit_eps=1e-6, **sizes)
+    if kernel is ops.delta_scan and max(counts) == 1:
+        options["single_rows"] = True
+    kernel(*args, read_only=read_only, **options)
     return cu, out
 
 
@@ -188,6 +191,7 @@ def delta_over_two_steps(kernel, heads, kv_heads, dim, vdim, taps, channels, dty
 def test_gated_delta_rule_token_by_token(heads, kv_heads, dim, vdim, taps, channels, dtype):
     from sglang_rs_b200 import ops
     delta_over_two_steps(ops.delta_scan, heads, kv_heads, dim, vdim, taps, channels, dtype, torch.float32, [45, 1, 33, 1], [2, 38, 1, 50], 3e-5)
+    delta_over_two_steps(ops.delta_scan, heads, kv_heads, dim, vdim, taps, channels, dtype, torch.float32, [1, 1, 33, 2], [1, 1, 1, 1], 3e-5)
 
 
 @pytest.mark.parametrize("channels", [False, True])
