@@ -1034,7 +1034,7 @@ __global__ void __launch_bounds__(128 * MT) delta_chunk_walk_kernel(DeltaArgs a,
         u[nt][e] = uv[nt][e];
         o[nt][e] = u_rest[0][nt][e] = u_rest[1][nt][e] = o_rest[0][nt][e] = o_rest[1][nt][e] = 0.f;
       }
-#pragma unroll 2
+#pragma unroll 4
     for (int kk = 0; kk < DP / 16; ++kk) {
       unsigned sh[4], sl[4], w[2][4], q[2][4];
       const __nv_bfloat16* at = ss + (tile * 16 + (matrix & 1) * 8 + inner) * XP + kk * 16 + (matrix >> 1) * 8;
