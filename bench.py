@@ -954,7 +954,7 @@ def sogodra_layers(width: int, count: int):
     heads = width // 128
     rule = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4}
     attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 1.0 / math.sqrt(128),
-                 "mask": {"size": 1024}, "rot": {"base": 50000.0, "dims": 64, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+                 "mask": {"size": 1024}, "rot": {"base": 50000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 6.0, "original": 4096}}}
     dense = {"kind": "dense", "ff": 3 * width, "limit": 7.0}
     kinds = [("delta", rule), ("parallel", {"left": attention, "right": rule, "left_scale": 0.8, "right_scale": 1.2}),
              ("mingru", {"width": width}), ("delta", rule)]

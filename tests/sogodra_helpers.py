@@ -72,7 +72,7 @@ SMALL_B = config(40, 70, [
 ], eps=1e-6)
 #: no size is a multiple of eight (columns off 16-byte borders everywhere); a window of one (a row sees itself only)
 SMALL_C = config(36, 50, [
-    layer(parallel(attention(3, 1, 10, 6, window=1, rot_dims=6), delta_sizes(2, 2, 7, 11, 3), 0.8, 1.1), 30, 1.5),
+    layer(parallel(attention(3, 1, 10, 6, window=1, rot_dims=6), delta_sizes(2, 2, 7, 11, 3), 0.85, 1.15), 30, 1.4),
     layer(delta(3, 1, 9, 5, 4), 20, 0.6),
     layer(mingru(21), 18, 1.0),
     layer(parallel(attention(2, 2, 6, 10, window=33, rot_dims=2, scaling=RAMP), delta_sizes(5, 5, 6, 3, 2), 1.2, 0.7)),
@@ -86,6 +86,10 @@ SMALL_D = config(64, 100, [
     layer(delta(3, 1, 40, 16, 3), 64, 1.3),
     layer(parallel(attention(2, 1, 64, 64, window=150), delta_sizes(1, 1, 104, 128, 2), 1.4, 0.6)),
 ])
+#: layers over a state only: no pages at all
+SMALL_E = config(32, 60, [layer(delta(6, 2, 8, 8, 2), 40, 1.0), layer(mingru(16), 24, 1.4), layer(delta(2, 1, 24, 40, 4))])
+#: more query heads on one kv head than a block has warps, one layer
+SMALL_F = config(56, 40, [layer(parallel(attention(34, 1, 8, 12, window=20, rot_dims=4), delta_sizes(3, 1, 16, 8, 4), 0.9, 0.8), 40, 1.0)])
 #: per configuration the ranks of the decays' and the gates' thin pairs
 RANKS = {48: (7, 13), 40: (8, 3), 36: (5, 1), 64: (24, 16)}
 

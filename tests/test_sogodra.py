@@ -10,7 +10,7 @@ import torch
 import plain_sogodra as ps
 import sogodra_helpers as sh
 
-ALL = [sh.SMALL_A, sh.SMALL_B, sh.SMALL_C, sh.SMALL_D]
+ALL = [sh.SMALL_A, sh.SMALL_B, sh.SMALL_C, sh.SMALL_D, sh.SMALL_E, sh.SMALL_F]
 
 
 def build(doc):
@@ -22,7 +22,7 @@ def build(doc):
     return config, entry.build_model(config)
 
 
-@pytest.mark.parametrize("doc", ALL, ids="abcd")
+@pytest.mark.parametrize("doc", ALL, ids="abcdef")
 def test_the_reader_takes_every_size_from_the_document(doc):
     config, model = build(doc)
     assert config.width == doc["width"] and config.vocab == doc["vocab"] and len(config.layers) == len(doc["layers"])

@@ -393,7 +393,7 @@ def test_the_stream_with_a_normed_term_added_is_handed_on_rounded(dtype):
 
 # ------------------------------------------------------------------------------ whole models
 @pytest.mark.parametrize("dtype_name,stored,tolerance", DTYPES)
-@pytest.mark.parametrize("doc", [sh.SMALL_A, sh.SMALL_B, sh.SMALL_C, sh.SMALL_D], ids="abcd")
+@pytest.mark.parametrize("doc", [sh.SMALL_A, sh.SMALL_B, sh.SMALL_C, sh.SMALL_D, sh.SMALL_E, sh.SMALL_F], ids="abcdef")
 def test_prompts_tails_portions_and_mixed_batches(tmp_path, doc, dtype_name, stored, tolerance):
     folder = sh.make_folder(tmp_path, "m", doc, seed=5, dtype=stored)
     requests = sh.random_requests(doc, (1, 2, 23, 64, 65, 150, 131), seed=3)
@@ -407,7 +407,8 @@ def test_prompts_tails_portions_and_mixed_batches(tmp_path, doc, dtype_name, sto
         worst[name] = rh.worst_error(rows, expected)
         whole_model_close(rows, expected, dtype_name, name)
         if name == "mixed":
-            assert any(len(owners) > 1 for owners in session.page_owners.values()), "no page was used again"
+            paged = any(entry["type"] == "parallel" for entry in doc["layers"])
+            assert any(len(owners) > 1 for owners in session.page_owners.values()) == paged, "no page was used again"
             assert len(requests) > session.cache.max_requests, "no state slot was used again"
     print(doc["width"], dtype_name, worst)
 
