@@ -12,7 +12,8 @@ zeroed when it is assigned, given back when the request ends).
 Here a page is the unit (not a token slot), pages are reference-counted so that a prefix
 tree can share full pages between requests, and layers are grouped by need: all layers
 that keep every key share one block table per request; layers that keep only a window
-share another, whose pages are given back as soon as the window has passed them.
+share another, whose pages are given back as soon as the window has passed them (a window
+may keep a sequence's first tokens visible: the pages that hold them stay).
 """
 from __future__ import annotations
 
@@ -25,7 +26,7 @@ import torch
 
 from ..parts.base import CacheNeed, JointNeed, PagedKV, RequestState, simple_needs
 
-GroupKey = Hashable        # ("kv", window) with window None for "all keys"
+GroupKey = Hashable        # ("kv", window) with window None for "all keys", or ("kv", window, kept first tokens)
 
 
 class OutOfPages(RuntimeError):
@@ -45,7 +46,7 @@ def _core_library():
         from ..csrc.build import load_library
         lib = load_library("host_core")
         lib.hc_create.restype = ctypes.c_void_p
-        lib.hc_create.argtypes = [ctypes.c_int, ctypes.c_int, ctypes.c_void_p, ctypes.c_void_p, ctypes.c_int]
+        lib.hc_create.argtypes = [ctypes.c_int, ctypes.c_int, ctypes.c_void_p, ctypes.c_void_p, ctypes.c_void_p, ctypes.c_int]
         lib.hc_destroy.argtypes = [ctypes.c_void_p]
         for name in ("hc_free_count", "hc_allocate", "hc_retain", "hc_release", "hc_refcount", "hc_free_list", "hc_open",
                      "hc_close", "hc_live_count", "hc_free_state_count", "hc_length", "hc_state_slot", "hc_table_length",
@@ -74,11 +75,12 @@ def _message(lib) -> str:
 class _Core:
     """Owner of one set of C++ books."""
 
-    def __init__(self, page_size: int, windows: Sequence[int], num_pages: Sequence[int], max_requests: int):
+    def __init__(self, page_size: int, windows: Sequence[int], num_pages: Sequence[int], max_requests: int,
+                 keep_first: Optional[Sequence[int]] = None):
         self.lib = _core_library()
         self.page_size = int(page_size)
-        w, n = _ints(windows), _ints(num_pages)
-        self.pointer = self.lib.hc_create(int(page_size), len(w), _pointer(w), _pointer(n), int(max_requests))
+        w, n, k = _ints(windows), _ints(num_pages), _ints(keep_first if keep_first is not None else [0] * len(windows))
+        self.pointer = self.lib.hc_create(int(page_size), len(w), _pointer(w), _pointer(k), _pointer(n), int(max_requests))
         if not self.pointer:
             raise ValueError("a page pool needs at least one page, a positive page size and room for a request")
         self.pointer = ctypes.c_void_p(self.pointer)
@@ -211,7 +213,7 @@ class RequestCache:
 
 
 def group_key(need: PagedKV) -> GroupKey:
-    return ("kv", need.window)
+    return ("kv", need.window, need.keep_first) if need.keep_first else ("kv", need.window)
 
 
 class CacheManager:
@@ -232,18 +234,20 @@ class CacheManager:
         self.needs = list(needs)
         default_pages = max(1, -(-int(max_tokens) // self.page_size))
         self.windows: Dict[GroupKey, Optional[int]] = {}
+        #: first tokens of a sequence that stay visible behind a group's window
+        self.keep_first: Dict[GroupKey, int] = {}
         counts: Dict[GroupKey, int] = {}
         for need in simple_needs(self.needs):
             if isinstance(need, PagedKV):
                 key = group_key(need)
                 if key not in counts:
                     counts[key] = (pages_per_group or {}).get(key, default_pages)
-                    self.windows[key] = need.window
+                    self.windows[key], self.keep_first[key] = need.window, need.keep_first
         for key, count in counts.items():
             if count <= 0:
                 raise ValueError("a page pool needs at least one page")
         self._core = _Core(self.page_size, [self.windows[key] or 0 for key in counts], list(counts.values()),
-                           self.max_requests)
+                           self.max_requests, [self.keep_first[key] for key in counts])
         self._lib, self._pointer = self._core.lib, self._core.pointer
         self._group_index: Dict[GroupKey, int] = {key: g for g, key in enumerate(counts)}
         self._group_keys: List[GroupKey] = list(counts)
@@ -342,7 +346,7 @@ class CacheManager:
         self.live.pop(handle.request_id, None)
 
     def first_kept_position(self, key: GroupKey, length: int) -> int:
-        """The first position whose key a query at position >= ``length`` can still see."""
+        """The first position whose key a query at position >= ``length`` can still see, the kept first tokens aside."""
         window = self.windows[key]
         return 0 if window is None else max(0, length - window + 1)
 

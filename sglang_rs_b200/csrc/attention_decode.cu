@@ -24,6 +24,8 @@
 #include "attention_kernels.cuh"
 #include "mma_helpers.cuh"
 
+#include <algorithm>
+
 SRB_DEFINE_LAST_ERROR()
 SRB_DEFINE_PDL_SWITCH()
 
@@ -34,21 +36,42 @@ SRB_DEFINE_PDL_SWITCH()
 
 struct DecodeParams {
   AttnParams a;              // split_size is unused; max_splits = blocks per (row, kv head)
-  float scale_log2;
+  float scale_log2;          // scores times this are in units of log2; with a cap: scores times this are 2 s / softcap * log2 e
+  float cap_log2;            // softcap * log2 e, or 0
 };
 
-__device__ __forceinline__ void decode_units(const AttnParams& p, int pos, int& first_unit, int& units, int& lo,
+// `units` counts what the row walks: `kept` units ahead of the window that hold kept first tokens, then those from
+// first_unit on (srb_piece gives the number of each).
+__device__ __forceinline__ void decode_units(const AttnParams& p, int pos, int& first_unit, int& kept, int& units, int& lo,
                                              int& hi) {
   lo = srb_first_visible(pos, p.window, p.chunk);
   hi = pos + 1;
   first_unit = lo / DEC_UNIT;
-  units = (hi - 1) / DEC_UNIT - first_unit + 1;
+  kept = srb_kept_pieces(p.keep_first, DEC_UNIT, first_unit);
+  units = (hi - 1) / DEC_UNIT - first_unit + 1 + kept;
+}
+
+// One warp: a head's two maps, [2][D] floats in shared memory, become its result: (a_1 - lambda a_2), divided by its root mean
+// square, times map_scale.
+template <int D>
+__device__ __forceinline__ void join_maps(const float* maps, __nv_bfloat16* out, const AttnParams& p, int lane) {
+  float o[D / 32], squares = 0.f;
+#pragma unroll
+  for (int j = 0; j < D / 32; ++j) {
+    o[j] = maps[lane + 32 * j] - p.map_lambda * maps[D + lane + 32 * j];
+    squares += o[j] * o[j];
+  }
+  const float factor = p.map_scale / sqrtf(srb_warp_sum(squares) / (float)D + p.map_eps);
+#pragma unroll
+  for (int j = 0; j < D / 32; ++j) out[lane + 32 * j] = __float2bfloat16_rn(o[j] * factor);
 }
 
 // CLUSTER: the blocks of a (row, kv head) form a thread-block cluster (at most 8 of them) and merge
 // their partial results through each other's shared memory; otherwise through global memory, where
 // the block that arrives last merges.
-template <int D, bool CLUSTER>
+// MAPS: two maps per head (AttnParams); the rows of the tile are the maps, 2 h + t, each with its half of the head's query row
+// and zeros elsewhere, and whoever merges joins a head's two maps.
+template <int D, bool CLUSTER, bool MAPS>
 __global__ void __launch_bounds__(DEC_WARPS * 32, 3)
 decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pool,
                         const __nv_bfloat16* __restrict__ v_pool, float* __restrict__ part_acc,
@@ -70,16 +93,16 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
   srb_mark(SRB_MARK_DECODE_ATTENTION, 0);
   srb_launch_dependents();
   const int pos = p.positions[row];
-  int first_unit, units, lo, hi;
-  decode_units(p, pos, first_unit, units, lo, hi);
+  int first_unit, kept_units, units, lo, hi;
+  decode_units(p, pos, first_unit, kept_units, units, lo, hi);
   const int per_split = (units + p.max_splits - 1) / p.max_splits;
   const int count = (units + per_split - 1) / per_split;           // splits that have work
   if (!CLUSTER && split >= count) {
     srb_grid_dependency_wait();
     return;
   }
-  const int unit_begin = first_unit + split * per_split;
-  const int unit_end = min(first_unit + units, unit_begin + per_split);     // a block without work: begin >= end
+  const int unit_begin = split * per_split;                                 // in the order of the walk
+  const int unit_end = min(units, unit_begin + per_split);                  // a block without work: begin >= end
   const int groups = p.n_q / p.n_kv;
   const int request = p.row_request[row];
   const int page_shift = (p.page_size & (p.page_size - 1)) == 0 ? __ffs(p.page_size) - 1 : -1;
@@ -87,12 +110,13 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
   __nv_bfloat16* warp_smem = reinterpret_cast<__nv_bfloat16*>(smem_raw) + (size_t)warp * DEC_STAGES * STAGE_ELEMS;
 
   // copies of one unit: lanes 0..15 look up the page of one key each, the row offsets travel by shuffle
-  auto issue = [&](int unit, int stage) {
+  auto issue = [&](int walked, int stage) {
+    const int unit = srb_piece(walked, kept_units, first_unit);
     __nv_bfloat16* ks = warp_smem + (size_t)stage * STAGE_ELEMS;
     __nv_bfloat16* vs = ks + DEC_KEYS * D;
     long long my_offset = -1;
     const int abs_key = unit * DEC_UNIT + warp * DEC_KEYS + (lane & (DEC_KEYS - 1));
-    if (abs_key >= lo && abs_key < hi) {
+    if (abs_key < hi && (abs_key >= lo || abs_key < p.keep_first)) {
       const int logical = page_shift >= 0 ? abs_key >> page_shift : abs_key / p.page_size;
       const int within = page_shift >= 0 ? abs_key & (p.page_size - 1) : abs_key % p.page_size;
       const int page = p.block_table[(size_t)request * p.table_stride + logical];
@@ -115,7 +139,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
     cp_async_commit();
   };
   const bool has_work = unit_begin < unit_end;
-  const bool first_unit_is_old = (unit_begin + 1) * DEC_UNIT <= pos;
+  const bool first_unit_is_old = (srb_piece(unit_begin, kept_units, first_unit) + 1) * DEC_UNIT <= pos;
   if (has_work && first_unit_is_old) issue(unit_begin, 0);
   srb_grid_dependency_wait();
   srb_mark(SRB_MARK_DECODE_ATTENTION, 1);
@@ -126,6 +150,19 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
   {
     const int r0 = lane >> 2, r1 = r0 + 8, col0 = (lane & 3) * 2;
     const __nv_bfloat16* qrow = q + ((size_t)row * p.n_q + (size_t)kv_head * groups) * D;
+    if (MAPS) {
+      // rows 2 h + t: the half t of head h's query row, zeros in the other half
+      const __nv_bfloat16* mrow = q + ((size_t)row * p.n_q + (size_t)kv_head * groups) / 2 * D;
+#pragma unroll
+      for (int kk = 0; kk < KSTEPS; ++kk) {
+        const int d0 = kk * 16 + col0, t = kk >= KSTEPS / 2;
+        const bool mine0 = r0 < groups && (r0 & 1) == t, mine1 = r1 < groups && (r1 & 1) == t;
+        qa[kk][0] = mine0 ? *reinterpret_cast<const unsigned*>(mrow + (size_t)(r0 >> 1) * D + d0) : 0u;
+        qa[kk][1] = mine1 ? *reinterpret_cast<const unsigned*>(mrow + (size_t)(r1 >> 1) * D + d0) : 0u;
+        qa[kk][2] = mine0 ? *reinterpret_cast<const unsigned*>(mrow + (size_t)(r0 >> 1) * D + d0 + 8) : 0u;
+        qa[kk][3] = mine1 ? *reinterpret_cast<const unsigned*>(mrow + (size_t)(r1 >> 1) * D + d0 + 8) : 0u;
+      }
+    } else
 #pragma unroll
     for (int kk = 0; kk < KSTEPS; ++kk) {
       const int d0 = kk * 16 + col0;
@@ -154,8 +191,8 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
     __syncwarp();
     const __nv_bfloat16* ks = warp_smem + (size_t)stage * STAGE_ELEMS;
     const __nv_bfloat16* vs = ks + DEC_KEYS * D;
-    const int key_base = unit * DEC_UNIT + warp * DEC_KEYS;
-    if (key_base < hi && key_base + DEC_KEYS > lo) {         // this warp's 16 keys are not all outside
+    const int key_base = srb_piece(unit, kept_units, first_unit) * DEC_UNIT + warp * DEC_KEYS;
+    if (key_base < hi && (key_base + DEC_KEYS > lo || key_base < p.keep_first)) {         // this warp's 16 keys are not all outside
       float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
       for (int kk = 0; kk < KSTEPS; ++kk) {
@@ -166,14 +203,22 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
         mma_bf16(s[0], qa[kk], b0, b1);
         mma_bf16(s[1], qa[kk], b2, b3);
       }
-      const bool all_visible = key_base >= lo && key_base + DEC_KEYS <= hi;
+      const bool all_visible = key_base + DEC_KEYS <= hi && (key_base >= lo || key_base + DEC_KEYS <= p.keep_first);
+      if (dp.cap_log2 > 0.f) {
+        // 2 s / softcap in units of log2 -> softcap * tanh(s / softcap) in units of log2
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[t][e] = dp.cap_log2 * (1.0f - __fdividef(2.0f, exp2f(s[t][e] * dp.scale_log2) + 1.0f));
+      }
+      const float to_log2 = dp.cap_log2 > 0.f ? 1.f : dp.scale_log2;
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int t = 0; t < 2; ++t) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int abs_key = key_base + t * 8 + col + (e & 1);
-          const float v = (all_visible || (abs_key >= lo && abs_key < hi)) ? s[t][e] * dp.scale_log2 : -INFINITY;
+          const float v = (all_visible || (abs_key < hi && (abs_key >= lo || abs_key < p.keep_first))) ? s[t][e] * to_log2 : -INFINITY;
           s[t][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
         }
@@ -279,6 +324,41 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
     // Every block of the cluster takes a slice of the (head, element) pairs and merges the blocks'
     // results for it, in block order, reading the others' shared memory.
     srb_cluster_sync();
+    if (MAPS) {
+      // whole heads per block: the join needs a head's two maps and all their entries
+      float* joined = mine + groups * (D + 2);             // [2][D] of the head at hand
+      for (int pair = (int)srb_cluster_rank(); pair < groups / 2; pair += p.max_splits) {
+        for (int i = threadIdx.x; i < 2 * D; i += blockDim.x) {
+          const float* base = mine + (2 * pair + i / D) * (D + 2);
+          float m = -INFINITY, acc = 0.f, l = 0.f;
+          float ms[8], ls[8], as[8];
+#pragma unroll
+          for (int b = 0; b < 8; ++b) {
+            if (b < p.max_splits) {
+              ms[b] = srb_load_peer_shared(base + D, b);
+              ls[b] = srb_load_peer_shared(base + D + 1, b);
+              as[b] = srb_load_peer_shared(base + i % D, b);
+              m = fmaxf(m, ms[b]);
+            }
+          }
+#pragma unroll
+          for (int b = 0; b < 8; ++b) {
+            if (b < p.max_splits) {
+              const float weight = ls[b] > 0.f ? exp2f(ms[b] - m) : 0.f;    // a block without keys adds nothing
+              acc += as[b] * weight;
+              l += ls[b] * weight;
+            }
+          }
+          joined[i] = l > 0.f ? acc / l : 0.f;
+        }
+        __syncthreads();
+        if (warp == 0) join_maps<D>(joined, out + (size_t)row * p.out_pitch + ((size_t)kv_head * groups / 2 + pair) * D, p, lane);
+        __syncthreads();                                   // the buffer is used again for the next head
+      }
+      srb_cluster_sync();                                  // nobody leaves while its memory may still be read
+      srb_mark(SRB_MARK_DECODE_ATTENTION, 2);
+      return;
+    }
     const int blocks = p.max_splits;                       // = cluster size
     const int total = groups * D;
     const int per_block = (total + blocks - 1) / blocks;
@@ -364,6 +444,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
     if (lane == 0) weights[head * (count + 1) + count] = (p.gates ? p.gates[(size_t)row * p.n_q + q_head] * p.out_scale : p.out_scale) / l;
   }
   __syncthreads();
+  float* joined = weights + groups * (count + 1);          // MAPS: [groups][D], the maps' results
   // four (head, element) pairs per thread and eight splits at a time: 32 loads in flight, added in split order
   const int total = groups * D;
   for (int i0 = threadIdx.x; i0 < total; i0 += 4 * blockDim.x) {
@@ -394,14 +475,20 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
       const int i = i0 + q * (int)blockDim.x;
       if (i < total) {
         const int head = i / D, e = i % D;
-        out[(size_t)row * p.out_pitch + ((size_t)kv_head * groups + head) * D + e] = __float2bfloat16_rn(acc[q] * w[q][count]);
+        if (MAPS) joined[i] = acc[q] * w[q][count];
+        else out[(size_t)row * p.out_pitch + ((size_t)kv_head * groups + head) * D + e] = __float2bfloat16_rn(acc[q] * w[q][count]);
       }
     }
+  }
+  if (MAPS) {
+    __syncthreads();
+    for (int pair = warp; pair < groups / 2; pair += DEC_WARPS)
+      join_maps<D>(joined + (size_t)2 * pair * D, out + (size_t)row * p.out_pitch + ((size_t)kv_head * groups / 2 + pair) * D, p, lane);
   }
   srb_mark(SRB_MARK_DECODE_ATTENTION, 2);
 }
 
-template <int D>
+template <int D, bool MAPS>
 static int launch_decode(const void* q, const void* k_pool, const void* v_pool, void* out, float* part_acc,
                          float* part_ml, int* counters, const DecodeParams& dp, int rows, cudaStream_t s) {
   const int groups = dp.a.n_q / dp.a.n_kv;
@@ -411,9 +498,11 @@ static int launch_decode(const void* q, const void* k_pool, const void* v_pool, 
   // more than it saves); the merge needs room for one more [head][D + 2]
   const bool cluster = dp.a.max_splits > 1 && dp.a.max_splits <= 8 &&
                        (long long)rows * dp.a.n_kv * dp.a.max_splits <= 3 * srb_sm_count();
-  const size_t merge = (size_t)(DEC_WARPS + 1) * groups * (D + 2) * sizeof(float);
-  const size_t smem = cluster && merge > keys ? merge : keys;
-  auto kernel = cluster ? decode_attention_kernel<D, true> : decode_attention_kernel<D, false>;
+  const size_t merge = ((size_t)(DEC_WARPS + 1) * groups * (D + 2) + (MAPS ? 2 * D : 0)) * sizeof(float);
+  // the last block's merge: a weight per (head, split) and, with two maps, the maps' results
+  const size_t last = (size_t)groups * (dp.a.max_splits + 1 + (MAPS ? D : 0)) * sizeof(float);
+  const size_t smem = std::max(keys, cluster ? merge : last);
+  auto kernel = cluster ? decode_attention_kernel<D, true, MAPS> : decode_attention_kernel<D, false, MAPS>;
   if (smem > 48 * 1024)
     SRB_CUDA_CALL(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   dim3 grid(dp.a.max_splits, dp.a.n_kv, rows);
@@ -437,12 +526,15 @@ extern "C" int srb_decode_attention_supports(int n_q, int n_kv, int head_dim, in
 // `sinks` (float [n_q], or null): exp(sink_h) joins the softmax's denominator of head h, once per row; `gates` (float
 // [rows, n_q], or null): a factor on the result of every (row, query head); `out_scale`: a factor on every result;
 // `out_pitch`: elements between rows of the output (0: dense).
-extern "C" int srb_decode_attention_gated(const void* q, const void* k_pool, const void* v_pool, void* out,
+// `terms` (or null): kept first tokens, a cap on the scores, two maps per head (AttnTerms; n_q then counts maps and q, out are
+// [rows, n_q / 2, head_dim]).
+extern "C" int srb_decode_attention_terms(const void* q, const void* k_pool, const void* v_pool, void* out,
                                           float* part_acc, float* part_ml, int* counters, const int* positions,
                                           const int* row_request, const int* block_table, int table_stride, int rows,
                                           int n_q, int n_kv, int head_dim, int page_size, int num_pages, int window,
                                           int chunk, int num_splits, float scale, int* error_word, const float* sinks,
-                                          const float* gates, long long out_pitch, float out_scale, void* stream) {
+                                          const float* gates, long long out_pitch, float out_scale, const AttnTerms* terms,
+                                          void* stream) {
   if (rows <= 0) return SRB_OK;
   if (chunk < 0) SRB_FAIL("decode_attention: the chunk size must be non-negative");
   if (!srb_decode_attention_supports(n_q, n_kv, head_dim, SRB_DTYPE_BF16))
@@ -458,12 +550,32 @@ extern "C" int srb_decode_attention_gated(const void* q, const void* k_pool, con
   p.table_stride = table_stride; p.n_q = n_q; p.n_kv = n_kv; p.head_dim = head_dim;
   p.page_size = page_size; p.num_pages = num_pages; p.window = window; p.chunk = chunk; p.split_size = 0;
   p.max_splits = num_splits; p.scale = scale; p.error_word = error_word; p.sinks = sinks; p.gates = gates;
-  p.value_dim = head_dim; p.out_pitch = out_pitch ? out_pitch : (long long)n_q * head_dim; p.out_scale = out_scale;
-  if (p.out_pitch < (long long)n_q * head_dim) SRB_FAIL("decode_attention: rows of the output overlap");
+  p.value_dim = head_dim; p.out_scale = out_scale;
+  if (const char* fault = srb_apply_terms(p, terms)) SRB_FAIL("decode_attention: %s", fault);
+  const long long out_width = (long long)n_q / p.maps * head_dim;
+  p.out_pitch = out_pitch ? out_pitch : out_width;
+  if (p.out_pitch < out_width) SRB_FAIL("decode_attention: rows of the output overlap");
   dp.scale_log2 = scale * 1.4426950408889634f;
+  dp.cap_log2 = p.softcap * 1.4426950408889634f;
+  if (p.softcap > 0.f) dp.scale_log2 *= 2.0f / p.softcap;
   cudaStream_t s = (cudaStream_t)stream;
-  if (head_dim == 64) return launch_decode<64>(q, k_pool, v_pool, out, part_acc, part_ml, counters, dp, rows, s);
-  return launch_decode<128>(q, k_pool, v_pool, out, part_acc, part_ml, counters, dp, rows, s);
+  if (p.maps == 2 && (n_q / n_kv) % 2) SRB_FAIL("decode_attention: a kv head serves whole heads");
+  if (p.maps == 2)
+    return head_dim == 64 ? launch_decode<64, true>(q, k_pool, v_pool, out, part_acc, part_ml, counters, dp, rows, s)
+                          : launch_decode<128, true>(q, k_pool, v_pool, out, part_acc, part_ml, counters, dp, rows, s);
+  if (head_dim == 64) return launch_decode<64, false>(q, k_pool, v_pool, out, part_acc, part_ml, counters, dp, rows, s);
+  return launch_decode<128, false>(q, k_pool, v_pool, out, part_acc, part_ml, counters, dp, rows, s);
+}
+
+extern "C" int srb_decode_attention_gated(const void* q, const void* k_pool, const void* v_pool, void* out,
+                                          float* part_acc, float* part_ml, int* counters, const int* positions,
+                                          const int* row_request, const int* block_table, int table_stride, int rows,
+                                          int n_q, int n_kv, int head_dim, int page_size, int num_pages, int window,
+                                          int chunk, int num_splits, float scale, int* error_word, const float* sinks,
+                                          const float* gates, long long out_pitch, float out_scale, void* stream) {
+  return srb_decode_attention_terms(q, k_pool, v_pool, out, part_acc, part_ml, counters, positions, row_request, block_table,
+                                    table_stride, rows, n_q, n_kv, head_dim, page_size, num_pages, window, chunk, num_splits,
+                                    scale, error_word, sinks, gates, out_pitch, out_scale, nullptr, stream);
 }
 
 extern "C" int srb_decode_attention_masked(const void* q, const void* k_pool, const void* v_pool, void* out,

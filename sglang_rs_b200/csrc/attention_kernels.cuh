@@ -21,7 +21,16 @@
 //    result (a mixer beside another one writes its columns of the row that one output product reads);
 //  * values of another width than the keys: the output and the value rows are `value_dim` wide.  With
 //    `shared_values` the value of a key is the first `value_dim` entries of its key row (a cache that
-//    keeps one latent row per token serves as key and as value), and v_pool is not read.
+//    keeps one latent row per token serves as key and as value), and v_pool is not read;
+//  * first tokens that a window keeps: with `keep_first` > 0 a row also sees the sequence's first keep_first keys, however
+//    far behind its window they lie;
+//  * a cap on the scores: with `softcap` > 0 a score s becomes softcap * tanh(s / softcap), taken in 32-bit;
+//  * two maps per head (differential attention): with `maps` 2 a head's query row and its key row are two halves,
+//    [map 1 | map 2]; each map is an attention of its own over the same values, and the head's result is
+//    o = a_1 - map_lambda * a_2, divided by its own root mean square and multiplied by map_scale.  The kernels see twice as
+//    many query heads (`n_q`): number 2 h + t is map t of head h, whose query is the head's row with the other half taken
+//    as zero; `q` itself holds each head's row once.  The generic kernel writes the maps' results as floats
+//    (`float_out`) and srb_map_combine (attention.cu) joins them; the tensor-core kernels join them in their last step.
 //
 // Work split: one block per (row, kv head and chunk of its query heads, split); the block's warp w
 // owns query head kv_head * G + chunk * heads_per_block + w (at most 32 warps, so more than 32 query
@@ -57,7 +66,48 @@ struct AttnParams {
   const float* gates = nullptr;   // [rows, n_q] or null: a factor on the result of every (row, query head)
   float out_scale = 1.0f;         // a factor on every result, taken in 32-bit before it is rounded
   long long out_pitch = 0;        // elements between rows of the output (a head's results are always dense); 0: n_q * value_dim
+  int keep_first = 0;             // with a window: the sequence's first keys that stay visible behind it
+  float softcap = 0.f;            // > 0: s -> softcap * tanh(s / softcap)
+  int maps = 1;                   // 2: two maps per head, n_q counts maps
+  float map_lambda = 0.f, map_scale = 1.f, map_eps = 0.f;
+  int float_out = 0;              // the generic kernel's results are floats
 };
+
+// What a caller may ask for beyond the arguments that every attention has (null pointer: nothing of it).
+struct AttnTerms {
+  int keep_first;
+  float softcap;
+  int maps;
+  float map_lambda, map_scale, map_eps;
+  int float_out;
+};
+
+// Takes the terms over and checks them against the mask; an error text or null.
+static inline const char* srb_apply_terms(AttnParams& p, const AttnTerms* terms) {
+  if (!terms) return nullptr;
+  if (terms->keep_first < 0 || (terms->keep_first > 0 && p.chunk > 0)) return "first tokens are kept behind a window, not behind a chunk";
+  if (!(terms->softcap >= 0.f)) return "the cap on the scores must be positive, or 0 for none";
+  if (terms->maps != 1 && terms->maps != 2) return "a head has one map or two";
+  if (terms->maps == 2 && (p.sinks || p.gates || p.n_q % 2 || p.head_dim % 2)) return "two maps come without sink and gate, with rows of two halves";
+  p.keep_first = p.window > 0 ? terms->keep_first : 0;
+  p.softcap = terms->softcap; p.maps = terms->maps;
+  p.map_lambda = terms->map_lambda; p.map_scale = terms->map_scale; p.map_eps = terms->map_eps; p.float_out = terms->float_out;
+  return nullptr;
+}
+
+// The pieces of `size` keys, cut at absolute multiples of `size`, that a row or tile walks: first those that hold kept first
+// tokens and lie ahead of the window's first piece, then the window's.  Piece number i of the walk is piece
+// srb_piece(i, ...) of the sequence.
+__host__ __device__ __forceinline__ int srb_kept_pieces(int keep_first, int size, int first_piece) {
+  const int kept = (keep_first + size - 1) / size;
+  return kept < first_piece ? kept : first_piece;
+}
+__host__ __device__ __forceinline__ int srb_piece(int i, int kept_pieces, int first_piece) {
+  return i < kept_pieces ? i : first_piece + i - kept_pieces;
+}
+
+// cap * tanh(x / cap) from x / cap: tanh(y) = 1 - 2 / (e^(2y) + 1), finite for every y
+__device__ __forceinline__ float srb_capped(float y, float cap) { return cap * (1.0f - 2.0f / (expf(2.0f * y) + 1.0f)); }
 
 // The first key that a row at `pos` may see: the start of its window, or of its chunk of positions, whichever is later.
 // It never falls as pos grows, so the first row of a tile has the lowest first key of the tile.
@@ -74,19 +124,21 @@ __device__ __forceinline__ void row_key_range(const AttnParams& p, int pos, int 
   const int begin = srb_first_visible(pos, p.window, p.chunk);
   const int end = pos + 1;
   if (p.split_size == 0) {
-    lo = begin;
+    lo = p.keep_first > 0 ? 0 : begin;
     hi = end;
     return;
   }
   const int first = begin / p.split_size;
-  lo = max(begin, (first + split) * p.split_size);
-  hi = min(end, (first + split + 1) * p.split_size);
+  const int piece = srb_piece(split, srb_kept_pieces(p.keep_first, p.split_size, first), first) * p.split_size;
+  lo = piece < p.keep_first ? piece : max(begin, piece);
+  hi = min(end, piece + p.split_size);
 }
 
 __device__ __forceinline__ int row_split_count(const AttnParams& p, int pos) {
   if (p.split_size == 0) return 1;
   const int begin = srb_first_visible(pos, p.window, p.chunk);
-  return pos / p.split_size - begin / p.split_size + 1;
+  const int first = begin / p.split_size;
+  return pos / p.split_size - first + 1 + srb_kept_pieces(p.keep_first, p.split_size, first);
 }
 
 template <typename T, int DIM_PER_LANE>
@@ -117,20 +169,35 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
   const bool live = warp < here;                         // a warp beyond the group's heads only helps to load
   const int q_head = kv_head * groups + first_head + (live ? warp : 0);
 
-  for (int i = threadIdx.x; i < here * d; i += blockDim.x)
-    q_tile[i] = srb_to_float(q[((size_t)row * p.n_q + (size_t)kv_head * groups + first_head) * d + i]);
+  if (p.maps == 2) {
+    // number 2 h + t: the head's row, of which map t is one half
+    for (int i = threadIdx.x; i < here * d; i += blockDim.x) {
+      const int number = kv_head * groups + first_head + i / d, e = i % d;
+      const bool mine = (e >= (d >> 1)) == (number & 1);
+      q_tile[i] = mine ? srb_to_float(q[((size_t)row * (p.n_q >> 1) + (number >> 1)) * d + e]) : 0.f;
+    }
+  } else {
+    for (int i = threadIdx.x; i < here * d; i += blockDim.x)
+      q_tile[i] = srb_to_float(q[((size_t)row * p.n_q + (size_t)kv_head * groups + first_head) * d + i]);
+  }
+  const int begin = srb_first_visible(pos, p.window, p.chunk);
+  // the entries of a row that its score sums over: all, or one map's half
+  const int e_begin = p.maps == 2 ? (q_head & 1) * (d >> 1) : 0, e_end = p.maps == 2 ? e_begin + (d >> 1) : d;
 
   float m = -INFINITY, l = 0.f;
   float acc[DIM_PER_LANE];
 #pragma unroll
   for (int j = 0; j < DIM_PER_LANE; ++j) acc[j] = 0.f;
 
-  for (int base = lo & ~(KEY_BLOCK - 1); base < hi; base += KEY_BLOCK) {
+  int base = lo & ~(KEY_BLOCK - 1);
+  for (int next; base < hi; base = next) {
+    next = base + KEY_BLOCK;
+    if (next >= p.keep_first && next < (begin & ~(KEY_BLOCK - 1))) next = begin & ~(KEY_BLOCK - 1);   // blocks without a visible key
     __syncthreads();                                     // previous tile fully consumed
     if (threadIdx.x < KEY_BLOCK) {
       const int key = base + threadIdx.x;
       long long offset = -1;
-      if (key >= lo && key < hi) {
+      if (key >= lo && key < hi && (key >= begin || key < p.keep_first)) {
         const int page = p.block_table[(size_t)request * p.table_stride + key / p.page_size];
         if (page < 0 || page >= p.num_pages) {
           atomicOr(p.error_word, SRB_FLAG_BAD_PAGE);
@@ -159,8 +226,10 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
     float s = 0.f;
     const float* qv = q_tile + (live ? warp : 0) * d;
     const float* kv = k_tile + lane * (d + 1);
-    for (int e = 0; e < d; ++e) s += qv[e] * kv[e];
-    s = key_offset[lane] < 0 ? -INFINITY : s * p.scale;
+    for (int e = e_begin; e < e_end; ++e) s += qv[e] * kv[e];
+    s *= p.scale;
+    if (p.softcap > 0.f) s = srb_capped(s / p.softcap, p.softcap);
+    if (key_offset[lane] < 0) s = -INFINITY;
 
     const float m_new = fmaxf(m, srb_warp_max(s));       // finite: the tile holds a visible key
     const float correction = expf(m - m_new);            // exp(-inf) = 0 on the first tile
@@ -194,7 +263,10 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
 #pragma unroll
     for (int j = 0; j < DIM_PER_LANE; ++j) {
       const int e = lane + 32 * j;
-      if (e < vd) out[(size_t)row * p.out_pitch + (size_t)q_head * vd + e] = srb_from_float<T>(acc[j] * inv);
+      if (e >= vd) continue;
+      const size_t at = (size_t)row * p.out_pitch + (size_t)q_head * vd + e;
+      if (p.float_out) reinterpret_cast<float*>(out)[at] = acc[j] * inv;
+      else out[at] = srb_from_float<T>(acc[j] * inv);
     }
   } else {
     const size_t slot = ((size_t)row * p.n_q + q_head) * p.max_splits + split;
@@ -233,7 +305,9 @@ __global__ void attention_combine_kernel(const float* __restrict__ part_acc, con
     float acc = 0.f;
     for (int s = 0; s < count; ++s)
       acc += part_acc[(first + s) * p.value_dim + e] * expf(part_ml[(first + s) * 2] - m);
-    out[(size_t)row * p.out_pitch + (size_t)q_head * p.value_dim + e] = srb_from_float<T>(acc * inv);
+    const size_t at = (size_t)row * p.out_pitch + (size_t)q_head * p.value_dim + e;
+    if (p.float_out) reinterpret_cast<float*>(out)[at] = acc * inv;
+    else out[at] = srb_from_float<T>(acc * inv);
   }
 }
 
@@ -270,7 +344,8 @@ static int paged_attention_dispatch_masked(const void* q, const void* k_pool, co
                                            int n_q, int n_kv, int head_dim, int page_size, int num_pages, int window,
                                            int chunk, int split_size, int max_splits, float scale, int* error_word,
                                            int dtype, const float* sinks, int value_dim, void* stream,
-                                           const float* gates = nullptr, long long out_pitch = 0, float out_scale = 1.0f) {
+                                           const float* gates = nullptr, long long out_pitch = 0, float out_scale = 1.0f,
+                                           const AttnTerms* terms = nullptr) {
   if (rows <= 0) return SRB_OK;
   if (chunk < 0) SRB_FAIL("paged_attention: the chunk size must be non-negative");
   if (n_q <= 0 || n_kv <= 0 || n_q % n_kv != 0)
@@ -297,6 +372,8 @@ static int paged_attention_dispatch_masked(const void* q, const void* k_pool, co
   p.sinks = sinks; p.value_dim = value_dim; p.shared_values = v_pool == nullptr; p.gates = gates;
   p.out_pitch = out_pitch ? out_pitch : (long long)n_q * value_dim; p.out_scale = out_scale;
   if (p.out_pitch < (long long)n_q * value_dim) SRB_FAIL("paged_attention: rows of the output overlap");
+  if (const char* fault = srb_apply_terms(p, terms)) SRB_FAIL("paged_attention: %s", fault);
+  if (p.maps == 2 && !p.float_out) SRB_FAIL("paged_attention: the results of two maps are floats that srb_map_combine joins");
   const int groups = n_q / n_kv;
   p.head_chunks = (groups + 31) / 32;
   p.heads_per_block = (groups + p.head_chunks - 1) / p.head_chunks;

@@ -48,7 +48,9 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
   const int request = tiles[4 * tile + 2], pos_begin = tiles[4 * tile + 3];
   const int kv_lo = srb_first_visible(pos_begin, p.window, p.chunk);
   const int kv_hi = pos_begin + n_rows;                                  // keys 0 .. last row's position
-  const int first_block = kv_lo / PF_KEYS, last_block = (kv_hi - 1) / PF_KEYS;
+  // the walk: blocks ahead of the window that hold kept first tokens, then the window's
+  const int first_block = kv_lo / PF_KEYS, kept_blocks = srb_kept_pieces(p.keep_first, PF_KEYS, first_block);
+  const int num_blocks = (kv_hi - 1) / PF_KEYS - first_block + 1 + kept_blocks;
 
   for (int i = threadIdx.x; i < PF_ROWS * CHUNKS; i += blockDim.x) {
     const int r = i / CHUNKS, c = i % CHUNKS;
@@ -59,13 +61,14 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
   cp_async_commit();
 
   const int page_shift = (p.page_size & (p.page_size - 1)) == 0 ? __ffs(p.page_size) - 1 : -1;
-  auto load_block = [&](int block, int stage) {
+  auto load_block = [&](int walked, int stage) {
+    const int block = srb_piece(walked, kept_blocks, first_block);
     __nv_bfloat16* ks = kv + (size_t)stage * 2 * PF_KEYS * D;
     __nv_bfloat16* vs = ks + PF_KEYS * D;
     for (int i = threadIdx.x; i < PF_KEYS * CHUNKS; i += blockDim.x) {
       const int key = i / CHUNKS, c = i % CHUNKS;
       const int abs_key = block * PF_KEYS + key;
-      bool valid = abs_key >= kv_lo && abs_key < kv_hi;
+      bool valid = abs_key < kv_hi && (abs_key >= kv_lo || abs_key < p.keep_first);
       long long offset = 0;
       if (valid) {
         const int logical = page_shift >= 0 ? abs_key >> page_shift : abs_key / p.page_size;
@@ -84,7 +87,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     }
     cp_async_commit();
   };
-  load_block(first_block, 0);
+  load_block(0, 0);
 
   const int g = lane >> 2, col = (lane & 3) * 2;
   const int mat = lane >> 3, mrow = lane & 7;
@@ -92,7 +95,10 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
   const int r_in[2] = {warp * 16 + g, warp * 16 + g + 8};
   const int pos_r[2] = {pos_begin + r_in[0], pos_begin + r_in[1]};
   const int lowest_r[2] = {srb_first_visible(pos_r[0], p.window, p.chunk), srb_first_visible(pos_r[1], p.window, p.chunk)};
-  const float scale_log2 = p.scale * 1.4426950408889634f;
+  // with a cap: first 2 s / softcap in units of log2, then softcap * tanh(s / softcap) in those units
+  const float cap_log2 = p.softcap * 1.4426950408889634f;
+  const float to_cap = p.softcap > 0.f ? 2.0f * p.scale / p.softcap * 1.4426950408889634f : 0.f;
+  const float scale_log2 = p.softcap > 0.f ? 1.0f : p.scale * 1.4426950408889634f;
   const int warp_first_pos = pos_begin + warp * 16;
   const int warp_last_pos = pos_begin + min(warp * 16 + 15, n_rows - 1);
   const bool warp_has_rows = warp * 16 < n_rows;
@@ -112,10 +118,11 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
 #pragma unroll
   for (int t = 0; t < NT_O; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.f;
 
-  for (int block = first_block; block <= last_block; ++block) {
-    const int stage = (block - first_block) & 1;
-    if (block < last_block) {
-      load_block(block + 1, stage ^ 1);
+  for (int walked = 0; walked < num_blocks; ++walked) {
+    const int block = srb_piece(walked, kept_blocks, first_block);
+    const int stage = walked & 1;
+    if (walked + 1 < num_blocks) {
+      load_block(walked + 1, stage ^ 1);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
@@ -124,7 +131,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     const int block_lo = block * PF_KEYS, block_hi = block_lo + PF_KEYS;
     // the block matters to this warp if some key in it is visible to one of the warp's rows
     const int warp_window_lo = srb_first_visible(warp_first_pos, p.window, p.chunk);
-    if (warp_has_rows && block_lo <= warp_last_pos && block_hi > warp_window_lo) {
+    if (warp_has_rows && block_lo <= warp_last_pos && (block_hi > warp_window_lo || block_lo < p.keep_first)) {
       const __nv_bfloat16* ks = kv + (size_t)stage * 2 * PF_KEYS * D;
       const __nv_bfloat16* vs = ks + PF_KEYS * D;
       float s[NT_S][4];
@@ -148,7 +155,14 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
       // the comparisons.
       float mx[2] = {-INFINITY, -INFINITY};
       const bool all_visible = warp * 16 + 15 < n_rows && block_hi - 1 <= warp_first_pos &&
-                               block_lo >= srb_first_visible(pos_begin + warp * 16 + 15, p.window, p.chunk);
+                               (block_lo >= srb_first_visible(pos_begin + warp * 16 + 15, p.window, p.chunk) ||
+                                block_hi <= p.keep_first);
+      if (to_cap > 0.f) {
+#pragma unroll
+        for (int t = 0; t < NT_S; ++t)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[t][e] = cap_log2 * (1.0f - __fdividef(2.0f, exp2f(s[t][e] * to_cap) + 1.0f));
+      }
       if (all_visible) {
 #pragma unroll
         for (int t = 0; t < NT_S; ++t) {
@@ -165,7 +179,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
           for (int e = 0; e < 4; ++e) {
             const int h = e >> 1;
             const int key = block_lo + t * 8 + col + (e & 1);
-            const bool visible = r_in[h] < n_rows && key <= pos_r[h] && key >= lowest_r[h];
+            const bool visible = r_in[h] < n_rows && key <= pos_r[h] && (key >= lowest_r[h] || key < p.keep_first);
             const float v = visible ? s[t][e] * scale_log2 : -INFINITY;
             s[t][e] = v;
             mx[h] = fmaxf(mx[h], v);
@@ -269,11 +283,12 @@ extern "C" int srb_prefill_tile_rows() { return PF_ROWS; }
 // `sinks` (float [n_q], or null): exp(sink_h) joins the softmax's denominator of head h; `gates` (float [rows, n_q], or
 // null): a factor on the result of every (row, query head); `out_scale`: a factor on every result; `out_pitch`: elements
 // between rows of the output (0: dense).
-extern "C" int srb_prefill_attention_gated(const void* q, const void* k_pool, const void* v_pool, void* out,
+// `terms` (or null): kept first tokens, a cap on the scores (AttnTerms); two maps per head are not taken here.
+extern "C" int srb_prefill_attention_terms(const void* q, const void* k_pool, const void* v_pool, void* out,
                                            const int* tiles, int num_tiles, const int* block_table, int table_stride,
                                            int n_q, int n_kv, int head_dim, int page_size, int num_pages, int window,
                                            int chunk, float scale, int* error_word, const float* sinks, const float* gates,
-                                           long long out_pitch, float out_scale, void* stream) {
+                                           long long out_pitch, float out_scale, const AttnTerms* terms, void* stream) {
   if (num_tiles <= 0) return SRB_OK;
   if (chunk < 0) SRB_FAIL("prefill_attention: the chunk size must be non-negative");
   if (!srb_prefill_attention_supports(n_q, n_kv, head_dim, SRB_DTYPE_BF16))
@@ -288,9 +303,21 @@ extern "C" int srb_prefill_attention_gated(const void* q, const void* k_pool, co
   p.max_splits = 1; p.scale = scale; p.error_word = error_word; p.sinks = sinks; p.gates = gates;
   p.value_dim = head_dim; p.out_pitch = out_pitch ? out_pitch : (long long)n_q * head_dim; p.out_scale = out_scale;
   if (p.out_pitch < (long long)n_q * head_dim || p.out_pitch % 2) SRB_FAIL("prefill_attention: rows of the output overlap or start off 4-byte borders");
+  if (const char* fault = srb_apply_terms(p, terms)) SRB_FAIL("prefill_attention: %s", fault);
+  if (p.maps != 1) SRB_FAIL("prefill_attention: two maps per head are not taken by this kernel");
   cudaStream_t s = (cudaStream_t)stream;
   if (head_dim == 64) return launch_prefill<64>(q, k_pool, v_pool, out, tiles, num_tiles, p, s);
   return launch_prefill<128>(q, k_pool, v_pool, out, tiles, num_tiles, p, s);
+}
+
+extern "C" int srb_prefill_attention_gated(const void* q, const void* k_pool, const void* v_pool, void* out,
+                                           const int* tiles, int num_tiles, const int* block_table, int table_stride,
+                                           int n_q, int n_kv, int head_dim, int page_size, int num_pages, int window,
+                                           int chunk, float scale, int* error_word, const float* sinks, const float* gates,
+                                           long long out_pitch, float out_scale, void* stream) {
+  return srb_prefill_attention_terms(q, k_pool, v_pool, out, tiles, num_tiles, block_table, table_stride, n_q, n_kv, head_dim,
+                                     page_size, num_pages, window, chunk, scale, error_word, sinks, gates, out_pitch, out_scale,
+                                     nullptr, stream);
 }
 
 extern "C" int srb_prefill_attention_masked(const void* q, const void* k_pool, const void* v_pool, void* out,

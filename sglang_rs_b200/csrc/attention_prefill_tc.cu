@@ -47,6 +47,9 @@ struct TcArgs {
   const float* gates;      // [rows, n_q] or null: a factor on the result of every (row, query head)
   long long out_pitch;     // elements between rows of the output
   float out_scale;         // a factor on every result
+  int keep_first;          // with a window: the sequence's first keys that stay visible behind it
+  float cap_log2;          // softcap * log2 e, or 0; with a cap `scale_log2` brings a score to 2 s / softcap in units of log2
+  float map_lambda, map_scale, map_eps;    // two maps per head: o = a_1 - map_lambda a_2, over its root mean square, times map_scale
 };
 
 // M = 128, N = n, A and B bfloat16, D float; b_mn_major: B is [K rows][N contiguous] (V), else K-major
@@ -102,7 +105,11 @@ __device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigne
 // HEADS query heads of one kv head share a block (1 or 2): they read the same K and V tiles from
 // shared memory, which halves the traffic from L2.  STAGES tiles of K and of V are in flight.
 
-template <int D, int HEADS, int STAGES>
+// MAPS (with HEADS 2): the block's two heads are the two maps of ONE head (AttnParams): its query and key rows are two
+// halves, one per map, and both maps read the same values, so the block has one tile of Q, a score sums over its map's half
+// of the row, and the two results meet in the last step: a row's 2 x D results lie in the same lanes of tensor memory.
+// CAP: scores go through softcap * tanh(s / softcap).
+template <int D, int HEADS, int STAGES, bool MAPS, bool CAP>
 __global__ void __launch_bounds__(64 + 160 * HEADS, HEADS == 1 ? 2 : 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_out,
@@ -112,32 +119,36 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   constexpr int HALF_BYTES = TC_KEYS * 128;                // [64 keys][64] bfloat16
   constexpr int Q_BYTES = HALVES * Q_HALF_BYTES;
   constexpr int KV_BYTES = HALVES * HALF_BYTES;
+  constexpr int Q_TILES = MAPS ? 1 : HEADS;                // maps share their head's tile of Q
+  static_assert(!MAPS || HEADS == 2, "two maps share a block");
   // tensor-memory columns, 256 per head: two S buffers of 64 columns, then O.  P (bfloat16 pairs,
   // 32 columns) overwrites the first half of the S buffer it was computed from.
   constexpr unsigned S_COL = 0, O_COL = 128, HEAD_COLUMNS = 256;
   constexpr unsigned TMEM_COLUMNS = HEAD_COLUMNS * HEADS;
   extern __shared__ unsigned char smem_unaligned[];
   unsigned char* smem = reinterpret_cast<unsigned char*>(((uintptr_t)smem_unaligned + 1023) & ~(uintptr_t)1023);
-  unsigned char* q_smem = smem;                            // HEADS tiles of Q
-  unsigned char* k_smem = smem + HEADS * Q_BYTES;          // STAGES tiles of K, then STAGES tiles of V
+  unsigned char* q_smem = smem;                            // Q_TILES tiles of Q
+  unsigned char* k_smem = smem + Q_TILES * Q_BYTES;        // STAGES tiles of K, then STAGES tiles of V
   unsigned char* v_smem = k_smem + STAGES * KV_BYTES;
   __shared__ __align__(8) unsigned long long q_full, k_full[STAGES], v_full[STAGES], k_empty[STAGES], v_empty[STAGES],
       s_ready[HEADS][2], p_ready[HEADS][2], pv_done[HEADS][2], o_ready[HEADS];
   __shared__ unsigned tmem_holder;
   __shared__ int abort_flag;
+  __shared__ float map_factor[MAPS ? 2 : 1][MAPS ? TC_ROWS : 1], map_squares[MAPS ? 2 : 1][MAPS ? TC_ROWS : 1];
 
   srb_mark(SRB_MARK_PREFILL_ATTENTION, 0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // heads are the fast grid dimension: tiles arrive sorted by falling work, so the long ones start first
-  const int tile = blockIdx.y, head0 = blockIdx.x * HEADS;
-  const int groups = args.n_q / args.n_kv;
+  const int tile = blockIdx.y, head0 = blockIdx.x * Q_TILES;
+  const int groups = args.n_q / args.n_kv;               // (n_q counts heads, not maps)
   const int kv_head = head0 / groups;
   const int row_begin = args.tiles[4 * tile], n_rows = args.tiles[4 * tile + 1];
   const int request = args.tiles[4 * tile + 2], pos_begin = args.tiles[4 * tile + 3];
   const int kv_lo = srb_first_visible(pos_begin, args.window, args.chunk);
   const int kv_hi = pos_begin + n_rows;
-  const int first_block = kv_lo / TC_KEYS, last_block = (kv_hi - 1) / TC_KEYS;
-  const int num_blocks = last_block - first_block + 1;
+  // the walk: blocks ahead of the window that hold kept first tokens, then the window's
+  const int first_block = kv_lo / TC_KEYS, kept_blocks = srb_kept_pieces(args.keep_first, TC_KEYS, first_block);
+  const int num_blocks = (kv_hi - 1) / TC_KEYS - first_block + 1 + kept_blocks;
 
   if (threadIdx.x == 0) {
     abort_flag = 0;
@@ -175,8 +186,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int pages_per_block = TC_KEYS / args.page_size;
     if (is_k && elect_one()) {
       // Q: [128 rows][D] of each head, as HALVES tiles of [128][64]
-      mbar_expect_tx(smem_u32(&q_full), HEADS * Q_BYTES);
-      for (int t = 0; t < HEADS; ++t)
+      mbar_expect_tx(smem_u32(&q_full), Q_TILES * Q_BYTES);
+      for (int t = 0; t < Q_TILES; ++t)
         for (int h = 0; h < HALVES; ++h)
           tma_load_3d(smem_u32(q_smem + t * Q_BYTES + h * Q_HALF_BYTES), &map_q, smem_u32(&q_full), h * 64, head0 + t,
                       row_begin);
@@ -184,8 +195,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     auto pool_row_of = [&](int block) {
       int row = args.pool_rows;                             // outside the pool: TMA fills zeros
       if (lane < pages_per_block && block < num_blocks) {
-        const int key = (first_block + block) * TC_KEYS + lane * args.page_size;
-        if (key < kv_hi && key + args.page_size > kv_lo) {
+        const int key = srb_piece(block, kept_blocks, first_block) * TC_KEYS + lane * args.page_size;
+        if (key < kv_hi && (key + args.page_size > kv_lo || key < args.keep_first)) {
           const int page = args.block_table[(size_t)request * args.table_stride + key / args.page_size];
           if (page < 0 || (long long)(page + 1) * args.n_kv * args.page_size > args.pool_rows)
             atomicOr(args.error_word, SRB_FLAG_BAD_PAGE);
@@ -233,7 +244,10 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int t = warp - 1;
     constexpr unsigned idesc_s = tc_idesc(TC_KEYS, false);
     constexpr unsigned idesc_o = tc_idesc(D, true);
-    const unsigned long long q_desc = smem_descriptor(smem_u32(q_smem) + t * Q_BYTES);
+    const unsigned long long q_desc = smem_descriptor(smem_u32(q_smem) + (MAPS ? 0 : t * Q_BYTES));
+    // the row's entries that a score sums over, in steps of 16: all, or the map's half
+    constexpr int K_STEPS = MAPS ? D / 32 : D / 16;
+    const int k_first = MAPS ? t * K_STEPS : 0;
     const unsigned long long k_desc = smem_descriptor(smem_u32(k_smem));
     const unsigned long long v_desc = smem_descriptor_mn(smem_u32(v_smem), HALF_BYTES);
     const unsigned head_tmem = tmem_base + t * HEAD_COLUMNS;
@@ -246,10 +260,11 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       const unsigned long long k_stage = k_desc + (unsigned long long)((s * KV_BYTES) >> 4);
       if (elect_one()) {
 #pragma unroll
-        for (int k = 0; k < D / 16; ++k) {
+        for (int step = 0; step < K_STEPS; ++step) {
+          const int k = k_first + step;
           const unsigned q_off = (unsigned)((k / 4) * Q_HALF_BYTES + (k % 4) * 32) >> 4;
           const unsigned k_off = (unsigned)((k / 4) * HALF_BYTES + (k % 4) * 32) >> 4;
-          umma_bf16(head_tmem + S_COL + (j & 1) * TC_KEYS, q_desc + q_off, k_stage + k_off, idesc_s, k > 0 ? 1u : 0u);
+          umma_bf16(head_tmem + S_COL + (j & 1) * TC_KEYS, q_desc + q_off, k_stage + k_off, idesc_s, step > 0 ? 1u : 0u);
         }
         umma_commit(smem_u32(&s_ready[t][j & 1]));
         umma_commit(smem_u32(&k_empty[s]));
@@ -283,13 +298,14 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   } else {
     // softmax: four warps per head, thread = row
     const int t = (warp - 1 - HEADS) >> 2;
-    const int head = head0 + t;
+    const int head = MAPS ? head0 : head0 + t;
     const int quarter = warp & 3;
     const int r = quarter * 32 + lane;
     const int pos_r = pos_begin + r;
     const int lowest_r = srb_first_visible(pos_r, args.window, args.chunk);
     const bool row_live = r < n_rows;
     const unsigned lane_address = tmem_base + t * HEAD_COLUMNS + ((unsigned)(quarter * 32) << 16);
+    const float to_log2 = CAP ? 1.0f : args.scale_log2;    // capped scores are in units of log2 already
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int i = 0; i < num_blocks && ok; ++i) {
@@ -297,17 +313,23 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       ok = mbar_wait(smem_u32(&s_ready[t][i & 1]), (unsigned)(i >> 1) & 1u, &abort_flag);
       if (!ok) break;
       tc_fence_after();
-      const int key0 = (first_block + i) * TC_KEYS;
+      const int key0 = srb_piece(i, kept_blocks, first_block) * TC_KEYS;
       const bool all_visible = n_rows == TC_ROWS && key0 + TC_KEYS - 1 <= pos_begin &&
-                               key0 >= srb_first_visible(pos_begin + TC_ROWS - 1, args.window, args.chunk);
+                               (key0 >= srb_first_visible(pos_begin + TC_ROWS - 1, args.window, args.chunk) ||
+                               key0 + TC_KEYS <= args.keep_first);
       // the row's 64 raw scores, once; masked keys become -inf
       float sv[TC_KEYS];
       tmem_load_64(lane_address + s_col, sv);
+      if (CAP) {
+        // 2 s / softcap in units of log2 -> softcap * tanh(s / softcap) in units of log2; tanh(y) = 1 - 2 / (e^(2y) + 1)
+#pragma unroll
+        for (int j = 0; j < TC_KEYS; ++j) sv[j] = args.cap_log2 * (1.0f - __fdividef(2.0f, ex2(sv[j] * args.scale_log2) + 1.0f));
+      }
       if (!all_visible) {
 #pragma unroll
         for (int j = 0; j < TC_KEYS; ++j) {
           const int key = key0 + j;
-          if (!(row_live && key <= pos_r && key >= lowest_r)) sv[j] = -INFINITY;
+          if (!(row_live && key <= pos_r && (key >= lowest_r || key < args.keep_first))) sv[j] = -INFINITY;
         }
       }
       // three-input maxima, four chains
@@ -319,7 +341,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       }
       mx[0] = max3(mx[0], sv[TC_KEYS - 4], sv[TC_KEYS - 3]);
       mx[1] = max3(mx[1], sv[TC_KEYS - 2], sv[TC_KEYS - 1]);
-      const float m_block = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * args.scale_log2;   // in units of log2
+      const float m_block = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * to_log2;   // in units of log2
       // the running maximum moves only when it must: P stays below 2^8
       float corr = 1.f;
       bool rescale = false;
@@ -349,7 +371,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       l_run *= corr;
       // P = 2^(s * scale * log2 e - m), rounded to bfloat16 pairs, over the scores it came from; the row's sum
       // (two-wide 32-bit multiply-adds and adds; the exponential is one ex2 per score)
-      const unsigned long long scale2 = pack2(args.scale_log2, args.scale_log2), neg_m2 = pack2(-m_use, -m_use);
+      const unsigned long long scale2 = pack2(to_log2, to_log2), neg_m2 = pack2(-m_use, -m_use);
       unsigned long long sums2[2] = {0ull, 0ull};
 #pragma unroll
       for (int c = 0; c < TC_KEYS; c += 32) {
@@ -378,13 +400,68 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       mbar_arrive(smem_u32(&p_ready[t][i & 1]));
     }
     if (ok) ok = mbar_wait(smem_u32(&o_ready[t]), 0, &abort_flag);
+    if (MAPS) {
+      // The join: thread r of either map's warps takes one half of row r's entries, from both maps' results.  (Every thread
+      // of the eight warps passes both barriers, also one whose wait gave up.)
+      if (ok) ok = mbar_wait(smem_u32(&o_ready[t ^ 1]), 0, &abort_flag);
+      tc_fence_after();
+      map_factor[t][r] = row_live && l_run > 0.f ? (t == 0 ? 1.0f : args.map_lambda) / l_run : 0.f;
+      asm volatile("bar.sync 1, 256;" ::: "memory");
+      constexpr int MINE = D / 2;
+      const float f1 = map_factor[0][r], f2 = map_factor[1][r];
+      const unsigned row_tmem = tmem_base + ((unsigned)(quarter * 32) << 16) + O_COL + t * MINE;
+      float o[MINE], squares = 0.f;
+      if (ok) {
+#pragma unroll
+        for (int c = 0; c < MINE; c += 32) {
+          float first[32], second[32];
+          tmem_load_32(row_tmem + c, first);
+          tmem_load_32(row_tmem + HEAD_COLUMNS + c, second);
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            o[c + j] = first[j] * f1 - second[j] * f2;
+            squares += o[c + j] * o[c + j];
+          }
+        }
+      }
+      map_squares[t][r] = squares;
+      asm volatile("bar.sync 1, 256;" ::: "memory");
+      const float factor = args.map_scale / sqrtf((map_squares[0][r] + map_squares[1][r]) / (float)D + args.map_eps);
+      const bool whole = n_rows == TC_ROWS;
+      if (ok) {
+        __nv_bfloat16* dst = args.out + (size_t)(row_begin + r) * args.out_pitch + (size_t)head * D + t * MINE;
+#pragma unroll
+        for (int c = 0; c < MINE; c += 8) {
+          uint4 packed;
+          __nv_bfloat162* pair = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) pair[j] = __floats2bfloat162_rn(o[c + 2 * j] * factor, o[c + 2 * j + 1] * factor);
+          if (whole) {
+            const int column = t * MINE + c, piece = (column & 63) >> 3;
+            *reinterpret_cast<uint4*>(q_smem + (column >> 6) * Q_HALF_BYTES + r * 128 + ((piece ^ (r & 7)) << 4)) = packed;
+          } else if (row_live) {
+            *reinterpret_cast<uint4*>(dst + c) = packed;
+          }
+        }
+      }
+      if (whole) {
+        fence_proxy_async_shared();
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        if (t == 0 && quarter == 0 && lane == 0 && !abort_flag) {
+#pragma unroll
+          for (int h = 0; h < HALVES; ++h)
+            tma_store_3d(&map_out, smem_u32(q_smem + h * Q_HALF_BYTES), h * 64, head, row_begin);
+          tma_store_commit_and_wait_read();
+        }
+      }
+    }
     // A whole tile leaves through shared memory and one bulk store per 64 columns: a thread's row lies 8 KB from its
     // neighbour's in the output, so stores from registers touch 32 lines per instruction.  The head's Q tile is free
     // (every S product has completed) and has the layout the store wants: [128 rows][128 bytes] per 64 columns,
     // 16-byte pieces exchanged by the 128-byte swizzle.
     const bool whole_tile = n_rows == TC_ROWS;
     unsigned char* stage = q_smem + t * Q_BYTES;
-    if (ok) {
+    if (!MAPS && ok) {
       tc_fence_after();
       float l_all = l_run, shrink = 1.f;
       if (args.sinks && row_live) {
@@ -418,7 +495,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
       }
     }
-    if (whole_tile) {
+    if (!MAPS && whole_tile) {
       // (every warp of the head comes here, also one whose wait gave up: the barrier below counts all four)
       fence_proxy_async_shared();
       if (t == 0)
@@ -474,13 +551,14 @@ extern "C" int srb_prefill_tc_supports(int n_q, int n_kv, int head_dim, int page
 
 extern "C" int srb_prefill_tc_tile_rows() { return TC_ROWS; }
 
-template <int D, int HEADS, int STAGES>
+template <int D, int HEADS, int STAGES, bool MAPS, bool CAP>
 static int launch_tc(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v, const CUtensorMap& map_out,
                      const TcArgs& args, int num_tiles, cudaStream_t s) {
-  const size_t smem = (size_t)(D / 64) * 128 * (HEADS * TC_ROWS + 2 * STAGES * TC_KEYS) + 1024;
-  auto kernel = prefill_attention_tc_kernel<D, HEADS, STAGES>;
+  constexpr int TILES = MAPS ? 1 : HEADS;                  // heads of a block
+  const size_t smem = (size_t)(D / 64) * 128 * (TILES * TC_ROWS + 2 * STAGES * TC_KEYS) + 1024;
+  auto kernel = prefill_attention_tc_kernel<D, HEADS, STAGES, MAPS, CAP>;
   SRB_CUDA_CALL(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  dim3 grid(args.n_q / HEADS, num_tiles);
+  dim3 grid(args.n_q / TILES, num_tiles);
   if (num_tiles > 65535) SRB_FAIL("prefill_attention_tc: %d tiles exceed one launch", num_tiles);
   kernel<<<grid, 64 + 160 * HEADS, smem, s>>>(map_q, map_k, map_v, map_out, args);
   SRB_LAUNCH_CHECK("prefill_attention_tc");
@@ -493,12 +571,14 @@ static int launch_tc(const CUtensorMap& map_q, const CUtensorMap& map_k, const C
 // `sinks` (float [n_q], or null): exp(sink_h) joins the softmax's denominator of head h; `gates` (float [rows, n_q], or
 // null): a factor on the result of every (row, query head); `out_scale`: a factor on every result; `out_pitch`: elements
 // between rows of the output (a multiple of 8; 0: dense).
-extern "C" int srb_prefill_attention_tc_gated(const void* q, const void* k_pool, const void* v_pool, void* out,
+// `terms` (or null): kept first tokens, a cap on the scores, two maps per head (AttnTerms; n_q then counts maps and q, out are
+// [rows, n_q / 2, head_dim]).
+extern "C" int srb_prefill_attention_tc_terms(const void* q, const void* k_pool, const void* v_pool, void* out,
                                               const int* tiles, int num_tiles, int rows, const int* block_table,
                                               int table_stride, int n_q, int n_kv, int head_dim, int page_size,
                                               int num_pages, int window, int chunk, float scale, int* error_word,
                                               const float* sinks, const float* gates, long long out_pitch,
-                                              float out_scale, void* stream) {
+                                              float out_scale, const AttnTerms* terms, void* stream) {
   if (num_tiles <= 0) return SRB_OK;
   if (chunk < 0) SRB_FAIL("prefill_attention_tc: the chunk size must be non-negative");
   if (!srb_prefill_tc_supports(n_q, n_kv, head_dim, page_size, SRB_DTYPE_BF16))
@@ -508,6 +588,11 @@ extern "C" int srb_prefill_attention_tc_gated(const void* q, const void* k_pool,
     SRB_FAIL("prefill_attention_tc: page count, table stride and rows must be positive");
   if ((((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15) != 0)
     SRB_FAIL("prefill_attention_tc: operands must be 16-byte aligned");
+  AttnParams p;
+  p.window = window; p.chunk = chunk; p.sinks = sinks; p.gates = gates; p.n_q = n_q; p.head_dim = head_dim;
+  if (const char* fault = srb_apply_terms(p, terms)) SRB_FAIL("prefill_attention_tc: %s", fault);
+  if (p.maps == 2 && (n_q / n_kv) % 2) SRB_FAIL("prefill_attention_tc: a kv head serves whole heads");
+  n_q /= p.maps;                                             // heads from here on
   if (out_pitch == 0) out_pitch = (long long)n_q * head_dim;
   if (out_pitch < (long long)n_q * head_dim || out_pitch % 8)
     SRB_FAIL("prefill_attention_tc: rows of the output overlap or start off 16-byte borders");
@@ -543,14 +628,37 @@ extern "C" int srb_prefill_attention_tc_gated(const void* q, const void* k_pool,
   args.n_q = n_q; args.n_kv = n_kv; args.page_size = page_size; args.pool_rows = (int)pool_rows; args.window = window; args.chunk = chunk;
   args.scale_log2 = scale * 1.4426950408889634f; args.error_word = error_word;
   args.sinks = sinks; args.gates = gates; args.out_pitch = out_pitch; args.out_scale = out_scale;
+  args.keep_first = p.keep_first; args.cap_log2 = p.softcap * 1.4426950408889634f;
+  if (p.softcap > 0.f) args.scale_log2 *= 2.0f / p.softcap;
+  args.map_lambda = p.map_lambda; args.map_scale = p.map_scale; args.map_eps = p.map_eps;
   cudaStream_t s = (cudaStream_t)stream;
   // two query heads per block when the heads of a kv head pair up
-  const bool pairs = (n_q / n_kv) % 2 == 0;
-  if (head_dim == 64)
-    return pairs ? launch_tc<64, 2, 4>(map_q, map_k, map_v, map_out, args, num_tiles, s)
-                 : launch_tc<64, 1, 2>(map_q, map_k, map_v, map_out, args, num_tiles, s);
-  return pairs ? launch_tc<128, 2, 4>(map_q, map_k, map_v, map_out, args, num_tiles, s)
-               : launch_tc<128, 1, 2>(map_q, map_k, map_v, map_out, args, num_tiles, s);
+  const bool pairs = (n_q / n_kv) % 2 == 0, cap = p.softcap > 0.f;
+#define SRB_TC_LAUNCH(D, HEADS, STAGES, MAPS)                                                                        \
+  return cap ? launch_tc<D, HEADS, STAGES, MAPS, true>(map_q, map_k, map_v, map_out, args, num_tiles, s)             \
+             : launch_tc<D, HEADS, STAGES, MAPS, false>(map_q, map_k, map_v, map_out, args, num_tiles, s)
+  if (p.maps == 2) {
+    if (head_dim == 64) { SRB_TC_LAUNCH(64, 2, 4, true); }
+    SRB_TC_LAUNCH(128, 2, 4, true);
+  }
+  if (head_dim == 64) {
+    if (pairs) { SRB_TC_LAUNCH(64, 2, 4, false); }
+    SRB_TC_LAUNCH(64, 1, 2, false);
+  }
+  if (pairs) { SRB_TC_LAUNCH(128, 2, 4, false); }
+  SRB_TC_LAUNCH(128, 1, 2, false);
+#undef SRB_TC_LAUNCH
+}
+
+extern "C" int srb_prefill_attention_tc_gated(const void* q, const void* k_pool, const void* v_pool, void* out,
+                                              const int* tiles, int num_tiles, int rows, const int* block_table,
+                                              int table_stride, int n_q, int n_kv, int head_dim, int page_size,
+                                              int num_pages, int window, int chunk, float scale, int* error_word,
+                                              const float* sinks, const float* gates, long long out_pitch,
+                                              float out_scale, void* stream) {
+  return srb_prefill_attention_tc_terms(q, k_pool, v_pool, out, tiles, num_tiles, rows, block_table, table_stride, n_q, n_kv,
+                                        head_dim, page_size, num_pages, window, chunk, scale, error_word, sinks, gates,
+                                        out_pitch, out_scale, nullptr, stream);
 }
 
 extern "C" int srb_prefill_attention_tc_masked(const void* q, const void* k_pool, const void* v_pool, void* out,

@@ -349,13 +349,13 @@ __global__ void norm_add_norm_kernel(float* __restrict__ residual, const T* __re
                                      const float* __restrict__ delta_f32, NormSpec inner, NormSpec outer,
                                      T* __restrict__ out, size_t out_pitch, const float* __restrict__ extra,
                                      const int* __restrict__ row_index, int width, int write_residual,
-                                     const float* __restrict__ addend, int num_parts, size_t part_stride) {
+                                     const float* __restrict__ addend, size_t addend_pitch, int num_parts, size_t part_stride) {
   extern __shared__ float staged[];          // width floats, then 33 floats of scratch
   float* scratch = staged + width;
   srb_launch_dependents();
   srb_grid_dependency_wait();
   const int row = blockIdx.x;
-  const size_t src = (size_t)(row_index ? row_index[row] : row) * width;
+  const size_t src_row = row_index ? row_index[row] : row, src = src_row * width;
   const bool pending = delta || delta_f32;
   if (pending) {
     if (num_parts > 0) {
@@ -383,7 +383,7 @@ __global__ void norm_add_norm_kernel(float* __restrict__ residual, const T* __re
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
     float x = residual[src + i];
     if (pending) x += staged[i];
-    if (addend) x += addend[src + i];
+    if (addend) x += addend[src_row * addend_pitch + i];
     if (write_residual && (pending || addend)) residual[src + i] = x;
     staged[i] = x;
   }
@@ -403,7 +403,8 @@ template <typename T, int ITEMS, bool PARTS>
 __global__ void __launch_bounds__(ITEMS == 1 ? 1024 : 256, ITEMS == 1 ? 1 : (ITEMS == 2 ? 4 : 1))
 norm_add_norm_vec_kernel(float* __restrict__ residual, const T* __restrict__ delta, const float* __restrict__ delta_f32,
                          NormSpec inner, NormSpec outer, T* __restrict__ out, size_t out_pitch, const int* __restrict__ row_index,
-                         int width, int write_residual, const float* __restrict__ addend, int num_parts, size_t part_stride) {
+                         int width, int write_residual, const float* __restrict__ addend, size_t addend_pitch, int num_parts,
+                         size_t part_stride) {
   __shared__ float scratch[33];
   srb_launch_dependents();
   const int step = blockDim.x * 4;
@@ -416,7 +417,7 @@ norm_add_norm_vec_kernel(float* __restrict__ residual, const T* __restrict__ del
     if (i < width && out && outer.kind != SRB_NORM_NONE) wo[it] = *reinterpret_cast<const float4*>(outer.weight + i);
   }
   srb_grid_dependency_wait();
-  const size_t src = (size_t)(row_index ? row_index[blockIdx.x] : blockIdx.x) * width;
+  const size_t src_row = row_index ? row_index[blockIdx.x] : blockIdx.x, src = src_row * width;
   const bool pending = delta || delta_f32;
   float4 x[ITEMS], d[ITEMS];
   float squares = 0.f;
@@ -470,7 +471,7 @@ norm_add_norm_vec_kernel(float* __restrict__ residual, const T* __restrict__ del
     const int i = threadIdx.x * 4 + it * step;
     if (i >= width) break;
     if (addend) {
-      const float4 a = load4(addend + src + i);
+      const float4 a = load4(addend + src_row * addend_pitch + i);
       x[it].x += a.x; x[it].y += a.y; x[it].z += a.z; x[it].w += a.w;
     }
     if (write_residual && (pending || addend)) *reinterpret_cast<float4*>(residual + src + i) = x[it];
@@ -494,7 +495,7 @@ norm_add_norm_vec_kernel(float* __restrict__ residual, const T* __restrict__ del
 template <typename T>
 static int launch_norm_add_norm_vec(float* residual, const void* delta, const float* delta_f32, const NormSpec& inner, const NormSpec& outer,
                                     void* out, long long out_pitch, const int* row_index, int rows, int width, int write_residual,
-                                    const float* addend, int num_parts, long long part_stride, cudaStream_t s) {
+                                    const float* addend, long long addend_pitch, int num_parts, long long part_stride, cudaStream_t s) {
   const int quads = width / 4;
   // few rows: as many threads as the row has pieces; many: two pieces a thread
   const int items = quads <= 1024 && rows <= 64 ? 1 : (quads <= 512 ? 2 : (quads <= 1024 ? 4 : 8));
@@ -502,7 +503,7 @@ static int launch_norm_add_norm_vec(float* residual, const void* delta, const fl
 #define SRB_NORM_VEC(ITEMS)                                                                                                    \
   SRB_CUDA_CALL(srb_launch(num_parts > 0 ? norm_add_norm_vec_kernel<T, ITEMS, true> : norm_add_norm_vec_kernel<T, ITEMS, false>, dim3(rows), dim3(threads), 0, s, residual, (const T*)delta,    \
                            delta_f32, inner, outer, (T*)out, (size_t)out_pitch, row_index, width, write_residual, addend,     \
-                           num_parts, (size_t)part_stride))
+                           (size_t)addend_pitch, num_parts, (size_t)part_stride))
   if (items == 1) SRB_NORM_VEC(1);
   else if (items == 2) SRB_NORM_VEC(2);
   else if (items == 4) SRB_NORM_VEC(4);
@@ -513,7 +514,8 @@ static int launch_norm_add_norm_vec(float* residual, const void* delta, const fl
 }
 
 // `*_groups` (RMS norms only; 1: the whole row) and `*_scale` (1: none) as NormSpec says.  `addend` (optional, float,
-// shaped like the residual): a second term of the sum, added after the pending one: x = residual + inner(delta) + addend.
+// rows `addend_pitch` floats apart; 0: one row for all): a second term of the sum, added after the pending one: x = residual +
+// inner(delta) + addend.
 // `num_parts` > 0: `delta_f32` holds that many partial sums of the pending term, `part_stride` floats apart, which are
 // added in part order before the inner norm.
 extern "C" int srb_norm_add_norm_parts(float* residual, const void* delta, const float* delta_f32, int inner_kind,
@@ -521,7 +523,8 @@ extern "C" int srb_norm_add_norm_parts(float* residual, const void* delta, const
                                     float inner_scale, int outer_kind, const float* outer_weight, const float* outer_bias,
                                     float outer_eps, int outer_groups, float outer_scale, void* out, long long out_pitch,
                                     const float* extra, const int* row_index, int rows, int width, int write_residual,
-                                    int dtype, const float* addend, int num_parts, long long part_stride, void* stream) {
+                                    int dtype, const float* addend, long long addend_pitch, int num_parts, long long part_stride,
+                                    void* stream) {
   if (rows <= 0) return SRB_OK;
   if (num_parts < 0 || (num_parts > 0 && (!delta_f32 || delta))) SRB_FAIL("norm_add_norm: partial sums come as float and alone");
   for (int groups : {inner_groups, outer_groups})
@@ -543,28 +546,28 @@ extern "C" int srb_norm_add_norm_parts(float* residual, const void* delta, const
   cudaStream_t s = (cudaStream_t)stream;
   const size_t element = dtype == SRB_DTYPE_BF16 ? 2 : 4;
   const bool plain = inner_kind != SRB_NORM_LAYER && outer_kind != SRB_NORM_LAYER && inner_groups == 1 && outer_groups == 1 && !extra &&
-                     width % 4 == 0 && width <= 8192 && out_pitch % 4 == 0 && part_stride % 4 == 0 &&
+                     width % 4 == 0 && width <= 8192 && out_pitch % 4 == 0 && part_stride % 4 == 0 && addend_pitch % 4 == 0 &&
                      (((uintptr_t)residual | (uintptr_t)delta_f32 | (uintptr_t)addend | (uintptr_t)inner_weight | (uintptr_t)outer_weight) & 15) == 0 &&
                      (((uintptr_t)delta | (uintptr_t)out) & (4 * element - 1)) == 0;
   if (plain && dtype == SRB_DTYPE_F32)
     return launch_norm_add_norm_vec<float>(residual, delta, delta_f32, inner, outer, out, out_pitch, row_index, rows, width, write_residual,
-                                           addend, num_parts, part_stride, s);
+                                           addend, addend_pitch, num_parts, part_stride, s);
   if (plain && dtype == SRB_DTYPE_BF16)
     return launch_norm_add_norm_vec<__nv_bfloat16>(residual, delta, delta_f32, inner, outer, out, out_pitch, row_index, rows, width,
-                                                   write_residual, addend, num_parts, part_stride, s);
+                                                   write_residual, addend, addend_pitch, num_parts, part_stride, s);
   if (dtype == SRB_DTYPE_F32) {
     if (smem > 48 * 1024)
       SRB_CUDA_CALL(cudaFuncSetAttribute(norm_add_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     SRB_CUDA_CALL(srb_launch(norm_add_norm_kernel<float>, dim3(rows), dim3(block), smem, s, residual, (const float*)delta,
                              delta_f32, inner, outer, (float*)out, (size_t)out_pitch, extra, row_index, width,
-                             write_residual, addend, num_parts, (size_t)part_stride));
+                             write_residual, addend, (size_t)addend_pitch, num_parts, (size_t)part_stride));
   } else if (dtype == SRB_DTYPE_BF16) {
     if (smem > 48 * 1024)
       SRB_CUDA_CALL(cudaFuncSetAttribute(norm_add_norm_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          (int)smem));
     SRB_CUDA_CALL(srb_launch(norm_add_norm_kernel<__nv_bfloat16>, dim3(rows), dim3(block), smem, s, residual,
                              (const __nv_bfloat16*)delta, delta_f32, inner, outer, (__nv_bfloat16*)out, (size_t)out_pitch,
-                             extra, row_index, width, write_residual, addend, num_parts, (size_t)part_stride));
+                             extra, row_index, width, write_residual, addend, (size_t)addend_pitch, num_parts, (size_t)part_stride));
   } else {
     SRB_FAIL("norm_add_norm: unknown dtype %d", dtype);
   }
@@ -580,7 +583,7 @@ extern "C" int srb_norm_add_norm_ex(float* residual, const void* delta, const fl
                                     int dtype, void* stream) {
   return srb_norm_add_norm_parts(residual, delta, delta_f32, inner_kind, inner_weight, inner_bias, inner_eps, inner_groups,
                                  inner_scale, outer_kind, outer_weight, outer_bias, outer_eps, outer_groups, outer_scale, out,
-                                 out_pitch, extra, row_index, rows, width, write_residual, dtype, nullptr, 0, 0, stream);
+                                 out_pitch, extra, row_index, rows, width, write_residual, dtype, nullptr, 0, 0, 0, stream);
 }
 
 extern "C" int srb_norm_add_norm(float* residual, const void* delta, const float* delta_f32, int inner_kind,

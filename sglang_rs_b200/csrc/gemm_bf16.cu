@@ -67,6 +67,7 @@ struct GemmArgs {
   // BLOCK_T - 1 as far as they belong to the expert, and whose weight rows start at expert * expert_rows.  Null: off.
   const int* plan;
   int experts, expert_rows;
+  const float* slot_weight;  // a factor on the input of every slot (its sums are multiplied by it), or null
 };
 
 template <int BLOCK_T, int EPI, int STAGES>
@@ -235,7 +236,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
           for (int j = 0; j < 16; ++j) {
             const int token = token0 + c + j;
             if (token >= token_limit) break;
-            const float g = acc[j], u = exchange[((quarter & 1) * 32 + lane) * 16 + j];
+            const float weight = args.slot_weight ? args.slot_weight[token] : 1.0f;
+            const float g = acc[j] * weight, u = exchange[((quarter & 1) * 32 + lane) * 16 + j] * weight;
             reinterpret_cast<__nv_bfloat16*>(args.out)[(size_t)token * args.ldo + feature] =
                 __float2bfloat16_rn(srb_gated<true>(args.activation, g, u, args.act_param));
           }
@@ -254,7 +256,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             reinterpret_cast<__nv_bfloat16*>(args.out)[(size_t)token * args.ldo + feature] = __float2bfloat16_rn(acc[j]);
           } else if (EPI == EPI_ACT) {
             reinterpret_cast<__nv_bfloat16*>(args.out)[(size_t)token * args.ldo + feature] =
-                __float2bfloat16_rn(srb_gated<true>(args.activation, acc[j], 1.0f, args.act_param));
+                __float2bfloat16_rn(srb_gated<true>(args.activation, args.slot_weight ? acc[j] * args.slot_weight[token] : acc[j], 1.0f, args.act_param));
           } else if (EPI == EPI_F32) {
             reinterpret_cast<float*>(args.out)[(size_t)token * args.ldo + feature] = acc[j];
           } else {
@@ -411,7 +413,7 @@ extern "C" int srb_gemm_bf16_param(const void* x, const void* w, void* out, int 
   args.out = out; args.tokens = tokens; args.features = features; args.k = k; args.ldo = ldo;
   args.up_row_offset = up_row_offset; args.activation = activation; args.error_word = error_word;
   args.act_param = act_param;
-  args.plan = nullptr; args.experts = 0; args.expert_rows = 0;
+  args.plan = nullptr; args.experts = 0; args.expert_rows = 0; args.slot_weight = nullptr;
   args.k_blocks_per_split = (total_k_blocks + splits - 1) / splits;
   const int used_splits = (total_k_blocks + args.k_blocks_per_split - 1) / args.k_blocks_per_split;
   if (used_splits != splits) SRB_FAIL("gemm_bf16: %d splits leave one without work for %d blocks of K", splits, total_k_blocks);
@@ -441,7 +443,8 @@ extern "C" int srb_gemm_bf16(const void* x, const void* w, void* out, int tokens
 // plan as in GemmArgs, with tiles of `tile_slots` slots (128 or 256) and room for `max_tiles` of them.  mode 1: out float [slots, ldo] =
 // x w_e^T over `features` rows of the expert's matrix; mode 2: the expert's matrix stacks gate rows [0, features) over
 // up rows [up_row_offset, + features), out bf16 [slots, ldo] = act(gate) * up.  Blocks of tiles beyond the plan's
-// count leave at once; rows of a tile behind its expert's last slot are computed and not stored.
+// count leave at once; rows of a tile behind its expert's last slot are computed and not stored.  `slot_weight` (float [slots],
+// or null): a factor on the input of every slot, taken on the 32-bit sums (modes 2 and 5).
 template <int EPI, int BLOCK_T>
 static int launch_grouped(const CUtensorMap& map_w, const CUtensorMap& map_x, const GemmArgs& args, int max_tiles,
                           cudaStream_t s) {
@@ -460,7 +463,8 @@ static int launch_grouped(const CUtensorMap& map_w, const CUtensorMap& map_x, co
 
 extern "C" int srb_gemm_bf16_grouped(const void* x, const void* w, void* out, const int* plan, int max_tiles, int tile_slots,
                                      int slots, int experts, int expert_rows, int features, int k, int ldo,
-                                     int up_row_offset, int mode, int activation, float act_param, int* error_word, void* stream) {
+                                     int up_row_offset, int mode, int activation, float act_param, const float* slot_weight,
+                                     int* error_word, void* stream) {
   if (slots <= 0 || features <= 0 || max_tiles <= 0) return SRB_OK;
   if (tile_slots != 128 && tile_slots != 256) SRB_FAIL("gemm_bf16_grouped: tiles of %d slots are not 128 or 256", tile_slots);
   if (k <= 0 || k % 8 != 0) SRB_FAIL("gemm_bf16_grouped: inner size %d must be a positive multiple of 8", k);
@@ -480,7 +484,7 @@ extern "C" int srb_gemm_bf16_grouped(const void* x, const void* w, void* out, co
   args.out = out; args.tokens = slots; args.features = features; args.k = k; args.ldo = ldo;
   args.up_row_offset = up_row_offset; args.activation = activation; args.error_word = error_word;
   args.act_param = act_param;
-  args.plan = plan; args.experts = experts; args.expert_rows = expert_rows;
+  args.plan = plan; args.experts = experts; args.expert_rows = expert_rows; args.slot_weight = slot_weight;
   args.k_blocks_per_split = (k + GEMM_BLOCK_K - 1) / GEMM_BLOCK_K;
   cudaStream_t s = (cudaStream_t)stream;
   if (tile_slots == 256)

@@ -34,6 +34,7 @@ int fail(int code, const char* format, ...) {
 
 struct Group {
   int window = 0;                  // 0: every key is kept
+  int keep_first = 0;              // with a window: the sequence's first tokens that stay visible behind it
   int num_pages = 0;
   std::vector<int> refs;
   std::vector<int> free_stack;     // back() is handed out next
@@ -88,8 +89,10 @@ extern "C" {
 
 const char* srb_last_error() { return error_text; }
 
-// windows[g] = 0 for a group that keeps every key; num_pages[g] pages per group
-void* hc_create(int page_size, int num_groups, const int* windows, const int* num_pages, int max_requests) {
+// windows[g] = 0 for a group that keeps every key; num_pages[g] pages per group; keep_first[g] (or a null array: none): how
+// many of a sequence's first tokens stay visible once the window has passed them: their pages are not given back
+void* hc_create(int page_size, int num_groups, const int* windows, const int* keep_first, const int* num_pages,
+                int max_requests) {
   if (page_size <= 0 || num_groups < 0 || max_requests <= 0) return nullptr;
   Core* core = new Core();
   core->page_size = page_size;
@@ -101,6 +104,7 @@ void* hc_create(int page_size, int num_groups, const int* windows, const int* nu
       return nullptr;
     }
     group.window = windows[g];
+    group.keep_first = keep_first ? std::max(0, keep_first[g]) : 0;
     group.num_pages = num_pages[g];
     group.refs.assign(num_pages[g], 0);
     group.free_stack.resize(num_pages[g]);
@@ -299,7 +303,7 @@ int hc_capacity(void* handle, int r) {
   return (int)least;
 }
 
-// `tokens` more tokens are stored; pages a window has passed are given back
+// `tokens` more tokens are stored; pages a window has passed are given back, but for those of the kept first tokens
 int hc_commit(void* handle, int r, int tokens) {
   Core* core = static_cast<Core*>(handle);
   if (!good_request(core, r) || tokens < 0) return fail(-4, "request %d has ended", r);
@@ -313,7 +317,8 @@ int hc_commit(void* handle, int r, int tokens) {
     const int first_kept = std::max(0, request.length - group.window + 1);
     std::vector<int>& table = request.tables[g];
     const int passed = std::min((int)table.size(), first_kept / core->page_size);
-    for (int logical = passed - 1; logical >= 0 && table[logical] >= 0; --logical) {   // earlier ones went before
+    const int kept = pages_for(core, group.keep_first);
+    for (int logical = passed - 1; logical >= kept && table[logical] >= 0; --logical) {   // earlier ones went before
       if (release_page(group, table[logical]) < 0) return -4;
       table[logical] = -1;
     }

@@ -11,6 +11,11 @@
 //   srb_moe_down      y[slot, :]   = W_down[e] act[slot]                              (32-bit result)
 //   srb_moe_combine   out[row, :]  = sum over the row's choices, in their order, of weight * y[slot]   (32-bit)
 //
+// A weight may belong to an expert's input instead of its result (act = activation(W_gate (w h)) ...): the plan then notes
+// the weight of every slot (`slot_weight`), the first products multiply their 32-bit sums by it, since W (w h) = w (W h), and
+// the sum takes the results as they are (null weights).  The router matrix may have one row more, a gate for the term that
+// every row gets beside its experts': its logit's sigmoid goes to `base_gate` and multiplies that term in the sum.
+//
 // The router may have more outputs than there are experts with matrices (srb_moe_route / srb_moe_select are then called
 // with the number of outputs, srb_moe_plan and the products with the number of experts): a choice beyond the experts gets
 // no slot, the products never see it, and srb_moe_combine_identity adds weight * h[row] for it: an expert that returns
@@ -107,13 +112,15 @@ __device__ __forceinline__ void moe_choose(float* score, float* pick, int expert
 // One block per row.  Warps share the experts' dot products; warp 0 then picks the largest scores.
 template <typename T>
 __global__ void moe_route_kernel(const T* __restrict__ h, const T* __restrict__ router, int width, int experts, int top,
-                                 RouteRule rule, int* __restrict__ chosen, float* __restrict__ weights) {
-  __shared__ float score[MOE_MAX_EXPERTS];
+                                 RouteRule rule, int* __restrict__ chosen, float* __restrict__ weights,
+                                 float* __restrict__ base_gate) {
+  __shared__ float score[MOE_MAX_EXPERTS + 1];
   __shared__ float pick[MOE_MAX_EXPERTS];
   srb_launch_dependents();
   srb_grid_dependency_wait();
   const int row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   const T* x = h + (size_t)row * width;
+  const int outputs = experts + (base_gate ? 1 : 0);
   if (sizeof(T) == 2 && width % 8 == 0 && (((uintptr_t)h | (uintptr_t)router) & 15) == 0) {
     // 16-byte loads: a lane's pieces of the row stay in registers for every expert of its warp (up to 4 pieces:
     // widths to 1024; wider rows read the later pieces again per expert)
@@ -122,7 +129,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const T* __restrict__ 
 #pragma unroll
     for (int j = 0; j < 4; ++j)
       mine[j] = lane + 32 * j < pieces ? *reinterpret_cast<const uint4*>(x + (size_t)(lane + 32 * j) * 8) : make_uint4(0u, 0u, 0u, 0u);
-    for (int e = warp; e < experts; e += warps) {
+    for (int e = warp; e < outputs; e += warps) {
       const T* w = router + (size_t)e * width;
       float partial = 0.f;
       for (int piece = lane, j = 0; piece < pieces; piece += 32, ++j) {
@@ -141,7 +148,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const T* __restrict__ 
       if (lane == 0) score[e] = partial;
     }
   } else {
-    for (int e = warp; e < experts; e += warps) {
+    for (int e = warp; e < outputs; e += warps) {
       const T* w = router + (size_t)e * width;
       float partial = 0.f;
       for (int i = lane; i < width; i += 32) partial += srb_to_float(x[i]) * srb_to_float(w[i]);
@@ -151,12 +158,13 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const T* __restrict__ 
   }
   __syncthreads();
   if (warp != 0) return;
+  if (base_gate && lane == 0) base_gate[row] = 1.0f / (1.0f + expf(-score[experts]));
   moe_choose(score, pick, experts, top, rule, lane, chosen + (size_t)row * top, weights + (size_t)row * top);
 }
 
 extern "C" int srb_moe_route_ex(const void* h, const void* router, int rows, int width, int experts, int top, int renormalize,
                                 int scoring, const float* choice_bias, float scale, float norm_eps, int* chosen, float* weights,
-                                int dtype, void* stream) {
+                                float* base_gate, int dtype, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (scoring != MOE_SCORE_SOFTMAX && scoring != MOE_SCORE_SIGMOID) SRB_FAIL("moe_route: unknown scoring %d", scoring);
   const RouteRule rule{scoring, renormalize, choice_bias, scale, norm_eps};
@@ -164,13 +172,14 @@ extern "C" int srb_moe_route_ex(const void* h, const void* router, int rows, int
   if (top <= 0 || top > experts || top > 32) SRB_FAIL("moe_route: %d chosen experts are outside 1 .. min(%d, 32)", top, experts);
   if (width <= 0) SRB_FAIL("moe_route: width %d must be positive", width);
   cudaStream_t s = (cudaStream_t)stream;
-  const int block = experts >= 32 ? 1024 : 32 * experts;          // a warp per expert, up to 32 warps
+  const int outputs = experts + (base_gate ? 1 : 0);
+  const int block = outputs >= 32 ? 1024 : 32 * outputs;          // a warp per output, up to 32 warps
   if (dtype == SRB_DTYPE_F32)
     SRB_CUDA_CALL(srb_launch(moe_route_kernel<float>, dim3(rows), dim3(block), 0, s, (const float*)h, (const float*)router,
-                             width, experts, top, rule, chosen, weights));
+                             width, experts, top, rule, chosen, weights, base_gate));
   else if (dtype == SRB_DTYPE_BF16)
     SRB_CUDA_CALL(srb_launch(moe_route_kernel<__nv_bfloat16>, dim3(rows), dim3(block), 0, s, (const __nv_bfloat16*)h,
-                             (const __nv_bfloat16*)router, width, experts, top, rule, chosen, weights));
+                             (const __nv_bfloat16*)router, width, experts, top, rule, chosen, weights, base_gate));
   else
     SRB_FAIL("moe_route: unknown dtype %d", dtype);
   SRB_LAUNCH_CHECK("moe_route");
@@ -180,13 +189,14 @@ extern "C" int srb_moe_route_ex(const void* h, const void* router, int rows, int
 extern "C" int srb_moe_route(const void* h, const void* router, int rows, int width, int experts, int top, int renormalize,
                              int* chosen, float* weights, int dtype, void* stream) {
   return srb_moe_route_ex(h, router, rows, width, experts, top, renormalize, MOE_SCORE_SOFTMAX, nullptr, 1.0f, 0.0f, chosen,
-                          weights, dtype, stream);
+                          weights, nullptr, dtype, stream);
 }
 
 // The choice alone, from logits that a product kernel made (float [rows, experts], `pitch` floats apart): a warp per
 // row does the softmax over all experts and picks the `top` largest as moe_route_kernel does.
 __global__ void moe_select_kernel(const float* __restrict__ logits, size_t pitch, int rows, int experts, int top,
-                                  RouteRule rule, int* __restrict__ chosen, float* __restrict__ weights) {
+                                  RouteRule rule, int* __restrict__ chosen, float* __restrict__ weights,
+                                  float* __restrict__ base_gate) {
   extern __shared__ float select_scores[];                  // [warps of the block][2][experts]
   srb_launch_dependents();
   srb_grid_dependency_wait();
@@ -196,21 +206,22 @@ __global__ void moe_select_kernel(const float* __restrict__ logits, size_t pitch
   float* score = select_scores + (size_t)warp * 2 * experts;
   const float* z = logits + (size_t)row * pitch;
   for (int e = lane; e < experts; e += 32) score[e] = z[e];
+  if (base_gate && lane == 0) base_gate[row] = 1.0f / (1.0f + expf(-z[experts]));
   moe_choose(score, score + experts, experts, top, rule, lane, chosen + (size_t)row * top, weights + (size_t)row * top);
 }
 
 extern "C" int srb_moe_select_ex(const float* logits, long long pitch, int rows, int experts, int top, int renormalize,
                                  int scoring, const float* choice_bias, float scale, float norm_eps, int* chosen,
-                                 float* weights, void* stream) {
+                                 float* weights, float* base_gate, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (scoring != MOE_SCORE_SOFTMAX && scoring != MOE_SCORE_SIGMOID) SRB_FAIL("moe_select: unknown scoring %d", scoring);
   const RouteRule rule{scoring, renormalize, choice_bias, scale, norm_eps};
   if (experts <= 0 || experts > MOE_MAX_EXPERTS) SRB_FAIL("moe_select: %d experts are outside 1 .. %d", experts, MOE_MAX_EXPERTS);
   if (top <= 0 || top > experts || top > 32) SRB_FAIL("moe_select: %d chosen experts are outside 1 .. min(%d, 32)", top, experts);
-  if (pitch < experts) SRB_FAIL("moe_select: rows of the logits overlap");
+  if (pitch < experts + (base_gate ? 1 : 0)) SRB_FAIL("moe_select: rows of the logits overlap");
   const int warps = 4;
   SRB_CUDA_CALL(srb_launch(moe_select_kernel, dim3((rows + warps - 1) / warps), dim3(32 * warps), (size_t)warps * experts * 8,
-                           (cudaStream_t)stream, logits, (size_t)pitch, rows, experts, top, rule, chosen, weights));
+                           (cudaStream_t)stream, logits, (size_t)pitch, rows, experts, top, rule, chosen, weights, base_gate));
   SRB_LAUNCH_CHECK("moe_select");
   return SRB_OK;
 }
@@ -218,14 +229,14 @@ extern "C" int srb_moe_select_ex(const float* logits, long long pitch, int rows,
 extern "C" int srb_moe_select(const float* logits, long long pitch, int rows, int experts, int top, int renormalize,
                               int* chosen, float* weights, void* stream) {
   return srb_moe_select_ex(logits, pitch, rows, experts, top, renormalize, MOE_SCORE_SOFTMAX, nullptr, 1.0f, 0.0f, chosen,
-                           weights, stream);
+                           weights, nullptr, stream);
 }
 
 // One block.  plan: [0] number of tiles, then offsets[experts + 1], then per tile (expert, first slot).
 // slot_row[slot]: the row whose entry sits in the slot; entry_slot[row * top + k]: the slot of that entry.
 __global__ void moe_plan_kernel(const int* __restrict__ chosen, int entries, int top, int experts, int max_tiles,
                                 int tile_rows, int* __restrict__ plan, int* __restrict__ slot_row, int* __restrict__ entry_slot,
-                                int* error_word) {
+                                const float* __restrict__ weights, float* __restrict__ slot_weight, int* error_word) {
   __shared__ int count[MOE_MAX_EXPERTS];
   __shared__ int first[MOE_MAX_EXPERTS + 1];
   __shared__ int tile_first[MOE_MAX_EXPERTS + 1];
@@ -272,6 +283,7 @@ __global__ void moe_plan_kernel(const int* __restrict__ chosen, int entries, int
     if (e < 0 || e >= experts) { entry_slot[i] = -1; continue; }
     const int slot = first[e] + atomicAdd(&count[e], 1);
     slot_row[slot] = i / top;
+    if (slot_weight) slot_weight[slot] = weights[i];
     entry_slot[i] = slot;
   }
 }
@@ -287,28 +299,27 @@ extern "C" int srb_moe_plan_ints_of(int rows, int top, int experts, int tile_row
   return 1 + experts + 1 + 2 * ((rows * top) / tile_rows + experts);
 }
 extern "C" int srb_moe_max_tiles_of(int rows, int top, int experts, int tile_rows) { return (rows * top) / tile_rows + experts; }
-extern "C" int srb_moe_plan_of(const int* chosen, int rows, int top, int experts, int tile_rows, int* plan, int* slot_row,
-                               int* entry_slot, int* error_word, void* stream);
 
 extern "C" int srb_moe_max_tiles(int rows, int top, int experts) {
   return (rows * top) / moe_tile_rows(rows, top, experts) + experts;
 }
 
+// `slot_weight` (or null) receives the weight of every slot's choice from `weights` [rows * top].
 extern "C" int srb_moe_plan_of(const int* chosen, int rows, int top, int experts, int tile_rows, int* plan, int* slot_row,
-                               int* entry_slot, int* error_word, void* stream) {
+                               int* entry_slot, const float* weights, float* slot_weight, int* error_word, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0 || tile_rows <= 0)
     SRB_FAIL("moe_plan: %d experts, %d chosen, tiles of %d", experts, top, tile_rows);
   SRB_CUDA_CALL(srb_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, (cudaStream_t)stream, chosen, rows * top, top, experts,
-                           (rows * top) / tile_rows + experts, tile_rows, plan, slot_row, entry_slot, error_word));
+                           (rows * top) / tile_rows + experts, tile_rows, plan, slot_row, entry_slot, weights, slot_weight, error_word));
   SRB_LAUNCH_CHECK("moe_plan");
   return SRB_OK;
 }
 
 extern "C" int srb_moe_plan(const int* chosen, int rows, int top, int experts, int* plan, int* slot_row, int* entry_slot,
                             int* error_word, void* stream) {
-  return srb_moe_plan_of(chosen, rows, top, experts, moe_tile_rows(rows, top, experts), plan, slot_row, entry_slot, error_word,
-                         stream);
+  return srb_moe_plan_of(chosen, rows, top, experts, moe_tile_rows(rows, top, experts), plan, slot_row, entry_slot, nullptr, nullptr,
+                         error_word, stream);
 }
 
 // Half a tile (up to 64 slots of one expert; blockIdx.z names the half) times 64 output columns.  GATED: two weight matrices (gate, up), rows of
@@ -322,7 +333,8 @@ template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 moe_product_kernel(const T* __restrict__ x, const T* __restrict__ w_a, const T* __restrict__ w_b,
                    const int* __restrict__ plan, const int* __restrict__ slot_row, int experts, int n_in, int n_out,
-                   int activation, float act_param, T* __restrict__ out_t, float* __restrict__ out_f, int tile_rows, size_t expert_stride) {
+                   int activation, float act_param, T* __restrict__ out_t, float* __restrict__ out_f, int tile_rows, size_t expert_stride,
+                   const float* __restrict__ slot_weight) {
   constexpr bool GATED = MODE == MOE_GATED, GATHER = MODE != MOE_DOWN;
   __shared__ float x_tile[MOE_K][MOE_TILE + 4];
   __shared__ float a_tile[MOE_K][MOE_TILE + 4];
@@ -381,14 +393,15 @@ moe_product_kernel(const T* __restrict__ x, const T* __restrict__ w_a, const T* 
     const int r = ty * 4 + i;
     if (r >= count) continue;
     const size_t slot = (size_t)first + r;
+    const float weight = MODE != MOE_DOWN && slot_weight ? slot_weight[slot] : 1.0f;       // on the expert's input
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int c = col0 + tx * 4 + j;
       if (c >= n_out) continue;
       if (GATED)
-        out_t[slot * n_out + c] = srb_from_float<T>(srb_gated<true>(activation, acc_a[i][j], acc_b[i][j], act_param));
+        out_t[slot * n_out + c] = srb_from_float<T>(srb_gated<true>(activation, acc_a[i][j] * weight, acc_b[i][j] * weight, act_param));
       else if (MODE == MOE_ACT)
-        out_t[slot * n_out + c] = srb_from_float<T>(srb_gated<true>(activation, acc_a[i][j], 1.0f, act_param));
+        out_t[slot * n_out + c] = srb_from_float<T>(srb_gated<true>(activation, acc_a[i][j] * weight, 1.0f, act_param));
       else
         out_f[slot * n_out + c] = acc_a[i][j];
     }
@@ -401,7 +414,8 @@ __global__ void __launch_bounds__(128)
 moe_product_mma_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w_a,
                        const __nv_bfloat16* __restrict__ w_b, const int* __restrict__ plan,
                        const int* __restrict__ slot_row, int experts, int n_in, int n_out, int activation, float act_param,
-                       __nv_bfloat16* __restrict__ out_t, float* __restrict__ out_f, int tile_rows, size_t expert_stride) {
+                       __nv_bfloat16* __restrict__ out_t, float* __restrict__ out_f, int tile_rows, size_t expert_stride,
+                   const float* __restrict__ slot_weight) {
   constexpr bool GATED = MODE == MOE_GATED, GATHER = MODE != MOE_DOWN;
   __shared__ __align__(16) TileMmaSmem s;
   srb_launch_dependents();
@@ -436,10 +450,11 @@ moe_product_mma_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16*
         const int r = tile_mma_row(i, c), col = col0 + tile_mma_col(j, c);
         if (r >= count || col >= n_out) continue;
         const size_t at = ((size_t)first + r) * n_out + col;
+        const float weight = MODE != MOE_DOWN && slot_weight ? slot_weight[first + r] : 1.0f;   // on the expert's input
         if (GATED)
-          out_t[at] = __float2bfloat16_rn(srb_gated<true>(activation, acc[0][i][j][c], acc[NW - 1][i][j][c], act_param));
+          out_t[at] = __float2bfloat16_rn(srb_gated<true>(activation, acc[0][i][j][c] * weight, acc[NW - 1][i][j][c] * weight, act_param));
         else if (MODE == MOE_ACT)
-          out_t[at] = __float2bfloat16_rn(srb_gated<true>(activation, acc[0][i][j][c], 1.0f, act_param));
+          out_t[at] = __float2bfloat16_rn(srb_gated<true>(activation, acc[0][i][j][c] * weight, 1.0f, act_param));
         else
           out_f[at] = acc[0][i][j][c];
       }
@@ -452,7 +467,8 @@ __global__ void __launch_bounds__(256)
 moe_product_async_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w_a,
                          const __nv_bfloat16* __restrict__ w_b, const int* __restrict__ plan,
                          const int* __restrict__ slot_row, int experts, int n_in, int n_out, int activation, float act_param,
-                         __nv_bfloat16* __restrict__ out_t, float* __restrict__ out_f, size_t expert_stride) {
+                         __nv_bfloat16* __restrict__ out_t, float* __restrict__ out_f, size_t expert_stride,
+                         const float* __restrict__ slot_weight) {
   constexpr bool GATED = MODE == MOE_GATED, GATHER = MODE != MOE_DOWN;
   constexpr int NW = GATED ? 2 : 1;
   extern __shared__ __align__(16) unsigned char moe_smem[];
@@ -489,8 +505,9 @@ moe_product_async_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat1
         const size_t at = ((size_t)first + r) * n_out + col;
         const bool pair = col + 1 < n_out;
         if (MODE != MOE_DOWN) {
-          const float lo = srb_gated<true>(activation, acc[0][i][j][c], GATED ? acc[NW - 1][i][j][c] : 1.0f, act_param);
-          const float hi = srb_gated<true>(activation, acc[0][i][j][c + 1], GATED ? acc[NW - 1][i][j][c + 1] : 1.0f, act_param);
+          const float weight = slot_weight ? slot_weight[first + r] : 1.0f;                    // on the expert's input
+          const float lo = srb_gated<true>(activation, acc[0][i][j][c] * weight, GATED ? acc[NW - 1][i][j][c] * weight : 1.0f, act_param);
+          const float hi = srb_gated<true>(activation, acc[0][i][j][c + 1] * weight, GATED ? acc[NW - 1][i][j][c + 1] * weight : 1.0f, act_param);
           if (pair && (at & 1) == 0) {
             *reinterpret_cast<unsigned*>(out_t + at) = pack_bf16(lo, hi);
           } else {
@@ -509,7 +526,7 @@ moe_product_async_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat1
 template <typename T>
 static int launch_moe_products(int mode, const void* x, const void* w_a, const void* w_b, const int* plan,
                                const int* slot_row, int rows, int top, int experts, int n_in, int n_out, int activation, float act_param,
-                               void* out_t, float* out_f, size_t expert_stride, cudaStream_t s) {
+                               void* out_t, float* out_f, size_t expert_stride, const float* slot_weight, cudaStream_t s) {
   const int tile_rows = moe_tile_rows(rows, top, experts);
   dim3 grid((n_out + MOE_TILE - 1) / MOE_TILE, srb_moe_max_tiles(rows, top, experts), (tile_rows + MOE_TILE - 1) / MOE_TILE);
   if (grid.y > 65535) SRB_FAIL("moe product: %d tiles exceed one launch", (int)grid.y);
@@ -523,7 +540,7 @@ static int launch_moe_products(int mode, const void* x, const void* w_a, const v
                                        cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));                       \
     SRB_CUDA_CALL(srb_launch(moe_product_async_kernel<MODE, ROWS, STAGES>, grid, dim3(256), smem, s,                   \
                              (const __nv_bfloat16*)x, (const __nv_bfloat16*)w_a, (const __nv_bfloat16*)w_b, plan,      \
-                             slot_row, experts, n_in, n_out, activation, act_param, (__nv_bfloat16*)out_t, out_f, expert_stride)); \
+                             slot_row, experts, n_in, n_out, activation, act_param, (__nv_bfloat16*)out_t, out_f, expert_stride, slot_weight)); \
   } while (0)
     if (tile_rows == MOE_FEW_ROWS) {
       if (mode == MOE_GATED) MOE_ASYNC_LAUNCH(MOE_GATED, MOE_FEW_ROWS, MOE_FEW_STAGES);
@@ -543,7 +560,7 @@ static int launch_moe_products(int mode, const void* x, const void* w_a, const v
 #define MOE_MMA_LAUNCH(MODE)                                                                                             \
   SRB_CUDA_CALL(srb_launch(moe_product_mma_kernel<MODE>, grid, dim3(128), 0, s, (const __nv_bfloat16*)x,                 \
                            (const __nv_bfloat16*)w_a, (const __nv_bfloat16*)w_b, plan, slot_row, experts, n_in, n_out,   \
-                           activation, act_param, (__nv_bfloat16*)out_t, out_f, tile_rows, expert_stride))
+                           activation, act_param, (__nv_bfloat16*)out_t, out_f, tile_rows, expert_stride, slot_weight))
     if (mode == MOE_GATED) MOE_MMA_LAUNCH(MOE_GATED);
     else if (mode == MOE_ACT) MOE_MMA_LAUNCH(MOE_ACT);
     else MOE_MMA_LAUNCH(MOE_DOWN);
@@ -553,7 +570,7 @@ static int launch_moe_products(int mode, const void* x, const void* w_a, const v
   }
 #define MOE_PLAIN_LAUNCH(MODE)                                                                                           \
   SRB_CUDA_CALL(srb_launch(moe_product_kernel<T, MODE>, grid, dim3(256), 0, s, (const T*)x, (const T*)w_a, (const T*)w_b, \
-                           plan, slot_row, experts, n_in, n_out, activation, act_param, (T*)out_t, out_f, tile_rows, expert_stride))
+                           plan, slot_row, experts, n_in, n_out, activation, act_param, (T*)out_t, out_f, tile_rows, expert_stride, slot_weight))
   if (mode == MOE_GATED) MOE_PLAIN_LAUNCH(MOE_GATED);
   else if (mode == MOE_ACT) MOE_PLAIN_LAUNCH(MOE_ACT);
   else MOE_PLAIN_LAUNCH(MOE_DOWN);
@@ -563,33 +580,35 @@ static int launch_moe_products(int mode, const void* x, const void* w_a, const v
 }
 
 // h: [rows, width]; w_gate, w_up: expert e's [inner, width] matrix starts expert_stride elements after expert e - 1's
-// (the two may be halves of one stacked tensor); act: [rows * top, inner]
+// (the two may be halves of one stacked tensor); act: [rows * top, inner]; `slot_weight` (float per slot, or null): a factor
+// on the expert's input
 extern "C" int srb_moe_gated_up(const void* h, const void* w_gate, const void* w_up, long long expert_stride, const int* plan,
                                 const int* slot_row, int rows, int top, int experts, int width, int inner, int activation, float act_param,
-                                void* act, int dtype, void* stream) {
+                                const float* slot_weight, void* act, int dtype, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (width <= 0 || inner <= 0) SRB_FAIL("moe_gated_up: sizes %d, %d must be positive", width, inner);
   if (activation < 0 || activation >= SRB_ACT_COUNT) SRB_FAIL("moe_gated_up: unknown activation %d", activation);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == SRB_DTYPE_F32)
-    return launch_moe_products<float>(MOE_GATED, h, w_gate, w_up, plan, slot_row, rows, top, experts, width, inner, activation, act_param, act, nullptr, (size_t)expert_stride, s);
+    return launch_moe_products<float>(MOE_GATED, h, w_gate, w_up, plan, slot_row, rows, top, experts, width, inner, activation, act_param, act, nullptr, (size_t)expert_stride, slot_weight, s);
   if (dtype == SRB_DTYPE_BF16)
-    return launch_moe_products<__nv_bfloat16>(MOE_GATED, h, w_gate, w_up, plan, slot_row, rows, top, experts, width, inner, activation, act_param, act, nullptr, (size_t)expert_stride, s);
+    return launch_moe_products<__nv_bfloat16>(MOE_GATED, h, w_gate, w_up, plan, slot_row, rows, top, experts, width, inner, activation, act_param, act, nullptr, (size_t)expert_stride, slot_weight, s);
   SRB_FAIL("moe_gated_up: unknown dtype %d", dtype);
 }
 
 // The first product of experts without a gate: act[slot, :] = activation(W_up[e] h[row]); w_up: [experts, inner, width].
 extern "C" int srb_moe_act_up(const void* h, const void* w_up, const int* plan, const int* slot_row, int rows, int top,
-                              int experts, int width, int inner, int activation, float act_param, void* act, int dtype, void* stream) {
+                              int experts, int width, int inner, int activation, float act_param, const float* slot_weight, void* act,
+                              int dtype, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (width <= 0 || inner <= 0) SRB_FAIL("moe_act_up: sizes %d, %d must be positive", width, inner);
   if (activation < 0 || activation >= SRB_ACT_COUNT) SRB_FAIL("moe_act_up: unknown activation %d", activation);
   cudaStream_t s = (cudaStream_t)stream;
   const size_t stride = (size_t)inner * width;
   if (dtype == SRB_DTYPE_F32)
-    return launch_moe_products<float>(MOE_ACT, h, w_up, nullptr, plan, slot_row, rows, top, experts, width, inner, activation, act_param, act, nullptr, stride, s);
+    return launch_moe_products<float>(MOE_ACT, h, w_up, nullptr, plan, slot_row, rows, top, experts, width, inner, activation, act_param, act, nullptr, stride, slot_weight, s);
   if (dtype == SRB_DTYPE_BF16)
-    return launch_moe_products<__nv_bfloat16>(MOE_ACT, h, w_up, nullptr, plan, slot_row, rows, top, experts, width, inner, activation, act_param, act, nullptr, stride, s);
+    return launch_moe_products<__nv_bfloat16>(MOE_ACT, h, w_up, nullptr, plan, slot_row, rows, top, experts, width, inner, activation, act_param, act, nullptr, stride, slot_weight, s);
   SRB_FAIL("moe_act_up: unknown dtype %d", dtype);
 }
 
@@ -600,28 +619,30 @@ extern "C" int srb_moe_down(const void* act, const void* w_down, const int* plan
   if (width <= 0 || inner <= 0) SRB_FAIL("moe_down: sizes %d, %d must be positive", width, inner);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == SRB_DTYPE_F32)
-    return launch_moe_products<float>(MOE_DOWN, act, w_down, nullptr, plan, nullptr, rows, top, experts, inner, width, 0, 0.f, nullptr, y, (size_t)width * inner, s);
+    return launch_moe_products<float>(MOE_DOWN, act, w_down, nullptr, plan, nullptr, rows, top, experts, inner, width, 0, 0.f, nullptr, y, (size_t)width * inner, nullptr, s);
   if (dtype == SRB_DTYPE_BF16)
-    return launch_moe_products<__nv_bfloat16>(MOE_DOWN, act, w_down, nullptr, plan, nullptr, rows, top, experts, inner, width, 0, 0.f, nullptr, y, (size_t)width * inner, s);
+    return launch_moe_products<__nv_bfloat16>(MOE_DOWN, act, w_down, nullptr, plan, nullptr, rows, top, experts, inner, width, 0, 0.f, nullptr, y, (size_t)width * inner, nullptr, s);
   SRB_FAIL("moe_down: unknown dtype %d", dtype);
 }
 
 // `base` (float [rows, width], or null): a term that every row gets beside its experts' (an expert that all rows share);
 // it is the first term of the sum.  `chosen` and `input` (both or neither): a choice whose number is `experts` or more
 // names an expert that returns its input, so its term is weight * input[row] (such choices have no slot in the plan).
+// `base_gate` (float [rows], or null) multiplies the shared term; `weights` null: the results are summed as they are.
 template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ entry_slot,
                                    const float* __restrict__ weights, int top, int width, float* __restrict__ out,
                                    const float* __restrict__ base, const int* __restrict__ chosen, int experts,
-                                   const T* __restrict__ input) {
+                                   const T* __restrict__ input, const float* __restrict__ base_gate) {
   srb_launch_dependents();
   srb_grid_dependency_wait();
   const int row = blockIdx.x;
+  const float gate = base_gate ? base_gate[row] : 1.0f;
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
-    float sum = base ? base[(size_t)row * width + i] : 0.f;
+    float sum = base ? base[(size_t)row * width + i] * gate : 0.f;
     for (int k = 0; k < top; ++k) {
       const int slot = entry_slot[(size_t)row * top + k];
-      if (slot >= 0) sum += weights[(size_t)row * top + k] * y[(size_t)slot * width + i];
+      if (slot >= 0) sum += (weights ? weights[(size_t)row * top + k] : 1.0f) * y[(size_t)slot * width + i];
       else if (input && chosen[(size_t)row * top + k] >= experts)
         sum += weights[(size_t)row * top + k] * srb_to_float(input[(size_t)row * width + i]);
     }
@@ -631,16 +652,17 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
 
 extern "C" int srb_moe_combine_identity(const float* y, const int* entry_slot, const float* weights, int rows, int top,
                                         int width, float* out, const float* base, const int* chosen, int experts,
-                                        const void* input, int dtype, void* stream) {
+                                        const void* input, const float* base_gate, int dtype, void* stream) {
   if (rows <= 0) return SRB_OK;
+  if (!weights && input) SRB_FAIL("moe_combine: experts that return their input need the weights");
   if ((chosen == nullptr) != (input == nullptr)) SRB_FAIL("moe_combine: the choices and the experts' input come together");
   const dim3 block(width >= 1024 ? 256 : 128);
   if (dtype == SRB_DTYPE_F32)
     SRB_CUDA_CALL(srb_launch(moe_combine_kernel<float>, dim3(rows), block, 0, (cudaStream_t)stream, y, entry_slot, weights, top,
-                             width, out, base, chosen, experts, (const float*)input));
+                             width, out, base, chosen, experts, (const float*)input, base_gate));
   else if (dtype == SRB_DTYPE_BF16)
     SRB_CUDA_CALL(srb_launch(moe_combine_kernel<__nv_bfloat16>, dim3(rows), block, 0, (cudaStream_t)stream, y, entry_slot,
-                             weights, top, width, out, base, chosen, experts, (const __nv_bfloat16*)input));
+                             weights, top, width, out, base, chosen, experts, (const __nv_bfloat16*)input, base_gate));
   else
     SRB_FAIL("moe_combine: unknown dtype %d", dtype);
   SRB_LAUNCH_CHECK("moe_combine");
@@ -649,7 +671,7 @@ extern "C" int srb_moe_combine_identity(const float* y, const int* entry_slot, c
 
 extern "C" int srb_moe_combine_onto(const float* y, const int* entry_slot, const float* weights, int rows, int top, int width,
                                     float* out, const float* base, void* stream) {
-  return srb_moe_combine_identity(y, entry_slot, weights, rows, top, width, out, base, nullptr, 0, nullptr, SRB_DTYPE_F32, stream);
+  return srb_moe_combine_identity(y, entry_slot, weights, rows, top, width, out, base, nullptr, 0, nullptr, nullptr, SRB_DTYPE_F32, stream);
 }
 
 extern "C" int srb_moe_combine(const float* y, const int* entry_slot, const float* weights, int rows, int top, int width,

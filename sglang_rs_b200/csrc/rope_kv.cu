@@ -653,6 +653,8 @@ extern "C" int srb_qk_norm_rope_kv_ex(const void* qkv, const float* qkv_parts, i
 // Row of the projection: [n_q * head_dim | n_kv * head_dim | n_kv * value_dim | gate_cols].
 // With `per_head` every q and k head is instead divided by its own root mean square and multiplied by a weight
 // [head_dim] that all heads of its kind share.
+// With `temp_every` > 0 q is multiplied by a factor that grows with the row's position p: 1 + temp_coef ln(floor((p + 1) /
+// temp_every) + 1).
 // One block per row; sums of squares, norms, angles and the rotation are 32-bit; a norm whose weight is null is left out.
 // Sum of two values over a block of up to 1024 threads at once; every thread receives both.  Warp partials are added in
 // warp order, so the results do not depend on timing.
@@ -677,7 +679,7 @@ proj_norm_rope_kv_kernel(const T* __restrict__ qkv, const float* __restrict__ qk
                          const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
                          const float* __restrict__ inv_freq, int rotary_dim, int interleaved, float magnitude, int n_q,
                          int n_kv, int head_dim, int value_dim, int gate_cols, int page_size, int num_pages,
-                         int* error_word, int per_head) {
+                         int* error_word, int per_head, float temp_coef, int temp_every) {
   extern __shared__ __align__(16) float staged[];       // the row (q, k, v, gate logits), rotary_dim cosines and sines, 66 of scratch
   const int q_width = n_q * head_dim, k_width = n_kv * head_dim, v_width = n_kv * value_dim;
   const int row_width = q_width + k_width + v_width + gate_cols;
@@ -687,6 +689,7 @@ proj_norm_rope_kv_kernel(const T* __restrict__ qkv, const float* __restrict__ qk
   srb_launch_dependents();
   const int row = blockIdx.x;
   const int half = rotary_dim >> 1;
+  const float q_factor = temp_every > 0 ? 1.0f + temp_coef * logf((float)((positions[row] + 1) / temp_every + 1)) : 1.0f;
   if (inv_freq) {                                        // needs the step's index arrays only: ahead of the wait
     const float pos = (float)positions[row];
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
@@ -738,9 +741,9 @@ proj_norm_rope_kv_kernel(const T* __restrict__ qkv, const float* __restrict__ qk
         }
     }
   };
-  auto store_eight = [&](T* to, const float* from) {       // `from`: shared memory, on a 16-byte border
+  auto store_eight = [&](T* to, const float* from, float factor) {       // `from`: shared memory, on a 16-byte border
     const float4 lo = *reinterpret_cast<const float4*>(from), hi = *reinterpret_cast<const float4*>(from + 4);
-    const float x[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+    const float x[8] = {lo.x * factor, lo.y * factor, lo.z * factor, lo.w * factor, hi.x * factor, hi.y * factor, hi.z * factor, hi.w * factor};
     if (sizeof(T) == 2) {
       uint4 raw;
       __nv_bfloat162* pair = reinterpret_cast<__nv_bfloat162*>(&raw);
@@ -819,18 +822,18 @@ proj_norm_rope_kv_kernel(const T* __restrict__ qkv, const float* __restrict__ qk
     const int total = q_width + (slot < 0 ? 0 : k_width + v_width);
     for (int i = threadIdx.x * 8; i < total; i += blockDim.x * 8) {
       if (i < q_width) {
-        store_eight(q_out + (size_t)row * q_width + i, staged + i);
+        store_eight(q_out + (size_t)row * q_width + i, staged + i, q_factor);
       } else if (i < q_width + k_width) {
         const int head = (i - q_width) / head_dim, e = (i - q_width) - head * head_dim;
-        store_eight(k_pool + ((page * n_kv + head) * page_size + inside) * head_dim + e, staged + i);
+        store_eight(k_pool + ((page * n_kv + head) * page_size + inside) * head_dim + e, staged + i, 1.0f);
       } else {
         const int c = i - q_width - k_width, head = c / value_dim, e = c - head * value_dim;
-        store_eight(v_pool + ((page * n_kv + head) * page_size + inside) * value_dim + e, staged + i);
+        store_eight(v_pool + ((page * n_kv + head) * page_size + inside) * value_dim + e, staged + i, 1.0f);
       }
     }
     return;
   }
-  for (int i = threadIdx.x; i < q_width; i += blockDim.x) q_out[(size_t)row * q_width + i] = srb_from_float<T>(staged[i]);
+  for (int i = threadIdx.x; i < q_width; i += blockDim.x) q_out[(size_t)row * q_width + i] = srb_from_float<T>(staged[i] * q_factor);
   if (slot < 0) return;
   for (int i = threadIdx.x; i < k_width; i += blockDim.x) {
     const int head = i / head_dim, e = i - head * head_dim;
@@ -847,7 +850,8 @@ extern "C" int srb_proj_norm_rope_kv(const void* qkv, const float* qkv_parts, in
                                      const int* positions, const int* slots, const float* q_weight, const float* k_weight,
                                      float eps, const float* inv_freq, int rotary_dim, int interleaved, float magnitude,
                                      int rows, int n_q, int n_kv, int head_dim, int value_dim, int gate_cols, int page_size,
-                                     int num_pages, int* error_word, int dtype, int per_head, void* stream) {
+                                     int num_pages, int* error_word, int dtype, int per_head, float temp_coef,
+                                     int temp_every, void* stream) {
   if (rows <= 0) return SRB_OK;
   if (n_q <= 0 || n_kv <= 0 || head_dim <= 0 || value_dim <= 0 || page_size <= 0 || gate_cols < 0)
     SRB_FAIL("proj_norm_rope_kv: head counts, widths and page size must be positive");
@@ -859,6 +863,7 @@ extern "C" int srb_proj_norm_rope_kv(const void* qkv, const float* qkv_parts, in
   if ((long long)qkv_stride < (long long)(n_q + n_kv) * head_dim + (long long)n_kv * value_dim + gate_cols)
     SRB_FAIL("proj_norm_rope_kv: rows of the projection are narrower than their parts together");
   if (gate_cols > 0 && !gate_out) SRB_FAIL("proj_norm_rope_kv: gate logits without a place for the gates");
+  if (temp_every < 0) SRB_FAIL("proj_norm_rope_kv: the positions per step of the temperature must be positive, or 0 for none");
   if (!(eps >= 0.f)) SRB_FAIL("proj_norm_rope_kv: eps must be finite and non-negative");
   const size_t smem = ((size_t)(n_q + n_kv) * head_dim + (size_t)n_kv * value_dim + gate_cols + 4 + rotary_dim + 66) * sizeof(float);
   if (smem > 227 * 1024) SRB_FAIL("proj_norm_rope_kv: %zu bytes of shared memory exceed 232448", smem);
@@ -876,7 +881,8 @@ extern "C" int srb_proj_norm_rope_kv(const void* qkv, const float* qkv_parts, in
     SRB_CUDA_CALL(srb_launch(proj_norm_rope_kv_kernel<T, EIGHT>, dim3(rows), dim3(threads), smem, s, (const T*)qkv, qkv_parts, \
                              num_parts, (size_t)part_stride, qkv_stride, (T*)q_out, (T*)k_pool, (T*)v_pool, gate_out,          \
                              positions, slots, q_weight, k_weight, eps, inv_freq, rotary_dim, interleaved, magnitude, n_q,     \
-                             n_kv, head_dim, value_dim, gate_cols, page_size, num_pages, error_word, per_head));               \
+                             n_kv, head_dim, value_dim, gate_cols, page_size, num_pages, error_word, per_head, temp_coef,      \
+                             temp_every));                                                                                     \
   } while (0)
   if (dtype == SRB_DTYPE_F32) {
     if (eight) SRB_PROJ_LAUNCH(float, true); else SRB_PROJ_LAUNCH(float, false);

@@ -21,7 +21,7 @@ import numpy as np
 import torch
 
 from .. import ops
-from .runner import AttentionLaunch, PagedBatch, StepContext, StepEntry, StepPlanner
+from .runner import AttentionLaunch, PagedBatch, StepContext, StepEntry, StepPlanner, visible_pieces
 
 
 def bucket_of(value: int, smallest: int = 1) -> int:
@@ -84,9 +84,8 @@ class DecodeGraphs:
         splits = []
         size = StepPlanner.SPLIT_SIZE
         for key in groups:
-            window = self.cache.windows[key]
-            begin = np.maximum(0, positions + 1 - window) if window else np.zeros_like(positions)
-            splits.append(bucket_of(int((positions // size - begin // size + 1).max())))
+            pieces, _ = visible_pieces(positions, self.cache.windows[key], self.cache.keep_first[key], size)
+            splits.append(bucket_of(int(pieces.max())))
         key = (bucket, stride, tuple(splits))
         step = self.captured.get(key)
         if step is None:

@@ -88,6 +88,15 @@ class StepContext:
     host_state_slots: Sequence[int] = ()
 
 
+def visible_pieces(positions: np.ndarray, window: Optional[int], keep_first: int, size: int):
+    """For rows at ``positions``: how many pieces of ``size`` keys, cut at absolute multiples of ``size``, hold a key that
+    the row sees, and a bound on the keys it sees.  With a window the pieces are those of the kept first tokens that lie
+    wholly ahead of the window's first piece, then the window's."""
+    begin = np.maximum(0, positions + 1 - window) if window else np.zeros_like(positions)
+    kept = np.minimum(-(-keep_first // size), begin // size) if window else 0
+    return positions // size - begin // size + 1 + kept, positions + 1 - begin + np.minimum(keep_first, begin)
+
+
 class StepPlanner:
     """Turns a step's entries into the flat device arrays and the per-group plans that the
     parts read.  It needs the cache manager and the scratch widths of the mixers, not the
@@ -209,15 +218,12 @@ class StepPlanner:
 
     def _plan(self, key, table_d, slots_d, positions: np.ndarray, split_rows: int, rows: int,
               tiles_d: Optional[torch.Tensor] = None, wide_tiles_d: Optional[torch.Tensor] = None) -> PagedBatch:
-        window = self.cache.windows[key]
         launches: List[AttentionLaunch] = []
         scratch_acc = scratch_ml = None
         if split_rows > 0:
             pos = positions[:split_rows]
-            begin = np.maximum(0, pos + 1 - window) if window else np.zeros_like(pos)
             split_size = self.SPLIT_SIZE
-            per_row = pos // split_size - begin // split_size + 1
-            visible_per_row = pos + 1 - begin
+            per_row, visible_per_row = visible_pieces(pos, self.cache.windows[key], self.cache.keep_first[key], split_size)
             # The keys are always cut every SPLIT_SIZE positions, so a row's arithmetic is a function of its
             # own position.  When the partial results of all rows do not fit the scratch memory, the rows go
             # in several launches, one after another over the same scratch, never in longer pieces.

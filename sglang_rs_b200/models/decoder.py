@@ -7,7 +7,8 @@ a layer twice (two calls, two caches, one set of weights), and a call may read t
 of an earlier call instead of keeping one (it then writes nothing).  A call may also name a
 part of ``pass_entries`` that runs right before it: the head of a pass over a stretch of
 layers that the program walks several times (``parts/loop.py``); it is handed the stream,
-the embedding output and the number of the pass, and returns the new stream.
+the embedding output and the number of the pass, and returns the new stream, or the stream and what is pending to be
+added to it.
 
 An embedding may keep state per request too (the token before, for a table indexed by pairs of tokens): its need
 is the entry after the calls' in ``cache_needs()``, and ``forward`` hands it the cache at that index.
@@ -96,7 +97,7 @@ class DecoderModel(Part):
             residual = self.embedding.forward(ctx, ctx.token_ids)
         delta = None
         origin = None
-        if any(call.entry is not None for call in self.program):
+        if any(call.entry is not None and getattr(self.pass_entries[call.entry], "reads_origin", True) for call in self.program):
             # the embedding output as the pass entries read it; layers ahead of the first pass change the stream in
             # place, and so does an entry that adds onto the stream it is given
             first_makes_new = self.program[0].entry is not None and not getattr(
@@ -107,7 +108,8 @@ class DecoderModel(Part):
             if call.cache_from is not None and cache is not None:
                 cache = cache.read_only()
             if call.entry is not None:
-                residual, delta = self.pass_entries[call.entry].forward(ctx, residual, delta, origin, call.pass_index), None
+                opened = self.pass_entries[call.entry].forward(ctx, residual, delta, origin, call.pass_index)
+                residual, delta = opened if isinstance(opened, tuple) else (opened, None)
             residual, delta = self.layers[call.layer].forward(ctx, cache, residual, delta)
         if logit_rows is None or logit_rows.numel() == 0:
             return None

@@ -9,6 +9,7 @@ from __future__ import annotations
 
 import ctypes
 import os
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -236,7 +237,8 @@ def norm_add_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], inner, 
                   row_index: Optional[torch.Tensor] = None, write_residual: bool = True,
                   extra: Optional[torch.Tensor] = None, addend: Optional[torch.Tensor] = None) -> None:
     """x = residual + inner(delta) (+ addend); residual = x if asked; out = outer(x), all sums and means in 32-bit.
-    ``addend`` (float32, shaped like the residual) is a second term of the sum, added after the pending one.
+    ``addend`` (float32, shaped like the residual, or one row [width] for all rows) is a second term of the sum, added after
+    the pending one.
     ``delta`` may also be float32 [parts, rows, width]: partial sums of a product cut along K, added in part order
     before the inner norm.
 
@@ -297,7 +299,7 @@ def norm_add_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], inner, 
             raise KernelError("norm_add_norm: extra and residual differ in shape")
     if addend is not None:
         _need(addend, "addend", torch.float32)
-        if addend.shape != residual.shape:
+        if addend.shape != residual.shape and addend.shape != (width,):
             raise KernelError("norm_add_norm: addend and residual differ in shape")
     if row_index is not None:
         _need(row_index, "row_index", torch.int32)
@@ -306,7 +308,8 @@ def norm_add_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], inner, 
         _ptr(residual), _ptr(whole), _ptr(as_float), inner_kind, _ptr(inner_w), _ptr(inner_b), ctypes.c_float(inner_eps),
         inner_groups, ctypes.c_float(inner_scale), outer_kind, _ptr(outer_w), _ptr(outer_b), ctypes.c_float(outer_eps),
         outer_groups, ctypes.c_float(outer_scale), _ptr(out), ctypes.c_longlong(pitch),
-        _ptr(extra), _ptr(row_index), rows, width, int(write_residual), dtype_code(dtype), _ptr(addend), num_parts,
+        _ptr(extra), _ptr(row_index), rows, width, int(write_residual), dtype_code(dtype), _ptr(addend),
+        ctypes.c_longlong(width if addend is not None and addend.dim() == 2 else 0), num_parts,
         ctypes.c_longlong(part_stride), _stream()))
 
 
@@ -420,7 +423,8 @@ def proj_norm_rope_kv(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[t
                       positions: torch.Tensor, slots: Optional[torch.Tensor], q_weight: Optional[torch.Tensor],
                       k_weight: Optional[torch.Tensor], eps: float, inv_freq: Optional[torch.Tensor], rotary_dim: int,
                       interleaved: bool, n_q: int, n_kv: int, head_dim: int, value_dim: int, error_word: torch.Tensor, *,
-                      magnitude: float = 1.0, gate_out: Optional[torch.Tensor] = None, per_head: bool = False) -> None:
+                      magnitude: float = 1.0, gate_out: Optional[torch.Tensor] = None, per_head: bool = False,
+                      temperature: Optional[tuple] = None) -> None:
     """The step between the q/k/v product and attention for a mixer that norms q and k over the WHOLE projection (all
     heads of a row together, a weight per entry: ``q_weight`` [n_q * head_dim], ``k_weight`` [n_kv * head_dim]; None: no
     norm), then rotates the leading ``rotary_dim`` entries of every head, writes q to ``q_out`` [rows, n_q, head_dim], k
@@ -428,8 +432,10 @@ def proj_norm_rope_kv(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[t
     page_size, value_dim].  Rows of ``qkv`` are [q | k | v | gate logits]; ``gate_out`` (float32 [rows, gates]) receives
     the sigmoids of the logits behind the values.  ``qkv`` is of ``q_out``'s dtype or float32 [parts, rows, width]
     partial sums; its rows may be columns of wider ones.  ``slots`` None: nothing is stored.  ``per_head``: every q and k
-    head is normed by itself with a weight that its kind's heads share (``q_weight``, ``k_weight`` [head_dim])."""
+    head is normed by itself with a weight that its kind's heads share (``q_weight``, ``k_weight`` [head_dim]).  ``temperature``
+    (coef, every): q of a row at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
     _need(q_out, "q_out"); _need(positions, "positions", torch.int32)
+    temp_coef, temp_every = temperature if temperature is not None else (0.0, 0)
     whole = parts = None
     num_parts = part_stride = 0
     if qkv.dim() == 3:
@@ -471,7 +477,7 @@ def proj_norm_rope_kv(qkv: torch.Tensor, q_out: torch.Tensor, k_pool: Optional[t
         _ptr(k_pool) if slots is not None else None, _ptr(v_pool) if slots is not None else None, _ptr(gate_out),
         _ptr(positions), _ptr(slots), _ptr(q_weight), _ptr(k_weight), ctypes.c_float(eps), _ptr(inv_freq), rotary_dim,
         int(interleaved), ctypes.c_float(magnitude), rows, n_q, n_kv, head_dim, value_dim, gate_cols, page_size, num_pages,
-        _ptr(error_word), dtype_code(q_out.dtype), int(per_head), _stream()))
+        _ptr(error_word), dtype_code(q_out.dtype), int(per_head), ctypes.c_float(temp_coef), int(temp_every), _stream()))
 
 
 @traced("rope_kv")
@@ -493,13 +499,40 @@ def attention_scratch_sizes(rows: int, n_q: int, head_dim: int, max_splits: int)
     return rows * n_q * max_splits * head_dim, rows * n_q * max_splits * 2
 
 
+@dataclass(frozen=True)
+class MapJoin:
+    """How the two maps of a head become its result: o = a_1 - ``subtract`` * a_2, divided by sqrt(mean(o^2) + ``eps``) over the
+    head's values, times ``scale``; all in 32-bit."""
+    subtract: float
+    scale: float
+    eps: float
+
+
+class _AttnTerms(ctypes.Structure):
+    """AttnTerms of csrc/attention_kernels.cuh."""
+    _fields_ = [("keep_first", ctypes.c_int), ("softcap", ctypes.c_float), ("maps", ctypes.c_int), ("map_lambda", ctypes.c_float),
+                ("map_scale", ctypes.c_float), ("map_eps", ctypes.c_float), ("float_out", ctypes.c_int)]
+
+
+def _attention_terms(keep_first: int, softcap: Optional[float], join: Optional[MapJoin], float_out: bool = False):
+    """A pointer to the terms, or None if the call has none of them."""
+    if not keep_first and not softcap and join is None and not float_out:
+        return None
+    if join is None:
+        terms = _AttnTerms(int(keep_first), float(softcap or 0.0), 1, 0.0, 1.0, 0.0, int(float_out))
+    else:
+        terms = _AttnTerms(int(keep_first), float(softcap or 0.0), 2, join.subtract, join.scale, join.eps, int(float_out))
+    return ctypes.byref(terms)
+
+
 @traced("attention_generic")
 def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
                     positions: torch.Tensor, row_request: torch.Tensor, block_table: torch.Tensor, *,
                     scale: float, window: int, split_size: int, max_splits: int,
                     scratch_acc: Optional[torch.Tensor], scratch_ml: Optional[torch.Tensor],
                     error_word: torch.Tensor, sinks: Optional[torch.Tensor] = None, chunk: int = 0,
-                    gates: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
+                    gates: Optional[torch.Tensor] = None, out_scale: float = 1.0, keep_first: int = 0,
+                    softcap: Optional[float] = None, join: Optional[MapJoin] = None) -> None:
     """out[r, h, :] = softmax over the keys row r may see of (q . k) * scale, times v.
 
     A row at position p sees the keys max(0, p - window + 1) .. p (``window`` 0: from 0) and, with ``chunk`` > 0,
@@ -511,6 +544,11 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     [rows, n_q]): a factor on the result of every (row, query head).  ``out_scale``: a factor on every result.  The rows of
     ``out`` may lie further apart than they are long (columns of a wider matrix).
 
+    ``keep_first``: beside its window a row sees the sequence's first ``keep_first`` keys.  ``softcap``: a score s becomes
+    softcap * tanh(s / softcap).  ``join``: every head has two maps over the same values; the rows of q and of the key pool
+    are [map 1 | map 2], two halves of ``head_dim``, each map is an attention of its own and their results are joined as
+    :class:`MapJoin` says (scratch then holds two results per head).
+
     q, out: [rows, n_q, head_dim]; pools [pages, n_kv, page_size, head_dim]; block_table
     [requests, stride].  ``split_size`` 0 walks all keys in one block per (row, kv head);
     otherwise partials go through the scratch tensors and are merged in split order.
@@ -519,7 +557,8 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     pitch = _head_rows(out, "out", q.dtype)
     _need(positions, "positions", torch.int32); _need(row_request, "row_request", torch.int32)
     _need(block_table, "block_table", torch.int32)
-    rows, n_q, head_dim = q.shape
+    rows, heads, head_dim = q.shape
+    n_q = heads * (2 if join is not None else 1)               # the kernels count maps
     num_pages, n_kv, page_size, pool_dim = k_pool.shape
     value_dim = out.shape[2]
     if pool_dim != head_dim or out.shape[:2] != q.shape[:2] or (v_pool is None and value_dim > head_dim):
@@ -542,12 +581,19 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
             raise KernelError("paged_attention: scratch tensors are too small for this split run")
         _need(scratch_acc, "scratch_acc", torch.float32); _need(scratch_ml, "scratch_ml", torch.float32)
     lib = load_library("attention")
-    _check(lib, lib.srb_paged_attention_gated(
-        _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(scratch_acc), _ptr(scratch_ml), _ptr(positions),
+    result = out
+    if join is not None:
+        result, pitch = torch.empty((rows, n_q, value_dim), dtype=torch.float32, device=q.device), 0
+    _check(lib, lib.srb_paged_attention_terms(
+        _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(result), _ptr(scratch_acc), _ptr(scratch_ml), _ptr(positions),
         _ptr(row_request), _ptr(block_table), block_table.stride(0), rows, n_q, n_kv, head_dim, page_size,
         num_pages, int(window), int(chunk), int(split_size), int(max_splits), ctypes.c_float(scale), _ptr(error_word),
         dtype_code(q.dtype), _ptr(sinks), value_dim, _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale),
-        _stream()), launches=2 if split_size else 1)
+        _attention_terms(keep_first, softcap, join, join is not None), _stream()), launches=2 if split_size else 1)
+    if join is not None:
+        _check(lib, lib.srb_map_combine(_ptr(result), _ptr(out), rows, heads, value_dim, ctypes.c_longlong(out.stride(0)),
+                                        ctypes.c_float(join.subtract), ctypes.c_float(join.scale), ctypes.c_float(join.eps),
+                                        dtype_code(out.dtype), _stream()))
 
 
 
@@ -609,10 +655,10 @@ def latent_attention(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, pos
 DECODE_MAX_SPLITS = 64
 
 
-def decode_attention_takes(dtype: torch.dtype, n_q: int, n_kv: int, head_dim: int) -> bool:
+def decode_attention_takes(dtype: torch.dtype, n_q: int, n_kv: int, head_dim: int, maps: int = 1) -> bool:
     """True if the tensor-core kernel for decoded tokens takes these sizes (the rule of
     srb_decode_attention_supports, asked here so that other models never compile it)."""
-    return dtype == torch.bfloat16 and head_dim in (64, 128) and n_kv > 0 and n_q % n_kv == 0 and n_q // n_kv <= 16
+    return dtype == torch.bfloat16 and head_dim in (64, 128) and n_kv > 0 and n_q % n_kv == 0 and n_q // n_kv * maps <= 16
 
 
 
@@ -641,9 +687,10 @@ def decode_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
                      scale: float, window: int, scratch_acc: torch.Tensor, scratch_ml: torch.Tensor,
                      counters: torch.Tensor, error_word: torch.Tensor, max_keys: Optional[int] = None,
                      chunk: int = 0, sinks: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None,
-                     out_scale: float = 1.0) -> None:
+                     out_scale: float = 1.0, keep_first: int = 0, softcap: Optional[float] = None,
+                     join: Optional[MapJoin] = None) -> None:
     """Attention of decoded tokens (one row each), bfloat16, head_dim 64 or 128; ``window``, ``chunk``, ``sinks``,
-    ``gates``, ``out_scale`` and the rows of ``out`` as in :func:`paged_attention` (the sink joins where a row's splits are merged, once).
+    ``gates``, ``out_scale``, ``keep_first``, ``softcap``, ``join`` and the rows of ``out`` as in :func:`paged_attention` (the sink joins where a row's splits are merged, once).
 
     The keys of a (row, kv head) are shared by ``decode_splits(rows, n_kv, max_keys)`` blocks
     (``max_keys``: the most keys any row sees, if known); the block that finishes last merges them.  ``counters``: int32, zero, at least rows * n_kv entries; they
@@ -656,6 +703,7 @@ def decode_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
     _need(scratch_acc, "scratch_acc", torch.float32); _need(scratch_ml, "scratch_ml", torch.float32)
     _need(counters, "counters", torch.int32)
     rows, n_q, head_dim = q.shape
+    n_q *= 2 if join is not None else 1                        # the kernel counts maps
     num_pages, n_kv, page_size, pool_dim = k_pool.shape
     if pool_dim != head_dim or v_pool.shape != k_pool.shape or out.shape != q.shape:
         raise KernelError("decode_attention: shapes of q, out and the pools do not agree")
@@ -676,11 +724,11 @@ def decode_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
         if gates.shape != (rows_, heads_):
             raise KernelError("decode_attention: one gate per row and query head is needed")
     lib = load_library("attention_decode")
-    _check(lib, lib.srb_decode_attention_gated(
+    _check(lib, lib.srb_decode_attention_terms(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(scratch_acc), _ptr(scratch_ml), _ptr(counters),
         _ptr(positions), _ptr(row_request), _ptr(block_table), block_table.stride(0), rows, n_q, n_kv, head_dim,
         page_size, num_pages, int(window), int(chunk), splits, ctypes.c_float(scale), _ptr(error_word), _ptr(sinks),
-        _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale), _stream()))
+        _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale), _attention_terms(keep_first, softcap, join), _stream()))
 
 
 def tiled_attention_takes(dtype: torch.dtype, n_q: int, n_kv: int, head_dim: int) -> bool:
@@ -694,8 +742,9 @@ def tiled_attention_takes(dtype: torch.dtype, n_q: int, n_kv: int, head_dim: int
 def tiled_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
                     tiles: torch.Tensor, block_table: torch.Tensor, *, scale: float, window: int,
                     error_word: torch.Tensor, chunk: int = 0, sinks: Optional[torch.Tensor] = None,
-                    gates: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
-    """Attention of prompt portions, bfloat16 (``sinks``, ``gates``, ``out_scale``, rows of ``out``: as in :func:`paged_attention`).  ``tiles`` is int32 [n, 4]: first row of the
+                    gates: Optional[torch.Tensor] = None, out_scale: float = 1.0, keep_first: int = 0,
+                    softcap: Optional[float] = None) -> None:
+    """Attention of prompt portions, bfloat16 (``sinks``, ``gates``, ``out_scale``, ``keep_first``, ``softcap``, rows of ``out``: as in :func:`paged_attention`).  ``tiles`` is int32 [n, 4]: first row of the
     step, rows (at most 64, consecutive rows of one request), request index, first position.
     Rows outside the tiles are left untouched."""
     _need(q, "q", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16)
@@ -716,10 +765,11 @@ def tiled_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
         if gates.shape != (rows_, heads_):
             raise KernelError("tiled_attention: one gate per row and query head is needed")
     lib = load_library("attention_prefill")
-    _check(lib, lib.srb_prefill_attention_gated(
+    _check(lib, lib.srb_prefill_attention_terms(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(tiles), tiles.shape[0], _ptr(block_table),
         block_table.stride(0), n_q, n_kv, head_dim, page_size, num_pages, int(window), int(chunk), ctypes.c_float(scale),
-        _ptr(error_word), _ptr(sinks), _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale), _stream()))
+        _ptr(error_word), _ptr(sinks), _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale),
+        _attention_terms(keep_first, softcap, None), _stream()))
 
 
 TC_TILE_ROWS = 128
@@ -736,9 +786,10 @@ def tiled_attention_tc_takes(dtype: torch.dtype, n_q: int, n_kv: int, head_dim: 
 def tiled_attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor,
                        tiles: torch.Tensor, block_table: torch.Tensor, *, scale: float, window: int,
                        error_word: torch.Tensor, chunk: int = 0, sinks: Optional[torch.Tensor] = None,
-                       gates: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
+                       gates: Optional[torch.Tensor] = None, out_scale: float = 1.0, keep_first: int = 0,
+                       softcap: Optional[float] = None, join: Optional[MapJoin] = None) -> None:
     """Attention of prompt portions on tcgen05 tensor cores (S, P and O in tensor memory, operands
-    by TMA; ``sinks``, ``gates``, ``out_scale``, rows of ``out`` (16-byte borders): as in :func:`paged_attention`).  ``tiles`` as for :func:`tiled_attention`, with at most 128 rows per tile."""
+    by TMA; ``sinks``, ``gates``, ``out_scale``, ``keep_first``, ``softcap``, ``join``, rows of ``out`` (16-byte borders): as in :func:`paged_attention`).  ``tiles`` as for :func:`tiled_attention`, with at most 128 rows per tile."""
     _need(q, "q", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16)
     pitch = _head_rows(out, "out", q.dtype)
     _need(v_pool, "v_pool", torch.bfloat16); _need(tiles, "tiles", torch.int32)
@@ -757,10 +808,11 @@ def tiled_attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tens
         if gates.shape != (rows_, heads_):
             raise KernelError("tiled_attention_tc: one gate per row and query head is needed")
     lib = load_library("attention_prefill_tc")
-    _check(lib, lib.srb_prefill_attention_tc_gated(
+    _check(lib, lib.srb_prefill_attention_tc_terms(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(tiles), tiles.shape[0], rows, _ptr(block_table),
-        block_table.stride(0), n_q, n_kv, head_dim, page_size, num_pages, int(window), int(chunk), ctypes.c_float(scale),
-        _ptr(error_word), _ptr(sinks), _ptr(gates), ctypes.c_longlong(pitch), ctypes.c_float(out_scale), _stream()))
+        block_table.stride(0), n_q * (2 if join is not None else 1), n_kv, head_dim, page_size, num_pages, int(window),
+        int(chunk), ctypes.c_float(scale), _ptr(error_word), _ptr(sinks), _ptr(gates), ctypes.c_longlong(pitch),
+        ctypes.c_float(out_scale), _attention_terms(keep_first, softcap, join), _stream()))
 
 
 # --------------------------------------------------------------------------- latents and per-head products
@@ -873,12 +925,17 @@ def routed_experts(h: torch.Tensor, router: torch.Tensor, w_gate_up: torch.Tenso
                    activation: str, renormalize: bool, error_word: torch.Tensor, *, gated: bool = True,
                    router_bias: Optional[torch.Tensor] = None, base: Optional[torch.Tensor] = None,
                    scoring: str = "softmax", choice_bias: Optional[torch.Tensor] = None, weight_scale: float = 1.0,
-                   norm_eps: float = 0.0, activation_param: float = 0.0, identity: int = 0) -> torch.Tensor:
+                   norm_eps: float = 0.0, activation_param: float = 0.0, identity: int = 0, weigh_inputs: bool = False,
+                   base_gated: bool = False) -> torch.Tensor:
     """sum over the ``top`` experts with the largest router scores of score * expert(h), float32 [rows, width].
 
     ``identity``: the router has this many outputs more than there are expert matrices; they stand for experts that return
     their input, so a row that chooses one gets weight * h[row] as that expert's term (the scores and the choice run over
     all outputs alike; ``router``, ``router_bias`` and ``choice_bias`` have experts + identity rows).
+
+    ``weigh_inputs``: a chosen expert's weight multiplies its input instead of its result (the sum is then of
+    expert(weight * h)).  ``base_gated``: ``router`` has one row more, the last; the sigmoid of its logit, one number per row
+    in 32-bit, multiplies ``base``.
 
     ``gated`` False: an expert is W_down act(W_up h) and ``w_gate_up`` holds the up matrices alone
     [experts, inner, width].  ``router_bias`` (float32 [experts]) is added to the router's logits before the choice.
@@ -903,7 +960,11 @@ def routed_experts(h: torch.Tensor, router: torch.Tensor, w_gate_up: torch.Tenso
     routes = experts + int(identity)
     if identity < 0 or routes > 1024:
         raise KernelError(f"routed_experts: {routes} router outputs are outside what the router kernels take (1024)")
-    if (router.shape != (routes, width) or w_gate_up.shape != (experts, (2 if gated else 1) * inner, width)
+    if identity and weigh_inputs:
+        raise KernelError("routed_experts: weights on inputs are not built for experts that return their input")
+    if base_gated and (base is None or router_bias is not None):
+        raise KernelError("routed_experts: the gate of the shared term needs that term and a router without bias")
+    if (router.shape != (routes + int(base_gated), width) or w_gate_up.shape != (experts, (2 if gated else 1) * inner, width)
             or w_down.shape != (experts, width, inner)):
         raise KernelError("routed_experts: shapes of the router and the experts do not agree")
     if router_bias is not None:
@@ -932,6 +993,8 @@ def routed_experts(h: torch.Tensor, router: torch.Tensor, w_gate_up: torch.Tenso
     slot_row = torch.empty(entries, dtype=torch.int32, device=device)
     entry_slot = torch.empty(entries, dtype=torch.int32, device=device)
     act = torch.empty((entries, inner), dtype=h.dtype, device=device)
+    slot_weight = torch.empty(entries, dtype=torch.float32, device=device) if weigh_inputs else None
+    base_gate = torch.empty(rows, dtype=torch.float32, device=device) if base_gated else None
     y = torch.empty((entries, width), dtype=torch.float32, device=device)
     out = torch.empty((rows, width), dtype=torch.float32, device=device)
     code, stream = dtype_code(h.dtype), _stream()
@@ -939,12 +1002,12 @@ def routed_experts(h: torch.Tensor, router: torch.Tensor, w_gate_up: torch.Tenso
         # many rows: the logits are a product like any other (32-bit accumulation, 32-bit result), the choice a kernel of its own
         logits = linear(h, router, router_bias, out_dtype=torch.float32, error_word=error_word)
         _check(lib, lib.srb_moe_select_ex(_ptr(logits), ctypes.c_longlong(logits.stride(0)), rows, routes, top, *rule,
-                                          _ptr(chosen), _ptr(weights), stream))
+                                          _ptr(chosen), _ptr(weights), _ptr(base_gate), stream))
     else:
         _check(lib, lib.srb_moe_route_ex(_ptr(h), _ptr(router), rows, width, routes, top, *rule, _ptr(chosen),
-                                         _ptr(weights), code, stream))
+                                         _ptr(weights), _ptr(base_gate), code, stream))
     _check(lib, lib.srb_moe_plan_of(_ptr(chosen), rows, top, experts, tile_slots, _ptr(plan), _ptr(slot_row),
-                                    _ptr(entry_slot), _ptr(error_word), stream))
+                                    _ptr(entry_slot), _ptr(weights), _ptr(slot_weight), _ptr(error_word), stream))
     if grouped:
         product = load_library("gemm_bf16")
         max_tiles = lib.srb_moe_max_tiles_of(rows, top, experts, tile_slots)
@@ -955,26 +1018,26 @@ def routed_experts(h: torch.Tensor, router: torch.Tensor, w_gate_up: torch.Tenso
         _check(product, product.srb_gemm_bf16_grouped(
             _ptr(gathered), _ptr(w_gate_up), _ptr(act), _ptr(plan), max_tiles, tile_slots, entries, experts,
             (2 if gated else 1) * inner, inner, width, inner, inner if gated else 0, GEMM_MODES["gated" if gated else "act"],
-            act_code, act_param, _ptr(error_word), stream))
+            act_code, act_param, _ptr(slot_weight), _ptr(error_word), stream))
         _check(product, product.srb_gemm_bf16_grouped(
             _ptr(act), _ptr(w_down), _ptr(y), _ptr(plan), max_tiles, tile_slots, entries, experts, width, width, inner, width, 0,
-            GEMM_MODES["f32"], 0, ctypes.c_float(0.0), _ptr(error_word), stream))
+            GEMM_MODES["f32"], 0, ctypes.c_float(0.0), None, _ptr(error_word), stream))
     else:
         element = h.element_size()
         if gated:
             w_up = ctypes.c_void_p(w_gate_up.data_ptr() + inner * width * element)
             _check(lib, lib.srb_moe_gated_up(_ptr(h), _ptr(w_gate_up), w_up, ctypes.c_longlong(2 * inner * width), _ptr(plan),
                                              _ptr(slot_row), rows, top, experts, width, inner, act_code, act_param,
-                                             _ptr(act), code, stream))
+                                             _ptr(slot_weight), _ptr(act), code, stream))
         else:
             _check(lib, lib.srb_moe_act_up(_ptr(h), _ptr(w_gate_up), _ptr(plan), _ptr(slot_row), rows, top, experts, width,
-                                           inner, act_code, act_param, _ptr(act), code, stream))
+                                           inner, act_code, act_param, _ptr(slot_weight), _ptr(act), code, stream))
         _check(lib, lib.srb_moe_down(_ptr(act), _ptr(w_down), _ptr(plan), rows, top, experts, width, inner, _ptr(y), code,
                                      stream))
     # choices of `experts` and above have no slot in the plan: they are the experts that return their input
-    _check(lib, lib.srb_moe_combine_identity(_ptr(y), _ptr(entry_slot), _ptr(weights), rows, top, width, _ptr(out), _ptr(base),
-                                             _ptr(chosen) if identity else None, experts, _ptr(h) if identity else None, code,
-                                             stream))
+    _check(lib, lib.srb_moe_combine_identity(_ptr(y), _ptr(entry_slot), None if weigh_inputs else _ptr(weights), rows, top, width, _ptr(out), _ptr(base),
+                                             _ptr(chosen) if identity else None, experts, _ptr(h) if identity else None,
+                                             _ptr(base_gate), code, stream))
     return out
 
 
@@ -991,7 +1054,7 @@ def route(h: torch.Tensor, router: torch.Tensor, top: int, renormalize: bool = F
     lib = load_library("moe")
     _check(lib, lib.srb_moe_route_ex(_ptr(h), _ptr(router), rows, width, router.shape[0], top, int(renormalize),
                                      ROUTER_SCORING[scoring], _ptr(choice_bias), ctypes.c_float(weight_scale),
-                                     ctypes.c_float(norm_eps), _ptr(chosen), _ptr(weights), dtype_code(h.dtype), _stream()))
+                                     ctypes.c_float(norm_eps), _ptr(chosen), _ptr(weights), None, dtype_code(h.dtype), _stream()))
     return chosen, weights
 
 

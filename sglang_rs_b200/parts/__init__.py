@@ -1,10 +1,10 @@
-from .attention import AttentionNames, GroupedQueryAttention
-from .base import (CacheNeed, FeedForward, JointNeed, Mixer, Norm, NormedDelta, PagedKV, Part, PositionEncoding, RequestState,
-                   TensorSpec, matrix_to, scale_to)
+from .attention import AttentionNames, DifferentialMaps, GroupedQueryAttention
+from .base import (CacheNeed, FeedForward, JointNeed, Mixer, Norm, NormedDelta, PagedKV, Part, PendingSum, PositionEncoding,
+                   RequestState, TensorSpec, matrix_to, scale_to)
 from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
 from .delta import DeltaNames, GatedDeltaRule
 from .latent_attention import LatentAttention, LatentAttentionNames
-from .loop import PassEntry, PassSum
+from .loop import PassEntry, PassStep, PassSum
 from .moe import RoutedExperts
 from .embedding import OutputHead, PairTokenEmbedding, TokenEmbedding
 from .hyper import StreamBlock, StreamConnection, StreamNames, StreamSumNorm, StreamUpdate
@@ -26,4 +26,5 @@ __all__ = [
     "LightningAttention", "LightningNames", "PlainMlp", "WavelengthScaling",
     "ParallelBlock", "GroupedRmsNorm", "MambaMixer", "MambaNames", "TokenSideInput", "TokenSideNames",
     "JointNeed", "PostNormBlock", "DeltaNames", "GatedDeltaRule", "MinGru", "MinGruNames", "ParallelMixer", "RampScaling",
+    "DifferentialMaps", "PassStep", "PendingSum",
 ]

@@ -22,19 +22,28 @@ that width).  ``sink``: a number that joins the softmax's denominator as exp(sin
 every head (0 adds one to the denominator), or, with ``names.sink``, a learned number per head; it has no key and no value.  ``names.gate``: a matrix [n_q, hidden] whose
 product with the mixer's input gives a logit per head; head h's result is multiplied by its sigmoid before the output
 projection (the matrix rides in the q/k/v product, the factor in the attention kernel's last step).  A mixer with any of
-these runs ``ops.proj_norm_rope_kv`` between the product and attention; every attention kernel takes the sink and the
+these, or of those below, runs ``ops.proj_norm_rope_kv`` between the product and attention; every attention kernel takes the sink and the
 gates, and the tensor-core ones serve where values are as wide as the keys.  In this arrangement the mixer can stand beside
 another one (``parts/parallel.py``): it reads its columns of a joint product and writes its columns of a joint result.
+
+In the same arrangement: ``keep_first``: beside its window a row sees the sequence's first ``keep_first`` tokens, whose pages
+stay.  ``softcap``: scores go through softcap * tanh(s / softcap).  ``temperature`` (coef, every): q at position p is
+multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  ``maps`` (:class:`DifferentialMaps`): differential attention.  Every
+head has two maps over the same values; a head's query row and a kv head's key row are the two maps' halves beside each other
+(``head_dim`` is the width of both), and with a_1 and a_2 the maps' results the head's is o = a_1 - lambda a_2, divided by
+sqrt(mean(o^2) + eps) over its values, times 1 - diff.  The tensor-core kernels join the maps in their last step, the generic
+one in a kernel behind it; in 32-bit everywhere.
 """
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Dict, Mapping, Optional
+from typing import Dict, Mapping, Optional, Tuple
 
 import torch
 
 from .. import ops
 from .base import PagedKV, PositionEncoding, TensorSpec, matrix_to, scale_to
+from .rope import NoPositionEncoding
 from .stacking import Stackable, aligned, result_columns, stack_rows
 
 
@@ -54,6 +63,27 @@ class AttentionNames:
     sink: Optional[str] = None
 
 
+@dataclass(frozen=True)
+class DifferentialMaps:
+    """Two maps per head: lambda = exp(sum(lq1 lk1)) - exp(sum(lq2 lk2)) + ``diff``, one number for the layer, from four
+    checkpoint vectors of half a head's width."""
+    diff: float
+    eps: float
+    lq1: str
+    lk1: str
+    lq2: str
+    lk2: str
+
+    def names(self) -> Tuple[str, str, str, str]:
+        return (self.lq1, self.lk1, self.lq2, self.lk2)
+
+    def join(self, tensors: Mapping[str, torch.Tensor]) -> "ops.MapJoin":
+        """The constants of the kernels (a number of the checkpoint, so it is taken once, in 64-bit, at load)."""
+        q1, k1, q2, k2 = (tensors[name].to("cpu", torch.float64) for name in self.names())
+        weight = float(torch.exp((q1 * k1).sum()) - torch.exp((q2 * k2).sum())) + self.diff
+        return ops.MapJoin(weight, 1.0 - self.diff, self.eps)
+
+
 class GroupedQueryAttention(Stackable):
     graph_safe = True
     #: what the attention kernels take: the generic one gives a warp to each query head of a kv head (at most
@@ -64,7 +94,9 @@ class GroupedQueryAttention(Stackable):
     def __init__(self, hidden: int, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                  position: PositionEncoding, names: AttentionNames, *, qk_norm_eps: Optional[float] = None,
                  window: Optional[int] = None, chunk: Optional[int] = None, whole_norm: bool = False,
-                 value_dim: Optional[int] = None, sink: Optional[float] = None, partial_sums: bool = True):
+                 value_dim: Optional[int] = None, sink: Optional[float] = None, partial_sums: bool = True,
+                 keep_first: int = 0, softcap: Optional[float] = None, temperature: Optional[Tuple[float, int]] = None,
+                 maps: Optional[DifferentialMaps] = None):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} kv heads")
         if not 0 < head_dim <= self.MAX_HEAD_DIM:
@@ -86,7 +118,20 @@ class GroupedQueryAttention(Stackable):
         self.partial_sums = bool(partial_sums)
         #: the arrangement that ``ops.proj_norm_rope_kv`` prepares
         self.wide = (self.whole_norm or self.vd != self.d or self.sink is not None or names.gate is not None
-                     or names.sink is not None)
+                     or names.sink is not None or bool(keep_first) or softcap is not None or temperature is not None
+                     or maps is not None)
+        if keep_first and (window is None or chunk is not None):
+            raise ValueError("first tokens are kept behind a window, and not together with a chunk")
+        if softcap is not None and not softcap > 0:
+            raise ValueError("the cap on the scores must be positive")
+        if temperature is not None and not temperature[1] > 0:
+            raise ValueError("the query temperature needs a positive number of positions per step")
+        if maps is not None and (head_dim % 2 or not isinstance(position, NoPositionEncoding) or names.q_norm or names.k_norm or names.gate
+                                 or names.sink or sink is not None):
+            raise ValueError("two maps per head are built without a rotation, norms of q and k, sinks and gates")
+        self.keep_first, self.softcap, self.temperature, self.maps = int(keep_first), softcap, temperature, maps
+        #: how the kernels join the two maps of a head; known from load on
+        self.join: Optional[ops.MapJoin] = None
         if self.sink is not None and names.sink is not None:
             raise ValueError("a sink is one number for all heads or a learned one per head, not both")
         if not self.wide and num_heads // num_kv_heads > self.MAX_HEADS_PER_KV_HEAD:
@@ -102,10 +147,12 @@ class GroupedQueryAttention(Stackable):
         self.w_qkv = self.w_o = self.b_qkv = self.b_o = self.q_norm = self.k_norm = self.sinks = None
 
     def cache_need(self) -> PagedKV:
-        return PagedKV(self.n_kv, self.d, self.window, value_dim=None if self.vd == self.d else self.vd)
+        return PagedKV(self.n_kv, self.d, self.window, value_dim=None if self.vd == self.d else self.vd,
+                       keep_first=self.keep_first)
 
     def split_scratch(self):
-        return (self.n_q * self.vd, self.n_q * 2)
+        results = self.n_q * (2 if self.maps is not None else 1)
+        return (results * self.vd, results * 2)
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         n = self.names
@@ -124,6 +171,9 @@ class GroupedQueryAttention(Stackable):
             specs[n.gate] = TensorSpec((self.n_q, self.hidden))
         if n.sink:
             specs[n.sink] = TensorSpec((self.n_q,))
+        if self.maps is not None:
+            for name in self.maps.names():
+                specs[name] = TensorSpec((self.d // 2,))
         for name, width in ((n.q_bias, self.n_q * self.d), (n.k_bias, self.n_kv * self.d),
                             (n.v_bias, self.n_kv * self.d), (n.o_bias, self.hidden)):
             if name:
@@ -150,6 +200,8 @@ class GroupedQueryAttention(Stackable):
         self.sinks = torch.full((self.n_q,), self.sink, dtype=torch.float32, device=device) if self.sink is not None else None
         if n.sink:
             self.sinks = scale_to(tensors[n.sink], device)
+        if self.maps is not None:
+            self.join = self.maps.join(tensors)
         first = torch.cat(stacked, dim=0)
         self.q_norm = scale_to(tensors[n.q_norm], device) if n.q_norm else None
         self.k_norm = scale_to(tensors[n.k_norm], device) if n.k_norm else None
@@ -211,6 +263,8 @@ class GroupedQueryAttention(Stackable):
         heads of 64 or 128), the generic kernel elsewhere; the sink, the gates and the factor ``scale`` go to whichever
         runs."""
         chunk, sinks = self.chunk or 0, self.sinks
+        terms = dict(keep_first=self.keep_first, softcap=self.softcap)
+        maps = 2 if self.join is not None else 1
         # (the tensor-core kernels for prompt portions store 16 bytes at a time)
         same_width = self.vd == self.d and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
         for launch in batch.launches:
@@ -219,35 +273,37 @@ class GroupedQueryAttention(Stackable):
                     q.dtype, self.n_q, self.n_kv, self.d, cache.k_pool.shape[2]):
                 ops.tiled_attention_tc(q, cache.k_pool, cache.v_pool, out, launch.wide_tiles, batch.block_table,
                                        scale=self.scale, window=self.window or 0, error_word=ctx.error_word, chunk=chunk,
-                                       sinks=sinks, gates=gates, out_scale=scale)
+                                       sinks=sinks, gates=gates, out_scale=scale, join=self.join, **terms)
                 continue
-            if same_width and launch.tiles is not None and ops.tiled_attention_takes(q.dtype, self.n_q, self.n_kv, self.d):
+            if same_width and maps == 1 and launch.tiles is not None and ops.tiled_attention_takes(q.dtype, self.n_q, self.n_kv, self.d):
                 ops.tiled_attention(q, cache.k_pool, cache.v_pool, out, launch.tiles, batch.block_table,
                                     scale=self.scale, window=self.window or 0, error_word=ctx.error_word, chunk=chunk,
-                                    sinks=sinks, gates=gates, out_scale=scale)
+                                    sinks=sinks, gates=gates, out_scale=scale, **terms)
                 continue
             row_gates = None if gates is None else gates[b:e]
             if (same_width and launch.tiles is None and launch.split_size and batch.counters is not None
                     and batch.counters.numel() >= (e - b) * self.n_kv
-                    and ops.decode_attention_takes(q.dtype, self.n_q, self.n_kv, self.d)):
+                    and ops.decode_attention_takes(q.dtype, self.n_q, self.n_kv, self.d, maps)):
                 ops.decode_attention(q[b:e], cache.k_pool, cache.v_pool, out[b:e], ctx.positions[b:e],
                                      ctx.row_request[b:e], batch.block_table, scale=self.scale,
                                      window=self.window or 0, scratch_acc=batch.scratch_acc,
                                      scratch_ml=batch.scratch_ml, counters=batch.counters,
                                      error_word=ctx.error_word, max_keys=launch.max_keys, chunk=chunk, sinks=sinks,
-                                     gates=row_gates, out_scale=scale)
+                                     gates=row_gates, out_scale=scale, join=self.join, **terms)
                 continue
             ops.paged_attention(q[b:e], cache.k_pool, cache.v_pool, out[b:e], ctx.positions[b:e],
                                 ctx.row_request[b:e], batch.block_table, scale=self.scale,
                                 window=self.window or 0, split_size=launch.split_size,
                                 max_splits=launch.max_splits, scratch_acc=batch.scratch_acc,
                                 scratch_ml=batch.scratch_ml, error_word=ctx.error_word, chunk=chunk, sinks=sinks,
-                                gates=row_gates, out_scale=scale)
+                                gates=row_gates, out_scale=scale, join=self.join, **terms)
 
     def mix(self, ctx, cache, proj: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
-        """Norms over the whole projections or per head, values of their own width, a sink and a gate per head: one kernel
-        between the product and attention, the attention kernels with the sink in the denominator and the gate and the
-        factor in their last step."""
+        """Norms over the whole projections or per head, values of their own width, a sink and a gate per head, a query
+        temperature: one kernel between the product and attention, the attention kernels with the sink in the denominator, the
+        cap on the scores, and the gate, the join of two maps and the factor in their last step."""
+        if self.maps is not None and scale != 1.0:
+            raise NotImplementedError("a factor on the result of two joined maps is not built")
         batch, rows = ctx.paged[cache.group], proj.shape[-2]
         rotary = self.position.fused_rotary()
         if rotary is not None and rotary.angles is not None:
@@ -260,6 +316,6 @@ class GroupedQueryAttention(Stackable):
             self.qk_norm_eps if self.qk_norm_eps is not None else 0.0, rotary.inv_freq if rotary else None,
             rotary.rotary_dim if rotary else 0, rotary.interleaved if rotary else False, self.n_q, self.n_kv, self.d,
             self.vd, ctx.error_word, magnitude=rotary.magnitude if rotary is not None else 1.0, gate_out=gates,
-            per_head=not self.whole_norm)
+            per_head=not self.whole_norm, temperature=self.temperature)
         heads = out.as_strided((rows, self.n_q, self.vd), (out.stride(0), self.vd, 1))
         self._attend(ctx, cache, batch, q, heads, gates, scale)

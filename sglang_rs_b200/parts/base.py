@@ -52,12 +52,19 @@ class PagedKV:
     """A mixer that keeps keys and values per token.  ``window`` None keeps all of them;
     a number keeps only what the last ``window`` positions can still see.  ``values`` False keeps one
     row per token and kv head only (a latent that serves as key and as value): no value pool is made.
-    ``value_dim``: the width of a value row where it differs from the keys' ``head_dim`` (None: the same)."""
+    ``value_dim``: the width of a value row where it differs from the keys' ``head_dim`` (None: the same).
+    ``keep_first``: with a window, how many of a sequence's first tokens every later position sees beside it (their pages
+    stay)."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     values: bool = True
     value_dim: Optional[int] = None
+    keep_first: int = 0
+
+    def __post_init__(self):
+        if self.keep_first < 0 or (self.keep_first and self.window is None):
+            raise ValueError("first tokens are kept behind a window: there is none, or their number is negative")
 
     @property
     def value_width(self) -> int:
@@ -110,6 +117,15 @@ class NormedDelta:
     norm, the sum and the next norm run in one kernel."""
     values: torch.Tensor
     norm: "Norm"
+
+
+@dataclass
+class PendingSum:
+    """A pending term of the residual sum and one row that is added to every row beside it: the hidden state is
+    ``residual + values + row`` (``values``: a tensor, a :class:`NormedDelta` or None; ``row``: float32 [width]).  The norms that
+    take a :class:`NormedDelta` take this too, in the same kernel."""
+    values: Union[torch.Tensor, NormedDelta, None]
+    row: torch.Tensor
 
 
 class Norm(Part):

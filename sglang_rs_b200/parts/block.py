@@ -3,7 +3,7 @@
 Pre-norm residual form (reference: crates/sglang-srt/src/cpu_reference.rs:257-317):
 h' = h + mixer(norm_1(h)); h'' = h' + feed_forward(norm_2(h')).  The hidden state travels
 as (residual, delta) with h = residual + delta; each norm takes the pending sum first, in
-32-bit, so no separate add kernel runs.  :class:`SandwichBlock` norms each sublayer on both sides;
+32-bit, so no separate add kernel runs; a layer may end after its mixer.  :class:`SandwichBlock` norms each sublayer on both sides;
 :class:`PostNormBlock` norms only what a sublayer returns;
 :class:`ParallelBlock` runs mixer and feed-forward side by side from one norm.
 """
@@ -19,7 +19,10 @@ from .norm import rounded_sum
 
 
 class PreNormBlock(Part):
-    def __init__(self, input_norm: Norm, mixer: Mixer, post_norm: Norm, feed_forward: FeedForward):
+    def __init__(self, input_norm: Norm, mixer: Mixer, post_norm: Optional[Norm] = None,
+                 feed_forward: Optional[FeedForward] = None):
+        if (feed_forward is None) != (post_norm is None):
+            raise ValueError("a feed-forward comes with the norm ahead of it, or not at all")
         self.input_norm, self.mixer, self.post_norm, self.feed_forward = input_norm, mixer, post_norm, feed_forward
 
     @property
@@ -27,7 +30,7 @@ class PreNormBlock(Part):
         return all(part.graph_safe for part in self.parts())
 
     def parts(self):
-        return (self.input_norm, self.mixer, self.post_norm, self.feed_forward)
+        return tuple(part for part in (self.input_norm, self.mixer, self.post_norm, self.feed_forward) if part is not None)
 
     def cache_need(self):
         return self.mixer.cache_need()
@@ -51,7 +54,7 @@ class PreNormBlock(Part):
         from ..ops.records import SxAttention, SxBlock, SxGatedMlp, SxNorm
         found = [part.native_record() if hasattr(part, "native_record") else None for part in self.parts()]
         kinds = (SxNorm, SxAttention, SxNorm, SxGatedMlp)
-        if not all(isinstance(record, kind) for record, kind in zip(found, kinds)):
+        if len(found) != len(kinds) or not all(isinstance(record, kind) for record, kind in zip(found, kinds)):
             return None
         return SxBlock(*found)
 
@@ -59,6 +62,8 @@ class PreNormBlock(Part):
                 delta: Optional[torch.Tensor]) -> Tuple[torch.Tensor, torch.Tensor]:
         normed = self.input_norm.add_norm(residual, delta, ctx.dtype)
         delta = self.mixer.forward(ctx, cache, normed)
+        if self.feed_forward is None:
+            return residual, delta
         normed = self.post_norm.add_norm(residual, delta, ctx.dtype)
         delta = self.feed_forward.forward(ctx, normed)
         return residual, delta

@@ -5,6 +5,8 @@ matrix [width, 2 width], and the pass's own vector step[t] (t = 0, 1, ...: the n
 The product's result and the sum are 32-bit: they become the residual stream.
 
 :class:`PassSum` is the head of a pass without tensors: x <- x + x0, the embedding output added to the stream, in 32-bit.
+
+:class:`PassStep` adds the pass's own vector alone: x <- x + step[t].
 """
 from __future__ import annotations
 
@@ -13,7 +15,7 @@ from typing import Dict, Mapping
 import torch
 
 from .. import ops
-from .base import Part, TensorSpec, matrix_to, scale_to
+from .base import Part, PendingSum, TensorSpec, matrix_to, scale_to
 from .norm import add_pending
 
 
@@ -51,3 +53,26 @@ class PassSum(Part):
     def forward(self, ctx, residual: torch.Tensor, delta, origin: torch.Tensor, pass_index: int) -> torch.Tensor:
         add_pending(residual, delta, None, None, addend=origin)
         return residual
+
+
+class PassStep(Part):
+    """x <- x + step[t], the vector of pass t, right before the pass's first layer.  Nothing is launched here: the vector
+    travels on beside the pending term (:class:`PendingSum`) and is added by the kernel that takes the sum and the next norm."""
+    graph_safe = True
+    in_place = True
+    #: the embedding output is not looked at
+    reads_origin = False
+
+    def __init__(self, width: int, passes: int, step_name: str):
+        self.width, self.passes, self.step_name = int(width), int(passes), step_name
+        self.steps = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        return {self.step_name: TensorSpec((self.passes, self.width))}
+
+    def load(self, tensors: Mapping[str, torch.Tensor], device, dtype: torch.dtype) -> None:
+        # rows of their own tensors, so that each starts on a 16-byte border whatever the width
+        self.steps = [scale_to(row.clone(), device) for row in tensors[self.step_name]]
+
+    def forward(self, ctx, residual: torch.Tensor, delta, origin, pass_index: int):
+        return residual, PendingSum(delta, self.steps[pass_index])

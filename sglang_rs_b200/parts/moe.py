@@ -17,6 +17,9 @@ Scores may be the sigmoid of each logit instead of the softmax over all (``scori
 ``renormalize`` the chosen scores are divided by their sum plus ``norm_eps``; ``weight_scale`` multiplies the weights.
 An activation with a parameter (``swiglu_clamp``: g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit) and
 u' = clamp(u, -limit, limit)) takes it as ``activation_param``.
+``weigh_inputs``: a chosen expert's weight multiplies its input, not its result: the sum is of expert_e(s_e h).
+``shared_gate_name``: a row [1, width] whose product with h gives one logit per row; its sigmoid, in 32-bit, multiplies the
+shared expert's term (the row is stacked under the router's, so the logit comes from the router's product).
 ``identity``: the router has this many outputs behind the experts' that stand for experts without tensors, whose result is
 their input: a row that chooses one gets weight * h as that term.  Scores, the correction and the choice run over all
 router outputs alike (the router matrix and the correction have experts + identity rows).
@@ -39,7 +42,8 @@ class RoutedExperts(FeedForward):
                  expert_names: Callable[[int], GatedMlpNames], renormalize: bool = False, *,
                  router_bias_name: Optional[str] = None, shared: Optional[FeedForward] = None,
                  scoring: str = "softmax", choice_bias_name: Optional[str] = None, weight_scale: float = 1.0,
-                 norm_eps: float = 0.0, activation_param: float = 0.0, identity: int = 0):
+                 norm_eps: float = 0.0, activation_param: float = 0.0, identity: int = 0, weigh_inputs: bool = False,
+                 shared_gate_name: Optional[str] = None):
         if activation not in ops.ACTIVATIONS:
             raise ValueError(f"unsupported activation {activation}; available: {sorted(ops.ACTIVATIONS)}")
         if scoring not in ops.ROUTER_SCORING:
@@ -50,7 +54,11 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"{top} chosen experts of {experts + identity}")
         if experts + identity > 1024 or top > 32:
             raise ValueError(f"the router kernel takes at most 1024 experts and 32 chosen ones, not {experts + identity} and {top}")
-        self.identity = int(identity)
+        if shared_gate_name and (shared is None or router_bias_name):
+            raise ValueError("a gate of the shared expert needs that expert and a router without bias")
+        if weigh_inputs and identity:
+            raise ValueError("weights on inputs are not built for experts that return their input")
+        self.identity, self.weigh_inputs, self.shared_gate_name = int(identity), bool(weigh_inputs), shared_gate_name
         self.hidden, self.inner, self.experts, self.top = int(hidden), int(inner), int(experts), int(top)
         self.activation, self.router_name, self.renormalize = activation, router_name, bool(renormalize)
         self.names = [expert_names(e) for e in range(self.experts)]
@@ -71,6 +79,8 @@ class RoutedExperts(FeedForward):
             specs[self.choice_bias_name] = TensorSpec((routes,))
         if self.shared is not None:
             specs.update(self.shared.tensor_specs())
+        if self.shared_gate_name:
+            specs[self.shared_gate_name] = TensorSpec((1, self.hidden))
         for n in self.names:
             if self.gated:
                 specs[n.gate] = TensorSpec((self.inner, self.hidden))
@@ -79,7 +89,10 @@ class RoutedExperts(FeedForward):
         return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor], device, dtype: torch.dtype) -> None:
-        self.router = matrix_to(tensors[self.router_name], device, dtype)
+        router = tensors[self.router_name]
+        if self.shared_gate_name:
+            router = torch.cat([router, tensors[self.shared_gate_name].to(router.dtype)], dim=0)
+        self.router = matrix_to(router, device, dtype)
         # per expert the gate rows over the up rows: the two matrices of a tile then lie a fixed distance apart
         if self.gated:
             stacked = [torch.cat([tensors[n.gate], tensors[n.up]], dim=0) for n in self.names]
@@ -100,4 +113,5 @@ class RoutedExperts(FeedForward):
                                   self.renormalize, ctx.error_word, gated=self.gated, router_bias=self.router_bias,
                                   base=base, scoring=self.scoring, choice_bias=self.choice_bias,
                                   weight_scale=self.weight_scale, norm_eps=self.norm_eps,
-                                  activation_param=self.activation_param, identity=self.identity)
+                                  activation_param=self.activation_param, identity=self.identity,
+                                  weigh_inputs=self.weigh_inputs, base_gated=bool(self.shared_gate_name))

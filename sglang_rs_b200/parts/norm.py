@@ -12,7 +12,7 @@ from typing import Dict, Mapping, Optional
 import torch
 
 from .. import ops
-from .base import Norm, NormedDelta, TensorSpec, scale_to
+from .base import Norm, NormedDelta, PendingSum, TensorSpec, scale_to
 
 
 class RmsNorm(Norm):
@@ -123,8 +123,13 @@ class LayerNorm(Norm):
 def add_pending(residual: torch.Tensor, delta, outer, out: Optional[torch.Tensor],
                 row_index: Optional[torch.Tensor] = None, extra: Optional[torch.Tensor] = None,
                 addend: Optional[torch.Tensor] = None) -> None:
-    """residual += delta (a tensor, a :class:`NormedDelta` or None) (+ ``addend``), then ``out`` = ``outer`` of the sum."""
+    """residual += delta (a tensor, a :class:`NormedDelta`, a :class:`PendingSum` or None) (+ ``addend``), then ``out`` =
+    ``outer`` of the sum."""
     inner = None
+    if isinstance(delta, PendingSum):
+        if addend is not None:
+            raise TypeError("a pending sum has its second term already")
+        delta, addend = delta.values, delta.row
     if isinstance(delta, NormedDelta):
         inner, delta = delta.norm.spec(), delta.values
     ops.norm_add_norm(residual, delta, inner, outer, out, row_index=row_index, write_residual=row_index is None,
