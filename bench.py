@@ -159,7 +159,7 @@ def main() -> int:
     parser.add_argument("--warmup", type=int, default=3)
     parser.add_argument("--impl", default="ours", choices=("ours", "reference"))
     parser.add_argument("--shape", default="qwen3-8b", choices=sorted(SHAPES))
-    parser.add_argument("--mode", default="decode", choices=("decode", "prefill", "serve", "compare-cublas", "kernels", "ablate", "probe-overlap", "timeline", "gegepel", "tosivik", "desarax", "titatar", "sogodra"))
+    parser.add_argument("--mode", default="decode", choices=("decode", "prefill", "serve", "compare-cublas", "kernels", "ablate", "probe-overlap", "timeline", "gegepel", "tosivik", "desarax", "titatar", "sogodra", "tekilorn"))
     parser.add_argument("--rows", default="1,8,64,2048", help="--mode compare-cublas: the row counts, comma-separated")
     parser.add_argument("--layers", type=int, default=None, help="fewer than the shape has, only where memory or time needs it")
     parser.add_argument("--batch", type=int, default=8)
@@ -172,7 +172,7 @@ def main() -> int:
     parser.add_argument("--requests", type=int, default=128, help="--mode serve: number of requests")
     parser.add_argument("--seed", type=int, default=0)
     parser.add_argument("--width", type=int, default=2048, choices=(1024, 2048, 4096),
-                        help="--mode tosivik, --mode desarax and --mode sogodra: the model's width; heads, feed-forwards and the shape beside it follow")
+                        help="--mode tosivik, --mode desarax, --mode sogodra and --mode tekilorn: the model's width; heads, feed-forwards and the shape beside it follow")
     args = parser.parse_args()
 
     if args.impl == "reference":
@@ -195,6 +195,8 @@ def main() -> int:
         return titatar_beside_gegepel(args, warmup)
     if args.mode == "sogodra":
         return sogodra_beside_tosivik(args, warmup)
+    if args.mode == "tekilorn":
+        return tekilorn_beside_titatar(args, warmup)
 
     if args.mode == "timeline":
         # the kernels of a decode step, built with marks that record when each block starts, stops waiting for the
@@ -978,6 +980,37 @@ def sogodra_beside_tosivik(args, warmup) -> int:
     note = {"layers": layers, "width": args.width, "vocab": vocab, "sogodra_layers": designs["sogodra"]["layers"][:4],
             "tosivik_layers": designs["tosivik"]["layers"][:4]}
     return designs_side_by_side(args, warmup, "sogodra", designs, vocab, note)
+
+
+def tekilorn_beside_titatar(args, warmup) -> int:
+    """``--mode tekilorn``: prefill and decode of a Tekilorn model with layers of a real model's size (random weights) beside a
+    Titatar model of equal width, depth and layer runs (the closest design: grouped attention in a window with a gate per head,
+    routed experts beside a shared one, a stretch of layers walked twice).  Heads of 128 on a quarter as many kv heads and a
+    window of 1,024 in the first two layers, no window in the others: there Tekilorn has two maps of 64 entries per head over
+    values of 128 with a cap on the scores, Titatar one of 128 entries.  A dense feed-forward of three widths in the first
+    layer, then 64 experts of 11/16 of the width (6 chosen) and a shared one of twice that.  ``--width`` 1024, 2048 or 4096."""
+    layers = args.layers if args.layers is not None else 4
+    vocab, width = 32768, args.width
+    loop = {"start": 1, "stop": min(3, layers), "times": 2} if layers >= 2 else None
+    heads = {"heads": width // 128, "kv_heads": max(1, width // 512)}
+    window = {**heads, "dim": 128, "vdim": 128, "scale": 1.0 / math.sqrt(128), "rot": {"base": 500000.0, "dims": 128}}
+    maps = {**heads, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.6, "softcap": 50.0, "q_temp": {"coef": 0.1, "every": 4096}}
+    ff, expert, shared, router = 3 * width, 11 * width // 16, 11 * width // 8, {"experts": 64, "top": 6}
+    ours = [("attention_2", {**window, "mask": {"size": 1024, "keep_first": 4}})] * 2 + [("attention", maps)] * 2
+    theirs = [{**window, "mask": {"size": 1024}}] * 2 + [window] * 2
+    designs = {
+        "tekilorn": {"architecture": "Tekilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "loop": loop, "layers": [
+            {"type": ours[i % 4][0], "mixer": ours[i % 4][1], "mlp": {"kind": "dense", "ff": ff, "limit": 7.0} if i % 4 == 0 else
+             {"kind": "moe", "router": router, "expert": {"ff": expert, "limit": 7.0}, "shared": {"ff": shared, "limit": 7.0}}}
+            for i in range(layers)]},
+        "titatar": {"architecture": "Titatar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "loop": loop, "embedding": {"scale": 1.0},
+                    "layers": [{"type": "attention", "mixer": theirs[i % 4], "mlp": {"kind": "dense", "ff": ff} if i % 4 == 0 else
+                                {"kind": "moe", "router": router, "expert": {"ff": expert}, "shared": {"ff": shared}}}
+                               for i in range(layers)]},
+    }
+    note = {"layers": layers, "width": width, "vocab": vocab, "tekilorn_layers": designs["tekilorn"]["layers"][:4],
+            "titatar_layers": designs["titatar"]["layers"][:4], "loop": loop}
+    return designs_side_by_side(args, warmup, "tekilorn", designs, vocab, note)
 
 
 def designs_side_by_side(args, warmup, mode, designs, vocab, note) -> int:

@@ -49,6 +49,9 @@ struct TcArgs {
   float out_scale;         // a factor on every result
   int keep_first;          // with a window: the sequence's first keys that stay visible behind it
   float cap_log2;          // softcap * log2 e, or 0; with a cap `scale_log2` brings a score to 2 s / softcap in units of log2
+  float cap_y;             // a score times this is s / softcap
+  float cap_poly[7];       // softcap * log2 e * tanh(y) = y (c0 + c1 y^2 + ... + c6 y^12) for |y| <= 1
+  int fixed_max;           // capped scores are small enough that exponentials need no running maximum
   float map_lambda, map_scale, map_eps;    // two maps per head: o = a_1 - map_lambda a_2, over its root mean square, times map_scale
 };
 
@@ -78,6 +81,11 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
   asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
   return d;
 }
+__device__ __forceinline__ float max3_abs(float a, float b, float c) {
+  float d;
+  asm("max.abs.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
 __device__ __forceinline__ float ex2(float a) {
   float d;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(d) : "f"(a));
@@ -94,6 +102,11 @@ __device__ __forceinline__ void unpack2(unsigned long long v, float& a, float& b
 __device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
   unsigned long long d;
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
+  unsigned long long d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
 }
 __device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigned long long b) {
@@ -306,7 +319,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const bool row_live = r < n_rows;
     const unsigned lane_address = tmem_base + t * HEAD_COLUMNS + ((unsigned)(quarter * 32) << 16);
     const float to_log2 = CAP ? 1.0f : args.scale_log2;    // capped scores are in units of log2 already
-    float m_run = -INFINITY, l_run = 0.f;
+    float m_run = CAP && args.fixed_max ? 0.f : -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int i = 0; i < num_blocks && ok; ++i) {
       const unsigned s_col = S_COL + (i & 1) * TC_KEYS;
@@ -321,9 +334,32 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       float sv[TC_KEYS];
       tmem_load_64(lane_address + s_col, sv);
       if (CAP) {
-        // 2 s / softcap in units of log2 -> softcap * tanh(s / softcap) in units of log2; tanh(y) = 1 - 2 / (e^(2y) + 1)
+        // raw scores -> softcap * tanh(s / softcap) in units of log2.  Scores within the cap (the common case) take a
+        // polynomial of y = s / softcap, which runs beside the exponentials; a block of keys in which some row of the warp
+        // goes beyond it takes tanh(y) = 1 - 2 / (e^(2y) + 1), two more steps of the unit that the exponentials need.
+        float far[4] = {fabsf(sv[0]), fabsf(sv[1]), fabsf(sv[2]), fabsf(sv[3])};
 #pragma unroll
-        for (int j = 0; j < TC_KEYS; ++j) sv[j] = args.cap_log2 * (1.0f - __fdividef(2.0f, ex2(sv[j] * args.scale_log2) + 1.0f));
+        for (int j = 4; j < TC_KEYS - 4; j += 8) {
+          far[0] = max3_abs(far[0], sv[j], sv[j + 1]); far[1] = max3_abs(far[1], sv[j + 2], sv[j + 3]);
+          far[2] = max3_abs(far[2], sv[j + 4], sv[j + 5]); far[3] = max3_abs(far[3], sv[j + 6], sv[j + 7]);
+        }
+        far[0] = max3_abs(far[0], sv[TC_KEYS - 4], sv[TC_KEYS - 3]);
+        far[1] = max3_abs(far[1], sv[TC_KEYS - 2], sv[TC_KEYS - 1]);
+        const bool within = fmaxf(fmaxf(far[0], far[1]), fmaxf(far[2], far[3])) * args.cap_y <= 1.0f;
+        if (__all_sync(0xffffffffu, within)) {
+          const unsigned long long to_y = pack2(args.cap_y, args.cap_y);
+#pragma unroll
+          for (int j = 0; j < TC_KEYS; j += 2) {
+            const unsigned long long y = mul2(pack2(sv[j], sv[j + 1]), to_y), u = mul2(y, y);
+            unsigned long long t = pack2(args.cap_poly[6], args.cap_poly[6]);
+#pragma unroll
+            for (int k = 5; k >= 0; --k) t = fma2(t, u, pack2(args.cap_poly[k], args.cap_poly[k]));
+            unpack2(mul2(t, y), sv[j], sv[j + 1]);
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < TC_KEYS; ++j) sv[j] = args.cap_log2 * (1.0f - __fdividef(2.0f, ex2(sv[j] * args.scale_log2) + 1.0f));
+        }
       }
       if (!all_visible) {
 #pragma unroll
@@ -332,43 +368,45 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           if (!(row_live && key <= pos_r && (key >= lowest_r || key < args.keep_first))) sv[j] = -INFINITY;
         }
       }
-      // three-input maxima, four chains
-      float mx[4] = {sv[0], sv[1], sv[2], sv[3]};
+      if (!CAP || !args.fixed_max) {
+        // three-input maxima, four chains
+        float mx[4] = {sv[0], sv[1], sv[2], sv[3]};
 #pragma unroll
-      for (int j = 4; j < TC_KEYS - 4; j += 8) {
-        mx[0] = max3(mx[0], sv[j], sv[j + 1]); mx[1] = max3(mx[1], sv[j + 2], sv[j + 3]);
-        mx[2] = max3(mx[2], sv[j + 4], sv[j + 5]); mx[3] = max3(mx[3], sv[j + 6], sv[j + 7]);
-      }
-      mx[0] = max3(mx[0], sv[TC_KEYS - 4], sv[TC_KEYS - 3]);
-      mx[1] = max3(mx[1], sv[TC_KEYS - 2], sv[TC_KEYS - 1]);
-      const float m_block = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * to_log2;   // in units of log2
-      // the running maximum moves only when it must: P stays below 2^8
-      float corr = 1.f;
-      bool rescale = false;
-      if (m_block > m_run + TC_RESCALE_STEP || m_run == -INFINITY) {
-        const float m_new = fmaxf(m_run, m_block);
-        if (m_new > -INFINITY) {
-          corr = ex2(m_run - m_new);                       // 0 the first time
-          rescale = m_run > -INFINITY;
-          m_run = m_new;
+        for (int j = 4; j < TC_KEYS - 4; j += 8) {
+          mx[0] = max3(mx[0], sv[j], sv[j + 1]); mx[1] = max3(mx[1], sv[j + 2], sv[j + 3]);
+          mx[2] = max3(mx[2], sv[j + 4], sv[j + 5]); mx[3] = max3(mx[3], sv[j + 6], sv[j + 7]);
         }
+        mx[0] = max3(mx[0], sv[TC_KEYS - 4], sv[TC_KEYS - 3]);
+        mx[1] = max3(mx[1], sv[TC_KEYS - 2], sv[TC_KEYS - 1]);
+        const float m_block = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * to_log2;   // in units of log2
+        // the running maximum moves only when it must: P stays below 2^8
+        float corr = 1.f;
+        bool rescale = false;
+        if (m_block > m_run + TC_RESCALE_STEP || m_run == -INFINITY) {
+          const float m_new = fmaxf(m_run, m_block);
+          if (m_new > -INFINITY) {
+            corr = ex2(m_run - m_new);                       // 0 the first time
+            rescale = m_run > -INFINITY;
+            m_run = m_new;
+          }
+        }
+        if (__any_sync(0xffffffffu, rescale)) {
+          // O is still being added to by P V of the block before: wait for that product
+          ok = mbar_wait(smem_u32(&pv_done[t][(i - 1) & 1]), (unsigned)((i - 1) >> 1) & 1u, &abort_flag);
+          if (!ok) break;
+          tc_fence_after();
+#pragma unroll 1
+          for (int c = 0; c < D; c += 32) {
+            float ov[32];
+            tmem_load_32(lane_address + O_COL + c, ov);
+#pragma unroll
+            for (int j = 0; j < 32; ++j) ov[j] *= corr;
+            tmem_store_32(lane_address + O_COL + c, ov);
+          }
+        }
+        l_run *= corr;
       }
       const float m_use = m_run == -INFINITY ? 0.f : m_run;
-      if (__any_sync(0xffffffffu, rescale)) {
-        // O is still being added to by P V of the block before: wait for that product
-        ok = mbar_wait(smem_u32(&pv_done[t][(i - 1) & 1]), (unsigned)((i - 1) >> 1) & 1u, &abort_flag);
-        if (!ok) break;
-        tc_fence_after();
-#pragma unroll 1
-        for (int c = 0; c < D; c += 32) {
-          float ov[32];
-          tmem_load_32(lane_address + O_COL + c, ov);
-#pragma unroll
-          for (int j = 0; j < 32; ++j) ov[j] *= corr;
-          tmem_store_32(lane_address + O_COL + c, ov);
-        }
-      }
-      l_run *= corr;
       // P = 2^(s * scale * log2 e - m), rounded to bfloat16 pairs, over the scores it came from; the row's sum
       // (two-wide 32-bit multiply-adds and adds; the exponential is one ex2 per score)
       const unsigned long long scale2 = pack2(to_log2, to_log2), neg_m2 = pack2(-m_use, -m_use);
@@ -623,13 +661,23 @@ extern "C" int srb_prefill_attention_tc_terms(const void* q, const void* k_pool,
                                    CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (status != CUDA_SUCCESS) SRB_FAIL("prefill_attention_tc: tensor map of a pool failed with %d", (int)status);
   }
-  TcArgs args;
+  TcArgs args = {};
   args.tiles = tiles; args.block_table = block_table; args.out = (__nv_bfloat16*)out; args.table_stride = table_stride;
   args.n_q = n_q; args.n_kv = n_kv; args.page_size = page_size; args.pool_rows = (int)pool_rows; args.window = window; args.chunk = chunk;
   args.scale_log2 = scale * 1.4426950408889634f; args.error_word = error_word;
   args.sinks = sinks; args.gates = gates; args.out_pitch = out_pitch; args.out_scale = out_scale;
   args.keep_first = p.keep_first; args.cap_log2 = p.softcap * 1.4426950408889634f;
-  if (p.softcap > 0.f) args.scale_log2 *= 2.0f / p.softcap;
+  if (p.softcap > 0.f) {
+    // tanh(y) / y as a polynomial of y^2 on [0, 1]: Chebyshev interpolation at seven nodes, off by at most 1.2e-7
+    static const double tanh_over_y[7] = {0.99999994864557, -0.3333282797860154, 0.1332507614612557, -0.053451646370651876,
+                                          0.020279708287252025, -0.006194324834984364, 0.0010380250971290484};
+    args.scale_log2 *= 2.0f / p.softcap;
+    args.cap_y = scale / p.softcap;
+    for (int k = 0; k < 7; ++k) args.cap_poly[k] = (float)(tanh_over_y[k] * (double)args.cap_log2);
+    // every exponential lies within 2^+-cap_log2: sums over 2^24 keys and products with values stay far from the ends of the
+    // range of a 32-bit float (and of a bfloat16)
+    args.fixed_max = args.cap_log2 <= 80.0f;
+  }
   args.map_lambda = p.map_lambda; args.map_scale = p.map_scale; args.map_eps = p.map_eps;
   cudaStream_t s = (cudaStream_t)stream;
   // two query heads per block when the heads of a kv head pair up

@@ -219,11 +219,18 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
     for (int c = 0; c < BLOCK_T; c += 16) {
       if (token0 + c >= token_limit) break;            // the same for all epilogue warps
       float acc[16];
+      // the factors of these 16 slots, a lane each, fetched ahead of the accumulators
+      const float factor = (EPI == EPI_SILU || EPI == EPI_ACT) && args.slot_weight
+                               ? args.slot_weight[min(token0 + c + (lane & 15), token_limit - 1)] : 1.0f;
       if (ok && num_kb > 0) {
         tmem_load_16(lane_address + c, acc);
       } else {
 #pragma unroll
         for (int j = 0; j < 16; ++j) acc[j] = 0.f;
+      }
+      if ((EPI == EPI_SILU || EPI == EPI_ACT) && args.slot_weight) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) acc[j] *= __shfl_sync(0xffffffffu, factor, j);
       }
       if (EPI == EPI_SILU) {
         if (quarter >= 2) {
@@ -236,8 +243,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
           for (int j = 0; j < 16; ++j) {
             const int token = token0 + c + j;
             if (token >= token_limit) break;
-            const float weight = args.slot_weight ? args.slot_weight[token] : 1.0f;
-            const float g = acc[j] * weight, u = exchange[((quarter & 1) * 32 + lane) * 16 + j] * weight;
+            const float g = acc[j], u = exchange[((quarter & 1) * 32 + lane) * 16 + j];
             reinterpret_cast<__nv_bfloat16*>(args.out)[(size_t)token * args.ldo + feature] =
                 __float2bfloat16_rn(srb_gated<true>(args.activation, g, u, args.act_param));
           }
@@ -256,7 +262,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             reinterpret_cast<__nv_bfloat16*>(args.out)[(size_t)token * args.ldo + feature] = __float2bfloat16_rn(acc[j]);
           } else if (EPI == EPI_ACT) {
             reinterpret_cast<__nv_bfloat16*>(args.out)[(size_t)token * args.ldo + feature] =
-                __float2bfloat16_rn(srb_gated<true>(args.activation, args.slot_weight ? acc[j] * args.slot_weight[token] : acc[j], 1.0f, args.act_param));
+                __float2bfloat16_rn(srb_gated<true>(args.activation, acc[j], 1.0f, args.act_param));
           } else if (EPI == EPI_F32) {
             reinterpret_cast<float*>(args.out)[(size_t)token * args.ldo + feature] = acc[j];
           } else {

@@ -27,6 +27,9 @@ def test_host_books_under_address_and_undefined_behaviour_sanitizers(tmp_path):
     library = str(tmp_path / "host_core_sanitized.so")
     subprocess.check_call(["g++", "-x", "c++", "-std=c++17", "-O1", "-g", "-fsanitize=address,undefined",
                            "-fno-sanitize-recover=undefined", "-shared", "-fPIC", "-o", library, SOURCE])
+    # (what else the child loads is built here: the compiler does not start under AddressSanitizer)
+    from sglang_rs_b200.csrc.build import compile_library
+    compile_library("step_exec")
     # (the child sees no GPU: the CUDA driver does not start under AddressSanitizer, and the host books need none)
     env = dict(os.environ, SRB_LIBRARY_HOST_CORE=library, LD_PRELOAD=runtime("libasan.so"), CUDA_VISIBLE_DEVICES="",
                ASAN_OPTIONS="detect_leaks=0:abort_on_error=1:protect_shadow_gap=0",
