@@ -137,7 +137,7 @@ def test_pages_of_kept_tokens_stay_and_the_others_behind_the_window_go_back(page
 def test_the_pieces_of_keys_that_a_decoded_row_walks():
     from sglang_rs_b200.engine.runner import visible_pieces
     positions = np.arange(0, 400)
-    for window, keep, size in ((None, 0, 32), (40, 0, 32), (40, 6, 32), (33, 70, 32), (1, 3, 64), (500, 9, 128), (64, 64, 64)):
+    for window, keep, size in ((None, 0, 32), (40, 0, 32), (41, 7, 32), (33, 70, 32), (1, 3, 64), (500, 9, 128), (64, 64, 64)):
         pieces, keys = visible_pieces(positions, window, keep, size)
         for p in positions:
             seen = [j for j in range(p + 1) if pt.visible(p, j, window, keep)]
